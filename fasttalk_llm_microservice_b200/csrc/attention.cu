@@ -4,7 +4,7 @@
 // and the softmax probabilities are fp16 with fp32 accumulation: same bytes as bf16, three more
 // mantissa bits, and the dtype the reference runs its engine with, docker-compose.vllm.yml:45).  The
 // K and V slabs of a (page, head) are adjacent, so one attention tile is ONE contiguous
-// 2*64*D*2-byte block that a single bulk-TMA copy (cp.async.bulk, SASS UBLKCP) drops into a
+// 2*64*D*2-byte block that a single bulk-TMA copy (cp.async.bulk) drops into a
 // shared-memory stage.  The 16-byte chunks of every token row are XOR-swizzled already in HBM
 // (rope_kv_append writes them that way), so ldmatrix reads the landed tile conflict-free
 // without a tensor map.

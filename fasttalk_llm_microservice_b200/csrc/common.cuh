@@ -113,7 +113,7 @@ __device__ __forceinline__ uint64_t policy_evict_last() {
 }
 
 // ------------------------------------------------------------------ TMA
-// 1-D bulk copy global -> shared, completion on an mbarrier (SASS: UBLKCP).
+// 1-D bulk copy global -> shared, completion on an mbarrier.
 __device__ __forceinline__ void tma_bulk_g2s(void* dst_smem, const void* src, uint32_t bytes,
                                              uint64_t* bar, uint64_t policy) {
     asm volatile(
@@ -122,7 +122,7 @@ __device__ __forceinline__ void tma_bulk_g2s(void* dst_smem, const void* src, ui
         "l"(src), "r"(bytes), "r"(smem_u32(bar)), "l"(policy)
         : "memory");
 }
-// 2-D tiled tensor-map copy global -> shared (SASS: UTMALDG).  c0 = innermost coordinate.
+// 2-D tiled tensor-map copy global -> shared.  c0 = innermost coordinate.
 __device__ __forceinline__ void tma_tile_2d(void* dst_smem, const CUtensorMap* map, int c0, int c1,
                                             uint64_t* bar, uint64_t policy) {
     asm volatile(
@@ -155,7 +155,7 @@ __device__ __forceinline__ void tc_fence_before() {
 __device__ __forceinline__ void tc_fence_after() {
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 }
-// D[tmem] (+)= A[smem desc] * B[smem desc], bf16 inputs, fp32 accumulate (SASS: UTCHMMA).
+// D[tmem] (+)= A[smem desc] * B[smem desc], bf16 inputs, fp32 accumulate.
 __device__ __forceinline__ void umma_bf16(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc,
                                           uint32_t idesc, uint32_t accumulate) {
     asm volatile(
@@ -230,7 +230,7 @@ __device__ __forceinline__ void mbar_arrive_leader(uint64_t* bar) {
     asm volatile("mbarrier.arrive.shared::cluster.b64 _, [%0];" ::"r"(smem_u32(bar) & kPeerBitMask) : "memory");
 }
 
-// 32 lanes x 16 consecutive fp32 columns of TMEM -> 16 registers per thread (SASS: LDTM).
+// 32 lanes x 16 consecutive fp32 columns of TMEM -> 16 registers per thread.
 __device__ __forceinline__ void tmem_ld16(uint32_t taddr, float* v) {
     uint32_t r[16];
     asm volatile(
