@@ -167,7 +167,8 @@ struct Engine {
 // of its recurrent layers and the fp32 work buffers of a step.
 struct LayeredLayer {
     ft_layer_desc d;
-    size_t cache_off = 0;              // floats: this layer's [num_pages][64][kv_rank] block in lat_cache
+    size_t cache_off = 0;              // floats: this layer's [num_pages][64][kv_rank + rot_dims] block in lat_cache
+    size_t cache16_off = 0;            // bf16: this layer's [num_pages][64][latent_row16] block in lat_cache16
     size_t s_off = 0, tail_off = 0;    // floats inside a state slot: S [heads][dim][vdim], tails [channels][conv - 1]
     // branch mixers: per branch its block in kv_cache (window attention), its S inside a state slot, and what else it keeps
     // there (the running maximum of a matrix memory, the convolution tails of a state space)
@@ -179,7 +180,8 @@ struct Layered {
     ft_layered_model m;
     std::vector<LayeredLayer> layers;
     float* lat_cache = nullptr;
-    void* lat_cache16 = nullptr;       // serving form: bf16 copy of the latents, same places (tensor-core attention)
+    void* lat_cache16 = nullptr;       // serving form: the latents in bf16 for the tensor-core attention (lat_cache is then only
+                                       // there when a layer's sizes are beyond that kernel)
     float* kv_cache = nullptr;         // window-attention branches: per layer [num_pages][64][kv_heads * (dim + vdim)] fp32
     float* state = nullptr;
     size_t slot_stride = 0;            // floats per state slot
@@ -213,6 +215,7 @@ struct Layered {
     // hyper-connected layers: the streams of a step [t_max][streams][width]
     float* streams = nullptr;
     bool hyper = false;
+    bool prenorm = false;
     float* trail = nullptr;            // debug: residual stream after every layer [n_layers][t_max][width]
     bool trail_on = false;
 };
@@ -603,6 +606,11 @@ static int dense(Engine* e, const float* A, const void* hi, const void* lo, cons
     return 0;
 }
 
+// layer forms whose feed-forward reads a normed input of its own: its projections (the router among them) are not part of w_in
+static bool own_ff(const ft_layer_desc& c) {
+    return c.form == FT_LAYER_SANDWICH || c.form == FT_LAYER_HYPER || c.form == FT_LAYER_PRENORM;
+}
+
 // The mixture of experts of one layer: routing from `logits` (row stride ldl, first column o_router), then every (token,
 // choice) pair through its expert, grouped by expert.  Reads the rows of L.hn; leaves the pairs' outputs in L.eout and their
 // weights / places in L.wts / L.slot_pos (the caller's residual kernel gathers them).
@@ -611,14 +619,14 @@ static int run_experts(Engine* e, const ft_layer_desc& c, const float* logits, i
     const int W = L.m.width;
     cudaStream_t st = e->stream;
     auto launched = [&](int n = 1) { e->st.kernel_launches += n; };
-    const bool sandwich = c.form == FT_LAYER_SANDWICH || c.form == FT_LAYER_HYPER;      // forms whose router is a matrix of its own
+    const bool sandwich = own_ff(c);                                  // forms whose router is a matrix of its own
     const int act = sandwich ? c.ff_act : FT_ACT_SWIGLU;
     const int n_up = act == FT_ACT_SWIGLU ? 2 * c.ff : c.ff;          // rows of an expert's first matrix
     const bool scaled_in = c.route_input != 0;                        // the experts read score * row, in sorted order
     const int top = c.top;
     FT_TRY(launch_route(logits, ldl, o_router, c.experts, c.top, sandwich ? 1 : c.groups, sandwich ? 1 : c.keep, L.ids, L.wts,
                         L.seg, L.slot_token, L.slot_pos, T, st, sandwich ? c.route_kind : FT_ROUTE_SOFTMAX,
-                        sandwich ? c.route_norm : 0, sandwich ? c.route_scale : 1.f));
+                        sandwich ? c.route_norm : 0, sandwich ? c.route_scale : 1.f, sandwich ? c.router_bias : nullptr));
     const int pairs = T * top;
     const bool on_tensor = L.tensor && pairs >= kMoeTensorMinPairs && n_up % 128 == 0 && c.ff % 64 == 0 && W % 128 == 0 &&
                            W % 64 == 0;
@@ -878,7 +886,19 @@ static int forward_layered(Engine* e, const Batch& b) {
         h.X = L.streams; h.S = n_streams; h.W = W; h.eps = M.eps;
         h.in_next = in_next; h.nw = nw; h.nb = nb; h.hn = L.hn; h.hi = hn_hi; h.lo = hn_lo;
     };
-    if (L.hyper) {
+    // what a pre-norm joint leaves for the next reader: the stream ahead of layer run `to` (null: the head), normed by nw
+    auto prenorm_next = [&](PreNormArgs& p, const ft_layer_desc* to, const float* nw) {
+        p.x = e->resid; p.W = W; p.eps = M.eps; p.nw = nw; p.hn = L.hn; p.hi = hn_hi; p.lo = hn_lo;
+        p.tokens = d + m.o_tokens; p.positions = d + m.o_pos; p.embed = M.embed; p.pos_embed = M.pos_embed;
+        p.embed_scale = M.embed_scale != 0.f ? M.embed_scale : 1.f;
+        if (to) { p.re_embed = to->re_embed; p.pre_add = to->pre_add; }
+    };
+    if (L.prenorm) {
+        PreNormArgs p;
+        prenorm_next(p, &L.layers[0].d, L.layers[0].d.norm_pre1);
+        p.first = 1;
+        FT_TRY(launch_prenorm_joint(p, T, st));
+    } else if (L.hyper) {
         HyperArgs h;
         const ft_layer_desc& c0 = L.layers[0].d;
         hyper_next(h, c0.hc_in[0], c0.norm_pre1, c0.norm_pre1_b);
@@ -922,23 +942,28 @@ static int forward_layered(Engine* e, const Batch& b) {
         } else {
         const float* mixed = nullptr;      // [T][heads * vdim], input of the output projection
         if (c.mixer == FT_MIXER_LATENT_ATTENTION) {
-            float* cache = L.lat_cache + ll.cache_off;
-            void* cache16 = L.lat_cache16 ? (uint8_t*)L.lat_cache16 + ll.cache_off * 2 : nullptr;
-            FT_TRY(launch_latent_write(L.proj, ld, c.o_dkv, c.dkv_norm, cache, cache16, d + m.o_pos, d + m.o_rows, d + m.o_pt,
-                                       e->max_pages, c.kv_rank, M.eps, T, st));
-            LinearArgs a;                   // queries into latent space, head by head: qlat_h = W_uk_h^T q_h
-            a.A = L.proj + c.o_q; a.lda = ld; a.a_col_stride = c.dim;
+            const int R = c.rot_dims, kd = c.kv_rank + R, hd = c.dim + R;
+            LatentArgs la;
+            la.proj = L.proj; la.ldp = ld; la.o_q = c.o_q; la.o_dkv = c.o_dkv; la.o_gate = c.gate_wide ? -1 : c.o_gate;
+            la.norm_w = c.dkv_norm; la.eps = M.eps; la.rot_freq = c.rot_freq; la.sink = c.sink; la.qlat = L.b1; la.out = L.b2;
+            la.cache = L.lat_cache ? L.lat_cache + ll.cache_off : nullptr;
+            la.cache16 = L.lat_cache16 ? (uint8_t*)L.lat_cache16 + ll.cache16_off * 2 : nullptr;
+            la.part = L.attn_part; la.positions = d + m.o_pos; la.seq_rows = d + m.o_rows; la.page_table = d + m.o_pt;
+            la.max_pages = e->max_pages; la.H = c.heads; la.dim = c.dim; la.rank = c.kv_rank; la.rot = R; la.scale = c.scale;
+            FT_TRY(launch_latent_prep(la, T, st));
+            LinearArgs a;                   // plain query parts into latent space, head by head: qlat_h = W_uk_h^T q_h
+            a.A = L.proj + c.o_q; a.lda = ld; a.a_col_stride = hd;
             a.W = (const __nv_bfloat16*)c.w_uk_t; a.w_stride = (long long)c.kv_rank * c.dim; a.ldw = c.dim;
-            a.C = L.b1; a.ldc = c.heads * c.kv_rank; a.c_col_stride = c.kv_rank;
+            a.C = L.b1; a.ldc = c.heads * kd; a.c_col_stride = kd;
             a.M = T; a.N = c.kv_rank; a.K = c.dim; a.P = c.heads;
             FT_TRY(launch_linear(a, T, st));
-            FT_TRY(launch_latent_attn(L.b1, cache, cache16, L.proj, ld, c.o_gate, L.b2, L.attn_part, d + m.o_pos, d + m.o_rows, d + m.o_pt,
-                                      e->max_pages, c.heads, c.kv_rank, c.scale, T, st));
+            FT_TRY(launch_latent_attn(la, T, st));
             LinearArgs v;                   // values out of latent space: o_h = W_uv_h (sum_j p_j c_j)
             v.A = L.b2; v.lda = c.heads * c.kv_rank; v.a_col_stride = c.kv_rank;
             v.W = (const __nv_bfloat16*)c.w_uv; v.w_stride = (long long)c.vdim * c.kv_rank; v.ldw = c.kv_rank;
             v.C = L.b3; v.ldc = c.heads * c.vdim; v.c_col_stride = c.vdim;
             v.M = T; v.N = c.vdim; v.K = c.kv_rank; v.P = c.heads;
+            if (c.gate_wide) { v.gate = L.proj + c.o_gate; v.ldg = ld; }
             FT_TRY(launch_linear(v, T, st));
             launched(4);
             mixed = L.b3;
@@ -980,7 +1005,38 @@ static int forward_layered(Engine* e, const Batch& b) {
         // gains of the norm that the next layer (or the head) reads: one number, or one per coordinate
         const float gain_next = nx ? nx->norm_gain : M.final_norm_gain;
         const float* gain_next_w = nx ? (nx->form == FT_LAYER_SANDWICH ? nx->norm_pre1 : nullptr) : M.final_norm_w;
-        if (c.form == FT_LAYER_HYPER) {
+        if (c.form == FT_LAYER_PRENORM) {
+            const bool has_ff = c.ff_kind != FT_FF_NONE;
+            const float* nw_after = nx ? nx->norm_pre1 : M.final_norm_w;
+            float* trail_row = trail ? L.trail + (size_t)l * e->t_max * W : nullptr;
+            PreNormArgs p1;
+            if (has_ff) prenorm_next(p1, nullptr, c.norm_pre2);
+            else { prenorm_next(p1, nx, nw_after); p1.trail = trail_row; }
+            p1.y0 = y0; p1.gain = c.res_gain[0];
+            FT_TRY(launch_prenorm_joint(p1, T, st));
+            launched();
+            if (has_ff) {
+                PreNormArgs p2;
+                prenorm_next(p2, nx, nw_after);
+                p2.trail = trail_row; p2.gain = c.res_gain[1];
+                if (c.ff_kind == FT_FF_DENSE) {
+                    FT_TRY(run_mlp(e, hn_hi, hn_lo, c.w_gu, c.w_down, c.ff, c.ff_act, L.mix, T));
+                    p2.y0 = L.mix;
+                } else {
+                    const int ldl = c.router_rows > 0 ? c.router_rows : c.experts + (c.shared_gate ? 1 : 0);
+                    FT_TRY(dense(e, L.hn, hn_hi, hn_lo, c.w_router, L.rlog, T, ldl, W));
+                    FT_TRY(run_experts(e, c, L.rlog, ldl, 0, T));
+                    p2.eout = L.eout; p2.wt = L.wts; p2.slot_pos = L.slot_pos; p2.top = c.top;
+                    if (c.shared_ff > 0) {
+                        FT_TRY(run_mlp(e, hn_hi, hn_lo, c.w_shared_up, c.w_shared_down, c.shared_ff, c.ff_act, L.mix, T));
+                        p2.y0 = L.mix;
+                        if (c.shared_gate) { p2.y_gate = L.rlog + c.experts; p2.ldg = ldl; }
+                    }
+                }
+                FT_TRY(launch_prenorm_joint(p2, T, st));
+                launched();
+            }
+        } else if (c.form == FT_LAYER_HYPER) {
             // every stream is rebuilt from the old ones and the sublayer's result; the same kernel forms what reads them next
             const bool has_ff = c.ff_kind != FT_FF_NONE;
             const float* in_after = nx ? nx->hc_in[0] : nullptr;          // the head reads the plain sum
@@ -1105,7 +1161,7 @@ static int forward_layered(Engine* e, const Batch& b) {
                                        L.slot_pos, top, T, W, M.eps, gain_next, hn_hi, hn_lo, st));
             launched();
         }
-        if (L.trail_on && L.trail)
+        if (trail && !L.prenorm)
             FT_CHECK_CUDA(cudaMemcpyAsync(L.trail + (size_t)l * e->t_max * W, e->resid, (size_t)T * W * 4,
                                           cudaMemcpyDeviceToDevice, st));
     }
@@ -1617,6 +1673,10 @@ static int engine_init_layered(Engine* e) {
     FT_CHECK_CUDA(cudaDeviceGetAttribute(&cc_major, cudaDevAttrComputeCapabilityMajor, e->dev));
     FT_REQUIRE(cc_major == 10, "engine: needs an sm_100 GPU (found compute capability %d.x)", cc_major);
     FT_CHECK_CUDA(cudaStreamCreateWithFlags(&e->stream, cudaStreamNonBlocking));
+    if (M.pos_embed) {               // a learned vector per position: no sequence grows beyond the table
+        FT_REQUIRE(M.max_positions >= 1, "engine: a position table without rows");
+        e->cfg.max_context = std::min(e->cfg.max_context, M.max_positions);
+    }
     e->max_pages = ceil_div(c.max_context, kKvTile);
     e->t_max = c.max_batched_tokens;
     e->r_max = c.max_batch;
@@ -1627,7 +1687,8 @@ static int engine_init_layered(Engine* e) {
     e->decode_prefill_cap = c.decode_prefill_cap == 0 ? kDefaultDecodePrefillCap : c.decode_prefill_cap < 0 ? 0 : c.decode_prefill_cap;
 
     // sizes over all layers; places of each layer in the latent cache and in a state slot
-    size_t cache_floats = 0, buf = 1, act_cols = 1;
+    size_t cache_floats = 0, cache16 = 0, buf = 1, act_cols = 1;
+    bool latent_f32 = M.exact_f32 != 0;
     size_t kv_floats = 0, br_q = 0, br_v = 0, br_o = 0, br_fin = 0, br_heads = 0, e_max_s = 1, scan_cn = 0;
     int n_in_max = 1, top_max = 1, heads_max = 1, rank_max = 0;
     size_t vfirst_cols = 0, lstage_cols = 0;
@@ -1637,11 +1698,17 @@ static int engine_init_layered(Engine* e) {
         const ft_layer_desc& d = ll.d;
         FT_REQUIRE(d.n_in >= 1 && d.w_in, "engine: layer %d is incomplete", l);
         const bool hyper = d.form == FT_LAYER_HYPER;
-        const bool sandwich = d.form == FT_LAYER_SANDWICH || hyper;      // forms whose feed-forward has projections of its own
+        const bool pre = d.form == FT_LAYER_PRENORM;
+        const bool sandwich = own_ff(d);
         const bool post = d.form == FT_LAYER_POSTNORM;
         FT_REQUIRE(post == (L.layers[0].d.form == FT_LAYER_POSTNORM), "engine: post-norm layers do not mix with other layer forms");
         FT_REQUIRE(hyper == (L.layers[0].d.form == FT_LAYER_HYPER), "engine: hyper-connected layers do not mix with other layer forms");
-        if (hyper) {
+        FT_REQUIRE(pre == (L.layers[0].d.form == FT_LAYER_PRENORM), "engine: pre-norm layers do not mix with other layer forms");
+        if (pre) {
+            FT_REQUIRE(d.norm_pre1 && (d.ff_kind == FT_FF_NONE || d.norm_pre2) && M.final_norm_w, "engine: pre-norm layer %d lacks norm gains", l);
+            FT_REQUIRE(d.mixer == FT_MIXER_LATENT_ATTENTION, "engine: pre-norm layer %d takes latent attention", l);
+            L.prenorm = true;
+        } else if (hyper) {
             FT_REQUIRE(d.norm_pre1 && (d.ff_kind == FT_FF_NONE || d.norm_pre2), "engine: hyper-connected layer %d lacks norm gains", l);
             FT_REQUIRE(M.streams <= 16 && M.final_norm_w, "engine: a hyper-connected model has 1 to 16 streams and a last norm with gains");
             FT_REQUIRE(d.mixer == FT_MIXER_BRANCHES || (d.mixer == FT_MIXER_CHANNEL_DELTA && d.rank_a == 0 && d.rank_g == 0),
@@ -1786,11 +1853,15 @@ static int engine_init_layered(Engine* e) {
                 L.slot_stride = (L.slot_stride + 3) & ~size_t(3);
             }
         } else if (d.mixer == FT_MIXER_LATENT_ATTENTION) {
-            FT_REQUIRE(d.kv_rank >= 1 && d.w_uk_t && d.w_uv && d.dkv_norm && d.o_q >= 0 && d.o_dkv >= 0 && d.o_gate >= 0,
+            FT_REQUIRE(d.kv_rank >= 1 && d.w_uk_t && d.w_uv && d.dkv_norm && d.o_q >= 0 && d.o_dkv >= 0 && d.o_gate >= 0 &&
+                           d.rot_dims >= 0 && d.rot_dims % 2 == 0 && (d.rot_dims == 0 || d.rot_freq),
                        "engine: latent-attention layer %d is incomplete", l);
             ll.cache_off = cache_floats;
-            cache_floats += (size_t)c.num_pages * kKvTile * d.kv_rank;
-            buf = std::max(buf, (size_t)d.heads * d.kv_rank);
+            cache_floats += (size_t)c.num_pages * kKvTile * (d.kv_rank + d.rot_dims);
+            ll.cache16_off = cache16;
+            cache16 += (size_t)c.num_pages * kKvTile * latent_row16(d.kv_rank, d.rot_dims);
+            if (!latent_attn_mma_ok(d.kv_rank, d.rot_dims)) latent_f32 = true;
+            buf = std::max(buf, (size_t)d.heads * (d.kv_rank + d.rot_dims));
             rank_max = std::max(rank_max, d.kv_rank);
         } else if (d.mixer == FT_MIXER_CHANNEL_DELTA) {
             FT_REQUIRE(d.kv_heads >= 1 && d.heads % d.kv_heads == 0 && d.conv >= 1 && d.rank_a >= 0 && d.rank_g >= 0 &&
@@ -1816,8 +1887,9 @@ static int engine_init_layered(Engine* e) {
                        "engine: layer %d lacks the shared expert's weights", l);
             top_max = std::max(top_max, d.top);
             act_cols = std::max(act_cols, (size_t)std::max(d.ff, sandwich ? d.shared_ff : 0));
-            FT_REQUIRE(d.router_rows == 0 || d.router_rows >= d.experts, "engine: layer %d: router_rows below the expert count", l);
-            e_max_s = std::max(e_max_s, (size_t)std::max(d.experts, d.router_rows));
+            const int logits = d.experts + (d.shared_gate ? 1 : 0);
+            FT_REQUIRE(d.router_rows == 0 || d.router_rows >= logits, "engine: layer %d: router_rows below the expert count", l);
+            e_max_s = std::max(e_max_s, (size_t)std::max(logits, d.router_rows));
         } else if (d.ff_kind == FT_FF_DENSE) {
             FT_REQUIRE((sandwich || post) && d.ff >= 1 && d.w_gu && d.w_down, "engine: dense feed-forward layer %d is incomplete", l);
             act_cols = std::max(act_cols, (size_t)d.ff);
@@ -1836,8 +1908,8 @@ static int engine_init_layered(Engine* e) {
         FT_CHECK_CUDA(cudaMemsetAsync(*p, 0, std::max<size_t>(bytes, 16), e->stream));
         return 0;
     };
-    FT_TRY(alloc(&L.lat_cache, cache_floats * 4));
-    if (M.exact_f32 == 0) FT_TRY(alloc(&L.lat_cache16, cache_floats * 2));
+    if (latent_f32) FT_TRY(alloc(&L.lat_cache, cache_floats * 4));
+    if (M.exact_f32 == 0) FT_TRY(alloc(&L.lat_cache16, cache16 * 2));
     FT_TRY(alloc(&L.state, L.slot_stride * (size_t)c.max_sessions * 4));
     if (kv_floats) FT_TRY(alloc(&L.kv_cache, kv_floats * 4));
     if (br_fin) {

@@ -97,6 +97,7 @@ enum { LIN_PLAIN = 0, LIN_SWIGLU_PAIR = 1, LIN_SOFTCAP = 2, LIN_RELU2 = 3 };
 // LIN_SWIGLU_PAIR: W rows (2j, 2j+1) are (gate_j, up_j); C[r, j] = silu(gate) * up, ldc counts those N/2 columns.
 // LIN_SOFTCAP:     C = cap * tanh(C / cap).
 // LIN_RELU2:       C = max(C, 0)^2.
+// gate (plain epilogue): C = C * sigmoid(gate[r * ldg + p * c_col_stride + n]), the gate's columns laid out as those of C.
 struct LinearArgs {
     const float* A = nullptr;
     const int* a_rows = nullptr;
@@ -107,6 +108,8 @@ struct LinearArgs {
     int lda = 0, ldw = 0, ldc = 0, a_col_stride = 0, c_col_stride = 0;
     int M = 0, N = 0, K = 0, P = 1, epi = LIN_PLAIN;
     float cap = 0.f;
+    const float* gate = nullptr;
+    int ldg = 0;
 };
 // rows_bound: M when batched; an upper bound of seg[P] when grouped
 int launch_linear(const LinearArgs& a, int rows_bound, cudaStream_t stream);
@@ -123,20 +126,36 @@ int launch_combine_norm(float* x, float* hn, const float* proj, int ldp, int o_r
                         const float* mix, const float* eout, const float* wt, const int* slot_pos, int top, int T, int W,
                         float eps, float gain, void* hi, void* lo, cudaStream_t stream);
 int launch_gather_rows(const float* src, const int* idx, float* dst, int n, int W, cudaStream_t stream);
-// cache16 (may be null): a bf16 copy of the latents, what the tensor-core attention reads
-int launch_latent_write(const float* proj, int ldp, int o_dkv, const float* w, float* cache, void* cache16, const int* positions,
-                        const int* seq_rows, const int* page_table, int max_pages, int rank, float eps, int T,
-                        cudaStream_t stream);
+// Latent attention.  A cache row holds [normed latent (rank) | rotated key part (rot)] of its position; queries live in the same
+// space, [folded plain part | rotated part] per head.
+struct LatentArgs {
+    const float* proj = nullptr;                  // [T][ldp]: raw latent (rank columns, then rot columns) at o_dkv, queries at
+    int ldp = 0, o_q = 0, o_dkv = 0;              // o_q (heads x (dim plain | rot)), output-gate logits of the heads at o_gate
+    int o_gate = -1;                              // (< 0: no gate here)
+    const float* norm_w = nullptr;                // [rank]
+    float eps = 0.f;
+    const float* rot_freq = nullptr;              // [rot / 2]
+    const float* sink = nullptr;                  // [H] or null: exp(sink) joins the softmax denominator
+    float* qlat = nullptr;                        // [T][H][rank + rot]
+    float* cache = nullptr;                       // this layer's [pages][64][rank + rot] fp32, or null
+    void* cache16 = nullptr;                      // this layer's [pages][64][latent_row16] bf16, or null
+    float* out = nullptr;                         // [T][H][rank] attended latents
+    float* part = nullptr;                        // room for split keys (see below), or null
+    const int *positions = nullptr, *seq_rows = nullptr, *page_table = nullptr;
+    int max_pages = 0, H = 0, dim = 0, rank = 0, rot = 0;
+    float scale = 1.f;
+};
+// Latent normed, shared key part rotated -> the caches; the rotated part of every query -> qlat.
+int launch_latent_prep(const LatentArgs& a, int T, cudaStream_t stream);
 // With fewer than kLatentSplitPairs (token, head) pairs in a step the keys of each are cut into up to kLatentMaxSplits
-// shares that run side by side; `part` then holds pairs x shares x (kv_rank + 2) floats (null: never split).
+// shares that run side by side; `part` then holds pairs x shares x (rank + 2) floats (null: never split).
 constexpr int kLatentSplitPairs = 2048, kLatentMaxSplits = 8;
 int latent_attn_splits(int T, int H);
-// With cache16 and a latent size the tensor-core kernel is built for (latent_attn_mma_ok) the attention runs on mma.sync
-// from bf16 operands; otherwise on the CUDA cores in fp32.
-bool latent_attn_mma_ok(int rank);
-int launch_latent_attn(const float* qlat, const float* cache, const void* cache16, const float* proj, int ldp, int o_gate,
-                       float* out, float* part, const int* positions, const int* seq_rows, const int* page_table, int max_pages,
-                       int H, int rank, float scale, int T, cudaStream_t stream);
+// With cache16 and sizes the tensor-core kernel is built for (latent_attn_mma_ok) the attention runs on mma.sync from bf16
+// operands and `cache` may be null; otherwise on the CUDA cores in fp32.
+bool latent_attn_mma_ok(int rank, int rot);
+int latent_row16(int rank, int rot);              // columns of a bf16 cache row: both parts padded with zeros to multiples of 32
+int launch_latent_attn(const LatentArgs& a, int T, cudaStream_t stream);
 struct DeltaArgs {
     const float* proj = nullptr;      // [T][ldp]: raw q | k | v at column o_q, beta logits at o_beta
     int ldp = 0, o_q = 0, o_beta = 0;
@@ -164,7 +183,7 @@ int launch_delta(const DeltaArgs& a, const float* gate, const float* out_norm, f
                  cudaStream_t stream, int ldg = 0, int gate_act = 0);
 int launch_route(const float* proj, int ldp, int o_router, int E, int top, int groups, int keep, int* ids, float* wts,
                  int* seg, int* slot_token, int* slot_pos, int T, cudaStream_t stream, int route_kind = FT_ROUTE_SOFTMAX,
-                 int normalise = 0, float scale = 1.f);
+                 int normalise = 0, float scale = 1.f, const float* bias = nullptr);
 
 // ---- branches.cu (branch mixers and the sandwich layer form: ft_branch_desc, FT_LAYER_SANDWICH; everything fp32)
 // x += rms(y) * post_w;  hn = rms(x) * next_w  with  y = s0 * y0 + s1 * y1 + sum_k wt[t, k] * eout[slot_pos[t, k]]
@@ -402,6 +421,32 @@ struct ScanArgs {
 };
 int selective_scan_ws_rows(int rows);             // the ws_rows a step of this many rows needs
 int launch_selective_scan(const ScanArgs& a, int n_req, cudaStream_t stream);
+
+// ---- prenorm.cu (FT_LAYER_PRENORM: the joint between two sublayers)
+// One CTA per row.  With `tokens` and no y0 / top: x = embedding output (a step's first joint).  Otherwise
+//   x += gain[c] * (g(t) * y0[t][c] + sum_k wt[t, k] * eout[slot_pos[t, k]][c])   (each part optional; gain null = ones;
+//   g(t) = sigmoid(y_gate[t * ldg]) when y_gate is given)
+// Then, if asked, x goes to trail as it is, takes the embedding output once more (re_embed) and a vector (pre_add), and
+// hn = x / sqrt(mean(x^2) + eps) * nw with its bf16 planes.  Embedding output: embed[token] * embed_scale + pos_embed[position].
+struct PreNormArgs {
+    float* x = nullptr;
+    int W = 0;
+    float eps = 0.f;
+    int first = 0, re_embed = 0;
+    const int *tokens = nullptr, *positions = nullptr;
+    const void *embed = nullptr, *pos_embed = nullptr;
+    float embed_scale = 1.f;
+    const float *y0 = nullptr, *y_gate = nullptr;
+    int ldg = 0;
+    const float *eout = nullptr, *wt = nullptr;
+    const int* slot_pos = nullptr;
+    int top = 0;
+    const float *gain = nullptr, *pre_add = nullptr, *nw = nullptr;
+    float* trail = nullptr;
+    float* hn = nullptr;
+    void *hi = nullptr, *lo = nullptr;
+};
+int launch_prenorm_joint(const PreNormArgs& a, int T, cudaStream_t stream);
 
 // ---- sampling.cu
 int launch_sample(const float* logits, int B, int V, const float* temperature, const int* top_k,

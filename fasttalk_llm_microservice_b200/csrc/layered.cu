@@ -166,6 +166,7 @@ __global__ void __launch_bounds__(LTHREADS) linear_tile_kernel(LinearArgs a) {
                     float v = acc[i][j];
                     if (a.epi == LIN_SOFTCAP) v = a.cap * tanhf(v / a.cap);
                     else if (a.epi == LIN_RELU2) { v = fmaxf(v, 0.f); v *= v; }
+                    if (a.gate) v *= sigmoid_exact(a.gate[(size_t)r * a.ldg + (size_t)p * a.c_col_stride + n]);
                     C[(size_t)r * a.ldc + n] = v;
                 }
             }
@@ -274,6 +275,8 @@ __global__ void __launch_bounds__(LWARPS * 32) linear_rows_kernel(LinearArgs a) 
                     v = warp_sum(acc[c][i]);
                     if (a.epi == LIN_SOFTCAP) v = a.cap * tanhf(v / a.cap);
                     else if (a.epi == LIN_RELU2) { v = fmaxf(v, 0.f); v *= v; }
+                    if (a.gate && lane == 0 && col0 + c < cols)
+                        v *= sigmoid_exact(a.gate[(size_t)(rb + i) * a.ldg + (size_t)p * a.c_col_stride + col0 + c]);
                 }
                 if (lane == 0 && col0 + c < cols) C[(size_t)(rb + i) * a.ldc + col0 + c] = v;
             }
@@ -475,26 +478,44 @@ int launch_gather_rows(const float* src, const int* idx, float* dst, int n, int 
 }
 
 // ------------------------------------------------------------------ latent attention
-// The latent of token t: c = raw / sqrt(mean(raw^2) + eps) * w, written to page_table[seq_rows[t]][pos / 64], row pos % 64
-// of the layer's cache [page][64][rank] fp32.
-__global__ void __launch_bounds__(128)
-latent_write_kernel(const float* __restrict__ proj, int ldp, int o_dkv, const float* __restrict__ w, float* __restrict__ cache,
-                    __nv_bfloat16* __restrict__ cache16, const int* __restrict__ positions, const int* __restrict__ seq_rows, const int* __restrict__ page_table,
-                    int max_pages, int rank, float eps) {
+// Token t: c = raw / sqrt(mean(raw^2) + eps) * w and the rotated shared key part go to page_table[seq_rows[t]][pos / 64], row
+// pos % 64 of the layer's caches ([page][64][rank + rot] fp32; bf16 with both parts padded to multiples of 32); the rotated part
+// of every query head goes to qlat.  Pairs (i, i + rot / 2); the angle's sine and cosine are formed once per token.
+__global__ void __launch_bounds__(128) latent_prep_kernel(LatentArgs a, int row16, int rot_at16) {
     __shared__ float red[33];
-    const int t = blockIdx.x;
-    const float* raw = proj + (size_t)t * ldp + o_dkv;
+    extern __shared__ float trig[];                        // [rot / 2] cosines, [rot / 2] sines
+    const int t = blockIdx.x, rank = a.rank, rot = a.rot, half = rot >> 1;
+    const float* pr = a.proj + (size_t)t * a.ldp;
+    const float* raw = pr + a.o_dkv;
+    const int pos = a.positions[t];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * a.rot_freq[i], &trig[half + i], &trig[i]);
     float ss = 0.f;
     for (int c = threadIdx.x; c < rank; c += blockDim.x) ss += raw[c] * raw[c];
-    ss = block_sum(ss, red);
-    const float r = 1.f / sqrtf(ss / (float)rank + eps);
-    const int pos = positions[t];
-    const int page = page_table[(size_t)seq_rows[t] * max_pages + pos / kKvTile];
-    const size_t at = ((size_t)page * kKvTile + pos % kKvTile) * rank;
+    ss = block_sum(ss, red);                               // its barriers also publish trig
+    const float r = 1.f / sqrtf(ss / (float)rank + a.eps);
+    const int page = a.page_table[(size_t)a.seq_rows[t] * a.max_pages + pos / kKvTile];
+    const size_t at = (size_t)page * kKvTile + pos % kKvTile;
+    float* c32 = a.cache ? a.cache + at * (rank + rot) : nullptr;
+    __nv_bfloat16* c16 = a.cache16 ? (__nv_bfloat16*)a.cache16 + at * row16 : nullptr;
     for (int c = threadIdx.x; c < rank; c += blockDim.x) {
-        const float v = raw[c] * r * w[c];
-        cache[at + c] = v;
-        if (cache16) cache16[at + c] = __float2bfloat16_rn(v);      // the tensor-core attention's copy
+        const float v = raw[c] * r * a.norm_w[c];
+        if (c32) c32[c] = v;
+        if (c16) c16[c] = __float2bfloat16_rn(v);
+    }
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        const float u = raw[rank + i], v = raw[rank + half + i], cs = trig[i], sn = trig[half + i];
+        const float x = u * cs - v * sn, y = v * cs + u * sn;
+        if (c32) { c32[rank + i] = x; c32[rank + half + i] = y; }
+        if (c16) { c16[rot_at16 + i] = __float2bfloat16_rn(x); c16[rot_at16 + half + i] = __float2bfloat16_rn(y); }
+    }
+    const int hd = a.dim + rot, kd = rank + rot;
+    for (int j = threadIdx.x; j < a.H * half; j += blockDim.x) {
+        const int h = j / half, i = j % half;
+        const float* q = pr + a.o_q + h * hd + a.dim;
+        const float u = q[i], v = q[half + i], cs = trig[i], sn = trig[half + i];
+        float* dst = a.qlat + ((size_t)t * a.H + h) * kd + rank;
+        dst[i] = u * cs - v * sn;
+        dst[half + i] = v * cs + u * sn;
     }
 }
 
@@ -504,43 +525,55 @@ latent_write_kernel(const float* __restrict__ proj, int ldp, int o_dkv, const fl
 // With n_split == 1 the warp finishes its (token, head): divides by the softmax sum and scales by the head's output gate
 // sigmoid(gate logit) — the value expansion that follows is linear, so gating before it is the same.  With n_split > 1
 // (few tokens: decode) it covers the s-th share of the keys and leaves (max, sum, unnormalised result) for the merge.
+// The softmax sum of a row whose maximum is m, with the sink's term, and the factor that finishes the row's result.
+__device__ __forceinline__ float latent_finish(float m, float l, const LatentArgs& a, int t, int h) {
+    float g = 1.f;
+    if (a.sink) {
+        // relative to the larger of m and the sink, so that neither exponential overflows
+        const float s = a.sink[h], top = fmaxf(m, s);
+        const float f = expf(m - top);
+        g = f;
+        l = l * f + expf(s - top);
+    }
+    if (a.o_gate >= 0) g *= sigmoid_exact(a.proj[(size_t)t * a.ldp + a.o_gate + h]);
+    return g / l;
+}
+
 template <int NR, int KB>
-__global__ void __launch_bounds__(128)
-latent_attn_kernel(const float* __restrict__ qlat, const float* __restrict__ cache, const float* __restrict__ proj, int ldp,
-                   int o_gate, float* __restrict__ out, float* __restrict__ part, const int* __restrict__ positions,
-                   const int* __restrict__ seq_rows, const int* __restrict__ page_table, int max_pages, int H, int rank,
-                   float scale, int n_pairs, int n_split) {
+__global__ void __launch_bounds__(128) latent_attn_kernel(LatentArgs a, int n_pairs, int n_split) {
     const int pair = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     const int split = blockIdx.y;
     if (pair >= n_pairs) return;
-    const int t = pair / H, h = pair % H;
-    const float* q = qlat + ((size_t)t * H + h) * rank;
+    const int rank = a.rank, kd = a.rank + a.rot;
+    const int t = pair / a.H, h = pair % a.H;
+    const float* cache = a.cache;
+    const float* q = a.qlat + (size_t)pair * kd;
     float qr[NR], acc[NR];
 #pragma unroll
     for (int i = 0; i < NR; ++i) {
         const int c = lane + 32 * i;
-        qr[i] = c < rank ? q[c] * scale : 0.f;
+        qr[i] = c < kd ? q[c] * a.scale : 0.f;
         acc[i] = 0.f;
     }
-    const int n_keys = positions[t] + 1;
+    const int n_keys = a.positions[t] + 1;
     int j_lo = 0, j_hi = n_keys;
     if (n_split > 1) {          // shares of whole pages
         const int share = ((n_keys + n_split - 1) / n_split + kKvTile - 1) / kKvTile * kKvTile;
         j_lo = min(split * share, n_keys);
         j_hi = min(j_lo + share, n_keys);
     }
-    const int* pt = page_table + (size_t)seq_rows[t] * max_pages;
+    const int* pt = a.page_table + (size_t)a.seq_rows[t] * a.max_pages;
     float m = -INFINITY, l = 0.f;
     for (int j0 = j_lo; j0 < j_hi; j0 += KB) {
         float cv[KB][NR], sc[KB];
 #pragma unroll
         for (int b = 0; b < KB; ++b) {
             const int j = min(j0 + b, j_hi - 1);
-            const float* c = cache + ((size_t)pt[j / kKvTile] * kKvTile + j % kKvTile) * rank;
+            const float* c = cache + ((size_t)pt[j / kKvTile] * kKvTile + j % kKvTile) * kd;
 #pragma unroll
             for (int i = 0; i < NR; ++i) {
                 const int cc = lane + 32 * i;
-                cv[b][i] = cc < rank ? c[cc] : 0.f;
+                cv[b][i] = cc < kd ? c[cc] : 0.f;
             }
         }
 #pragma unroll
@@ -574,7 +607,7 @@ latent_attn_kernel(const float* __restrict__ qlat, const float* __restrict__ cac
         m = mn;
     }
     if (n_split > 1) {
-        float* p = part + ((size_t)pair * n_split + split) * (rank + 2);
+        float* p = a.part + ((size_t)pair * n_split + split) * (rank + 2);
         if (lane == 0) { p[0] = m; p[1] = l; }
 #pragma unroll
         for (int i = 0; i < NR; ++i) {
@@ -583,8 +616,8 @@ latent_attn_kernel(const float* __restrict__ qlat, const float* __restrict__ cac
         }
         return;
     }
-    const float g = sigmoid_exact(proj[(size_t)t * ldp + o_gate + h]) / l;
-    float* o = out + ((size_t)t * H + h) * rank;
+    const float g = latent_finish(m, l, a, t, h);
+    float* o = a.out + (size_t)pair * rank;
 #pragma unroll
     for (int i = 0; i < NR; ++i) {
         const int c = lane + 32 * i;
@@ -593,12 +626,11 @@ latent_attn_kernel(const float* __restrict__ qlat, const float* __restrict__ cac
 }
 
 // The shares of one (token, head) put together: one warp each.
-__global__ void __launch_bounds__(128)
-latent_merge_kernel(const float* __restrict__ part, const float* __restrict__ proj, int ldp, int o_gate, float* __restrict__ out,
-                    int H, int rank, int n_pairs, int n_split) {
+__global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, int n_pairs, int n_split) {
     const int pair = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (pair >= n_pairs) return;
-    const float* p = part + (size_t)pair * n_split * (rank + 2);
+    const int rank = a.rank;
+    const float* p = a.part + (size_t)pair * n_split * (rank + 2);
     float m = -INFINITY;
     for (int s = 0; s < n_split; ++s) m = fmaxf(m, p[(size_t)s * (rank + 2)]);
     float l = 0.f;
@@ -606,80 +638,80 @@ latent_merge_kernel(const float* __restrict__ part, const float* __restrict__ pr
         const float ms = p[(size_t)s * (rank + 2)];
         if (ms > -INFINITY) l += p[(size_t)s * (rank + 2) + 1] * expf(ms - m);
     }
-    const int t = pair / H, h = pair % H;
-    const float g = sigmoid_exact(proj[(size_t)t * ldp + o_gate + h]) / l;
+    const float g = latent_finish(m, l, a, pair / a.H, pair % a.H);
     for (int c = lane; c < rank; c += 32) {
-        float a = 0.f;
+        float v = 0.f;
         for (int s = 0; s < n_split; ++s) {
             const float ms = p[(size_t)s * (rank + 2)];
-            if (ms > -INFINITY) a = fmaf(p[(size_t)s * (rank + 2) + 2 + c], expf(ms - m), a);
+            if (ms > -INFINITY) v = fmaf(p[(size_t)s * (rank + 2) + 2 + c], expf(ms - m), v);
         }
-        out[(size_t)pair * rank + c] = a * g;
+        a.out[(size_t)pair * rank + c] = v * g;
     }
 }
 
-int launch_latent_write(const float* proj, int ldp, int o_dkv, const float* w, float* cache, void* cache16, const int* positions,
-                        const int* seq_rows, const int* page_table, int max_pages, int rank, float eps, int T,
-                        cudaStream_t stream) {
-    latent_write_kernel<<<T, 128, 0, stream>>>(proj, ldp, o_dkv, w, cache, (__nv_bfloat16*)cache16, positions, seq_rows, page_table,
-                                               max_pages, rank, eps);
+int launch_latent_prep(const LatentArgs& a, int T, cudaStream_t stream) {
+    FT_REQUIRE(a.proj && a.norm_w && (a.cache || a.cache16) && (a.rot == 0 || (a.rot_freq && a.qlat && a.rot % 2 == 0)),
+               "latent prep: missing operands");
+    latent_prep_kernel<<<T, 128, (size_t)a.rot * 4, stream>>>(a, latent_row16(a.rank, a.rot), (a.rank + 31) / 32 * 32);
     FT_CHECK_CUDA(cudaGetLastError());
     return 0;
 }
 
 // The serving form of the same attention on the tensor cores (mma.sync m16n8k16, bf16 operands, fp32 accumulation and
-// softmax): one CTA per (token, key share, group of 16 heads).  The 16 heads are the M rows of every product, so all rows
+// softmax): one CTA per (token, key share, group of 16 heads and, for latents beyond 256, group of value columns).  The 16 heads are the M rows of every product, so all rows
 // of a tile see the same keys and one mask.  Each of the four warps takes every fourth 16-key tile of the share: the tile
 // (16 latents from the bf16 copy of the cache) is copied into the warp's own double buffer with cp.async one tile ahead,
 // S = Q C^T (ldmatrix fragments of Q and of the tile), online softmax in registers, O += P C with the SAME tile read
 // through ldmatrix.trans — keys and values are one array.  The warps' (max, sum, O) are merged through shared memory.
-// rank = 32 * RK <= 256 (O is rank / 8 accumulator tiles per thread).
+// Both parts of a row are padded with zeros to multiples of 32 columns: kc 32-column pieces per row, vc of them the latent.  A
+// CTA sums VC <= 8 of those (O is 4 * VC accumulator tiles per thread).
 __device__ __forceinline__ void cp_async16(void* dst_smem, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst_smem)), "l"(src) : "memory");
 }
 __device__ __forceinline__ void cp_async_wait_1() { asm volatile("cp.async.wait_group 1;" ::: "memory"); }
 
-template <int RK>
+template <int VC>
 __global__ void __launch_bounds__(128)
-latent_attn_mma_kernel(const float* __restrict__ qlat, const __nv_bfloat16* __restrict__ cache16, const float* __restrict__ proj,
-                       int ldp, int o_gate, float* __restrict__ out, float* __restrict__ part, const int* __restrict__ positions,
-                       const int* __restrict__ seq_rows, const int* __restrict__ page_table, int max_pages, int H, float scale,
-                       int n_split) {
-    constexpr int RANK = 32 * RK, RS = RANK * 2 + 16;      // row stride in bytes: 16 bytes of padding keep ldmatrix conflict-free
-    constexpr int TILE = 16 * RS;
+latent_attn_mma_kernel(LatentArgs a, int kc, int vc, int head_groups, int n_split) {
+    const int row = 32 * kc, RS = row * 2 + 16;            // row stride in bytes: 16 bytes of padding keep ldmatrix conflict-free
+    const int TILE = 16 * RS;
     extern __shared__ __align__(16) uint8_t lat_smem[];
     uint8_t* Qs = lat_smem;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     uint8_t* kbuf = lat_smem + TILE + (size_t)warp * 2 * TILE;
-    const int t = blockIdx.x, split = blockIdx.y, h0 = blockIdx.z * 16;
-    for (int idx = threadIdx.x; idx < 16 * RANK; idx += 128) {
-        const int r = idx / RANK, c = idx % RANK;
-        const float v = h0 + r < H ? qlat[((size_t)t * H + h0 + r) * RANK + c] * scale : 0.f;
+    const int t = blockIdx.x, split = blockIdx.y, h0 = (blockIdx.z % head_groups) * 16;
+    const int v_first = (blockIdx.z / head_groups) * VC;   // first 32-column piece of the values this CTA sums
+    const int H = a.H, rank = a.rank, kd = a.rank + a.rot, rot_at = 32 * vc;
+    const __nv_bfloat16* cache16 = (const __nv_bfloat16*)a.cache16;
+    for (int idx = threadIdx.x; idx < 16 * row; idx += 128) {
+        const int r = idx / row, c = idx % row;
+        const int src = c < rot_at ? (c < rank ? c : -1) : (c - rot_at < a.rot ? rank + c - rot_at : -1);
+        const float v = h0 + r < H && src >= 0 ? a.qlat[((size_t)t * H + h0 + r) * kd + src] * a.scale : 0.f;
         *reinterpret_cast<__nv_bfloat16*>(Qs + r * RS + c * 2) = __float2bfloat16_rn(v);
     }
     __syncthreads();
-    const int n_keys = positions[t] + 1;
+    const int n_keys = a.positions[t] + 1;
     int j_lo = 0, j_hi = n_keys;
     if (n_split > 1) {
         const int share = ((n_keys + n_split - 1) / n_split + kKvTile - 1) / kKvTile * kKvTile;
         j_lo = min(split * share, n_keys);
         j_hi = min(j_lo + share, n_keys);
     }
-    const int* pt = page_table + (size_t)seq_rows[t] * max_pages;
+    const int* pt = a.page_table + (size_t)a.seq_rows[t] * a.max_pages;
     const int n_tiles = (j_hi - j_lo + 15) / 16;
     auto stage = [&](int tile, int buf) {
         const int key0 = j_lo + tile * 16;
         uint8_t* dst = kbuf + buf * TILE;
-        for (int i = lane; i < 16 * 4 * RK; i += 32) {          // 16 rows of 4 * RK 16-byte pieces
-            const int r = i / (4 * RK), ch = i % (4 * RK);
+        for (int i = lane; i < 16 * 4 * kc; i += 32) {          // 16 rows of 4 * kc 16-byte pieces
+            const int r = i / (4 * kc), ch = i % (4 * kc);
             const int j = min(key0 + r, j_hi - 1);
-            cp_async16(dst + r * RS + ch * 16, cache16 + ((size_t)pt[j / kKvTile] * kKvTile + j % kKvTile) * RANK + ch * 8);
+            cp_async16(dst + r * RS + ch * 16, cache16 + ((size_t)pt[j / kKvTile] * kKvTile + j % kKvTile) * row + ch * 8);
         }
         cp_async_commit();
     };
-    float o[4 * RK][4];
+    float o[4 * VC][4];
 #pragma unroll
-    for (int nt = 0; nt < 4 * RK; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
+    for (int nt = 0; nt < 4 * VC; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;      // rows g and g + 8
     const int g = lane >> 2, tq = lane & 3;
     const uint32_t q_addr = smem_u32(Qs) + ((lane & 7) + ((lane >> 3) & 1) * 8) * RS + (lane >> 4) * 16;
@@ -693,8 +725,8 @@ latent_attn_mma_kernel(const float* __restrict__ qlat, const __nv_bfloat16* __re
         float sc[2][4];
 #pragma unroll
         for (int j = 0; j < 2; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
-#pragma unroll
-        for (int kp = 0; kp < RK; ++kp) {                        // 32 latent channels per round
+#pragma unroll 2
+        for (int kp = 0; kp < kc; ++kp) {                        // 32 columns per round
             uint32_t a0[4], a1[4];
             ldmatrix_x4(q_addr + (kp * 4) * 16, a0[0], a0[1], a0[2], a0[3]);
             ldmatrix_x4(q_addr + (kp * 4 + 2) * 16, a1[0], a1[1], a1[2], a1[3]);
@@ -740,9 +772,10 @@ latent_attn_mma_kernel(const float* __restrict__ qlat, const __nv_bfloat16* __re
         const uint32_t pa2 = pack_bf16(sc[1][0], sc[1][1]), pa3 = pack_bf16(sc[1][2], sc[1][3]);
         const int vrow = ((lane >> 3) & 1) * 8 + (lane & 7);
 #pragma unroll
-        for (int np = 0; np < 2 * RK; ++np) {                    // 16 latent channels per round
+        for (int np = 0; np < 2 * VC; ++np) {                    // 16 latent columns per round
+            if (v_first + (np >> 1) >= vc) break;                // the last group of columns may be a partial one
             uint32_t b0, b1, b2, b3;
-            ldmatrix_x4_trans(kb + vrow * RS + (2 * np + (lane >> 4)) * 16, b0, b1, b2, b3);
+            ldmatrix_x4_trans(kb + vrow * RS + (4 * v_first + 2 * np + (lane >> 4)) * 16, b0, b1, b2, b3);
             o[2 * np][0] *= alpha_a; o[2 * np][1] *= alpha_a; o[2 * np][2] *= alpha_b; o[2 * np][3] *= alpha_b;
             o[2 * np + 1][0] *= alpha_a; o[2 * np + 1][1] *= alpha_a; o[2 * np + 1][2] *= alpha_b; o[2 * np + 1][3] *= alpha_b;
             mma_bf16_16816(o[2 * np], pa0, pa1, pa2, pa3, b0, b1);
@@ -755,43 +788,43 @@ latent_attn_mma_kernel(const float* __restrict__ qlat, const __nv_bfloat16* __re
     l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 1);
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
-    constexpr int REC = RANK + 2;
+    constexpr int COLS = 32 * VC, REC = COLS + 2;
     float* rec = reinterpret_cast<float*>(kbuf);
 #pragma unroll
-    for (int nt = 0; nt < 4 * RK; ++nt) {
+    for (int nt = 0; nt < 4 * VC; ++nt) {
         rec[g * REC + nt * 8 + 2 * tq] = o[nt][0];
         rec[g * REC + nt * 8 + 2 * tq + 1] = o[nt][1];
         rec[(g + 8) * REC + nt * 8 + 2 * tq] = o[nt][2];
         rec[(g + 8) * REC + nt * 8 + 2 * tq + 1] = o[nt][3];
     }
     if (tq == 0) {
-        rec[g * REC + RANK] = m_a; rec[g * REC + RANK + 1] = l_a;
-        rec[(g + 8) * REC + RANK] = m_b; rec[(g + 8) * REC + RANK + 1] = l_b;
+        rec[g * REC + COLS] = m_a; rec[g * REC + COLS + 1] = l_a;
+        rec[(g + 8) * REC + COLS] = m_b; rec[(g + 8) * REC + COLS + 1] = l_b;
     }
     __syncthreads();
-    for (int idx = threadIdx.x; idx < 16 * RANK; idx += 128) {
-        const int r = idx / RANK, c = idx % RANK;
-        if (h0 + r >= H) continue;
+    for (int idx = threadIdx.x; idx < 16 * COLS; idx += 128) {
+        const int r = idx / COLS, c = idx % COLS, col = 32 * v_first + c;
+        if (h0 + r >= H || col >= rank) continue;
         float m = -INFINITY;
 #pragma unroll
-        for (int w = 0; w < 4; ++w) m = fmaxf(m, reinterpret_cast<const float*>(lat_smem + TILE + (size_t)w * 2 * TILE)[r * REC + RANK]);
-        float l = 0.f, a = 0.f;
+        for (int w = 0; w < 4; ++w) m = fmaxf(m, reinterpret_cast<const float*>(lat_smem + TILE + (size_t)w * 2 * TILE)[r * REC + COLS]);
+        float l = 0.f, v = 0.f;
 #pragma unroll
         for (int w = 0; w < 4; ++w) {
             const float* rw = reinterpret_cast<const float*>(lat_smem + TILE + (size_t)w * 2 * TILE) + r * REC;
-            if (rw[RANK] > -INFINITY) {
-                const float f = expf(rw[RANK] - m);
-                l = fmaf(rw[RANK + 1], f, l);
-                a = fmaf(rw[c], f, a);
+            if (rw[COLS] > -INFINITY) {
+                const float f = expf(rw[COLS] - m);
+                l = fmaf(rw[COLS + 1], f, l);
+                v = fmaf(rw[c], f, v);
             }
         }
         const size_t pair = (size_t)t * H + h0 + r;
         if (n_split > 1) {
-            float* p = part + (pair * n_split + split) * REC;
-            p[2 + c] = a;
-            if (c == 0) { p[0] = m; p[1] = l; }
+            float* p = a.part + (pair * n_split + split) * (rank + 2);
+            p[2 + col] = v;
+            if (col == 0) { p[0] = m; p[1] = l; }
         } else {
-            out[pair * RANK + c] = a / l * sigmoid_exact(proj[(size_t)t * ldp + o_gate + h0 + r]);
+            a.out[pair * rank + col] = v * latent_finish(m, l, a, t, h0 + r);
         }
     }
 }
@@ -802,55 +835,51 @@ int latent_attn_splits(int T, int H) {
     return std::max(1, std::min(kLatentMaxSplits, kLatentSplitPairs / std::max(pairs, 1)));
 }
 
-bool latent_attn_mma_ok(int rank) { return rank % 32 == 0 && rank >= 32 && rank <= 256; }
+int latent_row16(int rank, int rot) { return (rank + 31) / 32 * 32 + (rot + 31) / 32 * 32; }
+// the query tile and the four warps' double-buffered key tiles, 16 rows each
+static size_t latent_mma_smem(int rank, int rot) { return (size_t)9 * 16 * (latent_row16(rank, rot) * 2 + 16); }
+bool latent_attn_mma_ok(int rank, int rot) { return rank >= 1 && latent_mma_smem(rank, rot) <= 224 * 1024; }
 
-int launch_latent_attn(const float* qlat, const float* cache, const void* cache16, const float* proj, int ldp, int o_gate,
-                       float* out, float* part, const int* positions, const int* seq_rows, const int* page_table, int max_pages,
-                       int H, int rank, float scale, int T, cudaStream_t stream) {
-    const int n_pairs = T * H;
-    const int n_split = part ? latent_attn_splits(T, H) : 1;
-    if (cache16 && latent_attn_mma_ok(rank)) {
-        const dim3 grid(T, n_split, (H + 15) / 16);
-        const size_t smem = (size_t)9 * 16 * (rank * 2 + 16);
-#define FT_LATM(RK_)                                                                                                        \
-    case RK_: {                                                                                                             \
+int launch_latent_attn(const LatentArgs& a, int T, cudaStream_t stream) {
+    const int n_pairs = T * a.H;
+    const int n_split = a.part ? latent_attn_splits(T, a.H) : 1;
+    if (a.cache16 && latent_attn_mma_ok(a.rank, a.rot)) {
+        const int vc = (a.rank + 31) / 32, kc = latent_row16(a.rank, a.rot) / 32;
+        const int groups = (vc + 7) / 8, per = (vc + groups - 1) / groups, hg = (a.H + 15) / 16;
+        const dim3 grid(T, n_split, hg * groups);
+        const size_t smem = latent_mma_smem(a.rank, a.rot);
+#define FT_LATM(VC_)                                                                                                        \
+    case VC_: {                                                                                                             \
         static PerDeviceFlag attr;                                                                                          \
         if (!attr.done()) {                                                                                                 \
-            FT_CHECK_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<RK_>, cudaFuncAttributeMaxDynamicSharedMemorySize,    \
-                                               9 * 16 * (RK_ * 64 + 16)));                                                  \
+            FT_CHECK_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<VC_>, cudaFuncAttributeMaxDynamicSharedMemorySize,    \
+                                               224 * 1024));                                                                \
             attr.mark();                                                                                                    \
         }                                                                                                                   \
-        latent_attn_mma_kernel<RK_><<<grid, 128, smem, stream>>>(qlat, (const __nv_bfloat16*)cache16, proj, ldp, o_gate, out, \
-                                                                 part, positions, seq_rows, page_table, max_pages, H, scale, \
-                                                                 n_split);                                                  \
+        latent_attn_mma_kernel<VC_><<<grid, 128, smem, stream>>>(a, kc, vc, hg, n_split);                                   \
         break;                                                                                                              \
     }
-        switch (rank / 32) {
+        switch (per) {
             FT_LATM(1) FT_LATM(2) FT_LATM(3) FT_LATM(4) FT_LATM(5) FT_LATM(6) FT_LATM(7) FT_LATM(8)
             default: break;
         }
 #undef FT_LATM
-        FT_CHECK_CUDA(cudaGetLastError());
-        if (n_split > 1) {
-            latent_merge_kernel<<<(n_pairs + 3) / 4, 128, 0, stream>>>(part, proj, ldp, o_gate, out, H, rank, n_pairs, n_split);
-            FT_CHECK_CUDA(cudaGetLastError());
-        }
-        return 0;
-    }
-    const dim3 grid((n_pairs + 3) / 4, n_split);
-#define FT_LAT(NR_, KB_)                                                                                                   \
-    latent_attn_kernel<NR_, KB_><<<grid, 128, 0, stream>>>(qlat, cache, proj, ldp, o_gate, out, part, positions, seq_rows, \
-                                                           page_table, max_pages, H, rank, scale, n_pairs, n_split)
-    if (rank <= 32) FT_LAT(1, 8);
-    else if (rank <= 64) FT_LAT(2, 8);
-    else if (rank <= 128) FT_LAT(4, 8);
-    else if (rank <= 256) FT_LAT(8, 4);
-    else if (rank <= 512) FT_LAT(16, 4);
-    else { FT_REQUIRE(rank <= 1024, "latent attention: latent size %d is beyond 1024", rank); FT_LAT(32, 2); }
+    } else {
+        FT_REQUIRE(a.cache, "latent attention: no fp32 cache");
+        const int kd = a.rank + a.rot;
+        const dim3 grid((n_pairs + 3) / 4, n_split);
+#define FT_LAT(NR_, KB_) latent_attn_kernel<NR_, KB_><<<grid, 128, 0, stream>>>(a, n_pairs, n_split)
+        if (kd <= 32) FT_LAT(1, 8);
+        else if (kd <= 64) FT_LAT(2, 8);
+        else if (kd <= 128) FT_LAT(4, 8);
+        else if (kd <= 256) FT_LAT(8, 4);
+        else if (kd <= 512) FT_LAT(16, 4);
+        else { FT_REQUIRE(kd <= 1024, "latent attention: a cache row of %d columns is beyond 1024", kd); FT_LAT(32, 2); }
 #undef FT_LAT
+    }
     FT_CHECK_CUDA(cudaGetLastError());
     if (n_split > 1) {
-        latent_merge_kernel<<<(n_pairs + 3) / 4, 128, 0, stream>>>(part, proj, ldp, o_gate, out, H, rank, n_pairs, n_split);
+        latent_merge_kernel<<<(n_pairs + 3) / 4, 128, 0, stream>>>(a, n_pairs, n_split);
         FT_CHECK_CUDA(cudaGetLastError());
     }
     return 0;
@@ -1105,12 +1134,12 @@ int launch_delta(const DeltaArgs& a, const float* gate, const float* out_norm, f
 }
 
 // ------------------------------------------------------------------ router
-// One warp per token: s = softmax(z) over all E experts (or sigmoid(z) of each); a group's score is its largest s; only
+// One warp per token: z = logits (+ bias); s = softmax(z) over all E experts (or sigmoid(z) of each); a group's score is its largest s; only
 // experts of the `keep` best groups can be chosen; the `top` largest s among them, lowest index first on a tie; weights = s
 // as it is, or (normalise) divided by the sum of the chosen ones (+ 1e-20); then times `scale`.
 __global__ void __launch_bounds__(128)
 route_kernel(const float* __restrict__ proj, int ldp, int o_router, int E, int top, int groups, int keep, int* __restrict__ ids,
-             float* __restrict__ wts, int T, int sigmoid_scores, int normalise, float scale) {
+             float* __restrict__ wts, int T, int sigmoid_scores, int normalise, float scale, const float* __restrict__ bias) {
     extern __shared__ float sh[];
     const int wid = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * (blockDim.x >> 5) + wid;
@@ -1119,13 +1148,16 @@ route_kernel(const float* __restrict__ proj, int ldp, int o_router, int E, int t
     float* gs = s + E;
     const float* z = proj + (size_t)t * ldp + o_router;
     if (sigmoid_scores) {
-        for (int e = lane; e < E; e += 32) s[e] = sigmoid_exact(z[e]);
+        for (int e = lane; e < E; e += 32) s[e] = sigmoid_exact(z[e] + (bias ? bias[e] : 0.f));
     } else {
         float m = -INFINITY;
-        for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
+        for (int e = lane; e < E; e += 32) {
+            s[e] = z[e] + (bias ? bias[e] : 0.f);
+            m = fmaxf(m, s[e]);
+        }
         m = warp_max(m);
         float sum = 0.f;
-        for (int e = lane; e < E; e += 32) { const float v = expf(z[e] - m); s[e] = v; sum += v; }
+        for (int e = lane; e < E; e += 32) { const float v = expf(s[e] - m); s[e] = v; sum += v; }
         sum = warp_sum(sum);
         __syncwarp();
         for (int e = lane; e < E; e += 32) s[e] = s[e] / sum;
@@ -1213,13 +1245,13 @@ route_sort_kernel(const int* __restrict__ ids, int n_pairs, int top, int E, int*
 
 int launch_route(const float* proj, int ldp, int o_router, int E, int top, int groups, int keep, int* ids, float* wts,
                  int* seg, int* slot_token, int* slot_pos, int T, cudaStream_t stream, int route_kind, int normalise,
-                 float scale) {
+                 float scale, const float* bias) {
     FT_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && top >= 1 && top <= (E / groups) * keep,
                "router: %d experts, %d groups, keep %d, top %d do not fit together", E, groups, keep, top);
     const size_t smem = (size_t)4 * (E + groups) * 4;
     FT_REQUIRE(smem <= 48 * 1024 && (size_t)(E + 1) * 4 <= 48 * 1024, "router: %d experts are too many", E);
     route_kernel<<<(T + 3) / 4, 128, smem, stream>>>(proj, ldp, o_router, E, top, groups, keep, ids, wts, T,
-                                                     route_kind == FT_ROUTE_SIGMOID, normalise, scale > 0.f ? scale : 1.f);
+                                                     route_kind == FT_ROUTE_SIGMOID, normalise, scale > 0.f ? scale : 1.f, bias);
     FT_CHECK_CUDA(cudaGetLastError());
     route_sort_kernel<<<1, 1024, (size_t)(E + 1) * 4, stream>>>(ids, T * top, top, E, seg, slot_token, slot_pos);
     FT_CHECK_CUDA(cudaGetLastError());

@@ -116,7 +116,7 @@ class Engine:
         pages_per_ctx = -(-lim.max_context // 64)
         num_pages = lim.num_pages or int(lim.max_batch * pages_per_ctx * 1.25) + 8
         cfg = N.EngineConfig()
-        cfg.hidden, cfg.layers, cfg.vocab, cfg.rms_eps = spec.width, len(spec.layers), spec.vocab, spec.eps
+        cfg.hidden, cfg.layers, cfg.vocab, cfg.rms_eps = spec.width, len(spec.runs()), spec.vocab, spec.eps
         cfg.max_batch, cfg.max_batched_tokens = lim.max_batch, max(lim.max_batched_tokens, lim.max_batch)
         cfg.num_pages, cfg.max_context = num_pages, lim.max_context
         cfg.max_sessions = lim.max_sessions or 4 * lim.max_batch
@@ -259,7 +259,7 @@ class Engine:
 
     def read_trail(self, rows: int) -> np.ndarray:
         """Residual stream after every layer of the most recent step: float32 [layers, rows, width]."""
-        out = np.empty((len(self.spec.layers), rows, self.spec.width), dtype=np.float32)
+        out = np.empty((len(self.spec.runs()), rows, self.spec.width), dtype=np.float32)
         N.check(self.lib.ft_engine_debug_read_trail(self._h, out.ctypes.data, rows), "ft_engine_debug_read_trail")
         return out
 

@@ -27,6 +27,12 @@ convolutions on q, k, v, one RMS norm over all heads, stretched rotary frequenci
 selective state-space scan, each side RMS-normed over the width — and a feed-forward that is a dense SwiGLU or a mixture of
 experts whose sigmoid scores multiply the experts' inputs.  Its logits come from the embedding table itself.
 
+The fifth design is Gedalix: pre-norm layers (RMS norms with a gain per coordinate, results scaled coordinate by coordinate and
+by one residual multiplier), latent attention without a query latent whose scores add a shared rotated key part, with a sink in
+the softmax and an element-wise output gate, a mixture of experts with biased softmax routing over the chosen logits plus a
+shared expert under a gate of its own, learned position vectors, and a run of layers that is repeated with the same weights: a
+pass takes the embedding output again and a vector of its own.  The engine sees the repeated layers as further layer RUNS.
+
 The reference names models by tag only and owns no model code (app/utils/config.py:86, docker-compose.vllm.yml:39); this
 module is the model side of what its engine container would load: config.json -> LayeredSpec, model.safetensors -> the
 tensors by their names in the file, pack() -> the device arrays and descriptors the native engine reads.
@@ -43,7 +49,7 @@ import torch
 
 MIXER_LATENT_ATTENTION, MIXER_CHANNEL_DELTA, MIXER_BRANCHES = 1, 2, 3
 FF_NONE, FF_MOE, FF_DENSE = 0, 1, 2
-LAYER_GATED, LAYER_SANDWICH, LAYER_POSTNORM, LAYER_HYPER = 0, 1, 2, 3
+LAYER_GATED, LAYER_SANDWICH, LAYER_POSTNORM, LAYER_HYPER, LAYER_PRENORM = 0, 1, 2, 3, 4
 ACT_SWIGLU, ACT_RELU2 = 0, 1
 ROUTE_SOFTMAX, ROUTE_SIGMOID = 0, 1
 BRANCH_WINDOW_ATTENTION, BRANCH_DECAY_ATTENTION, BRANCH_MATRIX_MEMORY, BRANCH_STATE_SPACE, BRANCH_LATENT_WINDOW = 1, 2, 3, 4, 5
@@ -117,11 +123,14 @@ class LayerSpec:
     groups: int = 1
     keep: int = 1
     # sandwich layers (Gedelorn)
-    form: str = "gated"             # "gated" | "sandwich" | "postnorm" | "hyper"
+    form: str = "gated"             # "gated" | "sandwich" | "postnorm" | "hyper" | "prenorm"
     branches: Tuple[BranchSpec, ...] = ()
     ff_kind: str = ""               # sandwich: "" (none) | "dense" | "moe"
     route_scale: float = 1.0
     shared_ff: int = 0
+    # latent attention of pre-norm layers (Gedalix): rotated size (query and shared key part) and its base
+    rot_dims: int = 0
+    rot_base: float = 10000.0
 
 
 @dataclass(frozen=True)
@@ -136,6 +145,21 @@ class LayeredSpec:
     embed_scale: float = 1.0        # post-norm and hyper-connected models
     canon_taps: int = 0             # post-norm models: taps of the input convolutions
     streams: int = 0                # hyper-connected models: copies of the stream (0: one, and no mixing tensors)
+    # pre-norm models
+    residual_mult: float = 1.0
+    max_positions: int = 0          # rows of the position table
+    loop: Tuple[int, int, int] = () # (start, stop, times): layers start .. stop - 1 run `times` times in a row
+
+    def runs(self) -> List[Tuple[int, Optional[int]]]:
+        """(layer, pass) in the order the layers run; the pass number stands only at the first layer of a pass over the loop."""
+        n = len(self.layers)
+        if not self.loop:
+            return [(i, None) for i in range(n)]
+        start, stop, times = self.loop
+        out: List[Tuple[int, Optional[int]]] = [(i, None) for i in range(start)]
+        for t in range(times):
+            out += [(i, t if i == start else None) for i in range(start, stop)]
+        return out + [(i, None) for i in range(stop, n)]
 
     # the attributes the serving code reads from any model spec
     @property
@@ -145,6 +169,13 @@ class LayeredSpec:
     def config(self) -> Dict:
         """The config.json of this spec."""
         out = []
+        if self.layers and self.layers[0].form == "prenorm":
+            cfg = {"architecture": self.architecture, "embedding": {"scale": self.embed_scale},
+                   "layers": [_prenorm_layer_config(l) for l in self.layers], "max_positions": self.max_positions,
+                   "norm": {"eps": self.eps}, "residual_mult": self.residual_mult, "vocab": self.vocab, "width": self.width}
+            if self.loop:
+                cfg["loop"] = dict(zip(("start", "stop", "times"), self.loop))
+            return cfg
         if self.layers and self.layers[0].form == "hyper":
             cfg = {"architecture": self.architecture, "embedding": {"scale": self.embed_scale},
                    "layers": [_hyper_layer_config(l) for l in self.layers], "norm": {"eps": self.eps}, "vocab": self.vocab,
@@ -176,6 +207,46 @@ class LayeredSpec:
             cfg["canon"] = {"taps": self.canon_taps}
             cfg["embedding"] = {"scale": self.embed_scale}
         return cfg
+
+
+def _prenorm_layer_config(l: LayerSpec) -> Dict:
+    mixer = {"dim": l.dim, "heads": l.heads, "kv_rank": l.kv_rank, "rot_dim": l.rot_dims, "scale": l.scale, "vdim": l.vdim}
+    if l.rot_dims:
+        mixer["rot"] = {"base": l.rot_base, "dims": l.rot_dims}
+    mlp = None
+    if l.ff_kind:
+        mlp = {"expert": {"ff": l.ff}, "kind": "moe", "router": {"experts": l.experts, "top": l.top}}
+        if l.shared_ff:
+            mlp["shared"] = {"ff": l.shared_ff}
+    return {"mixer": mixer, "mlp": mlp, "type": l.mixer}
+
+
+def _prenorm_layer_from_config(i: int, l: Dict) -> LayerSpec:
+    kind, m, mlp = l["type"], l["mixer"], l.get("mlp")
+    if kind != "latent_attention":
+        raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+    rot = m.get("rot") or {}
+    rd = int(m.get("rot_dim", rot.get("dims", 0)))
+    if rd % 2 or (rd and int(rot.get("dims", rd)) != rd):
+        raise ValueError(f"layer {i}: the rotated part has {rd} coordinates, the rotation covers {rot.get('dims')}")
+    kw = dict(mixer=kind, form="prenorm", heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), kv_rank=int(m["kv_rank"]),
+              scale=float(m["scale"]), rot_dims=rd, rot_base=float(rot.get("base", 10000.0)))
+    if mlp:
+        if mlp.get("kind", "moe") != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+        kw.update(ff_kind="moe", ff=int(mlp["expert"]["ff"]), experts=int(mlp["router"]["experts"]), top=int(mlp["router"]["top"]),
+                  shared_ff=int((mlp.get("shared") or {}).get("ff", 0)))
+    return LayerSpec(**kw)
+
+
+def _loop_from_config(cfg: Dict) -> Tuple[int, ...]:
+    loop = cfg.get("loop")
+    if not loop:
+        return ()
+    start, stop, times = (int(loop[k]) for k in ("start", "stop", "times"))
+    if not (0 <= start < stop <= len(cfg["layers"]) and times >= 1):
+        raise ValueError(f"loop {loop} does not fit {len(cfg['layers'])} layers")
+    return (start, stop, times)
 
 
 def _hyper_attention_config(b: BranchSpec) -> Dict:
@@ -413,8 +484,12 @@ def spec_from_config(cfg: Dict, shapes: Optional[Dict[str, Tuple[int, ...]]] = N
     layers = []
     postnorm = cfg.get("architecture") == "Vonedra"
     hyper = cfg.get("architecture") == "Lotinex"
+    prenorm = cfg.get("architecture") == "Gedalix"
     for i, l in enumerate(cfg["layers"]):
         kind, m = l["type"], l["mixer"]
+        if prenorm:
+            layers.append(_prenorm_layer_from_config(i, l))
+            continue
         if hyper:
             layers.append(_hyper_layer_from_config(i, l))
             continue
@@ -448,13 +523,23 @@ def spec_from_config(cfg: Dict, shapes: Optional[Dict[str, Tuple[int, ...]]] = N
     return LayeredSpec(name=name, architecture=str(cfg.get("architecture", "Gitozen")), width=int(cfg["width"]),
                        vocab=int(cfg["vocab"]), eps=float(cfg["norm"]["eps"]), logit_softcap=float(cap) if cap else 0.0,
                        layers=tuple(layers), embed_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)),
-                       canon_taps=int((cfg.get("canon") or {}).get("taps", 0)), streams=int(cfg.get("streams") or 0) if hyper else 0)
+                       canon_taps=int((cfg.get("canon") or {}).get("taps", 0)), streams=int(cfg.get("streams") or 0) if hyper else 0,
+                       residual_mult=float(cfg.get("residual_mult", 1.0)), max_positions=int(cfg["max_positions"]) if prenorm else 0,
+                       loop=_loop_from_config(cfg) if prenorm else ())
 
 
 def tensor_shapes(spec: LayeredSpec) -> Dict[str, Tuple[int, ...]]:
     """Names and shapes of a checkpoint of this spec."""
     W = spec.width
     out: Dict[str, Tuple[int, ...]] = {"embed": (spec.vocab, W)}
+    if spec.layers and spec.layers[0].form == "prenorm":
+        out["pos"] = (spec.max_positions, W)
+        if spec.loop:
+            out["loop.step"] = (spec.loop[2], W)
+        for i, l in enumerate(spec.layers):
+            out.update(_prenorm_shapes(f"l{i}.", l, W))
+        out.update({"final.norm": (W,), "head": (spec.vocab, W)})
+        return out
     if spec.layers and spec.layers[0].form == "hyper":
         for i, l in enumerate(spec.layers):
             out.update(_hyper_shapes(f"l{i}.", l, W, spec.streams))
@@ -489,6 +574,23 @@ def tensor_shapes(spec: LayeredSpec) -> Dict[str, Tuple[int, ...]]:
         out.update({p + "rg1": (W, W), p + "rg1.b": (W,)})
     out["final.norm"] = (W,) if spec.layers and spec.layers[-1].form in ("sandwich", "postnorm") else ()
     out["head"] = (spec.vocab, W)
+    return out
+
+
+def _prenorm_shapes(p: str, l: LayerSpec, W: int) -> Dict[str, Tuple[int, ...]]:
+    m, hv = p + "mix.", l.heads * l.vdim
+    out: Dict[str, Tuple[int, ...]] = {
+        p + "norm1": (W,), p + "ls1": (W,), m + "q": (l.heads * (l.dim + l.rot_dims), W), m + "dkv": (l.kv_rank + l.rot_dims, W),
+        m + "dkv.norm": (l.kv_rank,), m + "uk": (l.heads * l.dim, l.kv_rank), m + "uv": (hv, l.kv_rank), m + "sink": (l.heads,),
+        m + "g": (hv, W), m + "o": (W, hv)}
+    if l.ff_kind:
+        f = p + "mlp."
+        out.update({p + "norm2": (W,), p + "ls2": (W,), f + "router": (l.experts, W), f + "router.b": (l.experts,)})
+        for e in range(l.experts):
+            out.update({f"{f}e{e}.gate": (l.ff, W), f"{f}e{e}.up": (l.ff, W), f"{f}e{e}.down": (W, l.ff)})
+        if l.shared_ff:
+            out.update({f + "shared.gate": (l.shared_ff, W), f + "shared.up": (l.shared_ff, W), f + "shared.down": (W, l.shared_ff),
+                        f + "shared.sg": (1, W)})
     return out
 
 
@@ -602,6 +704,7 @@ def init_weights(spec: LayeredSpec, seed: int = 0, device: str = "cpu") -> Dict[
     sandwich = bool(spec.layers) and spec.layers[-1].form == "sandwich"
     postnorm = bool(spec.layers) and spec.layers[-1].form == "postnorm"
     hyper = bool(spec.layers) and spec.layers[-1].form == "hyper"
+    prenorm = bool(spec.layers) and spec.layers[-1].form == "prenorm"
     for name, shape in tensor_shapes(spec).items():
         leaf = name.split(".")[-1]
         part = name.split(".")[-2] if "." in name else ""
@@ -619,6 +722,10 @@ def init_weights(spec: LayeredSpec, seed: int = 0, device: str = "cpu") -> Dict[
             t = 1.0 + 0.1 * torch.randn(shape, generator=g)
         elif hyper and leaf == "D":
             t = 1.0 + 0.2 * torch.randn(shape, generator=g)
+        elif prenorm and (leaf in ("norm1", "norm2", "ls1", "ls2") or (leaf == "norm" and part in ("final", "dkv"))):
+            t = 1.0 + 0.2 * torch.randn(shape, generator=g)
+        elif prenorm and (name in ("pos", "loop.step") or leaf in ("sink", "b")):
+            t = 0.5 * torch.randn(shape, generator=g)
         elif postnorm and leaf in ("canon1", "canon2"):
             t = 0.3 * torch.randn(shape, generator=g)
         elif postnorm and leaf == "dwa":
@@ -739,6 +846,9 @@ class LayerDesc(C.Structure):
         ("canon_taps", C.c_int), ("canon1", C.c_void_p), ("canon2", C.c_void_p), ("depth_w", C.c_void_p), ("gate_act", C.c_int),
         ("norm_pre1_b", C.c_void_p), ("norm_pre2_b", C.c_void_p),
         ("hc_in", C.c_void_p * 2), ("hc_out", C.c_void_p * 2), ("hc_mix", C.c_void_p * 2), ("route_input", C.c_int),
+        ("res_gain", C.c_void_p * 2), ("re_embed", C.c_int), ("pre_add", C.c_void_p),
+        ("rot_dims", C.c_int), ("rot_freq", C.c_void_p), ("sink", C.c_void_p), ("gate_wide", C.c_int),
+        ("router_bias", C.c_void_p), ("shared_gate", C.c_int),
     ]
 
 
@@ -749,6 +859,7 @@ class LayeredModel(C.Structure):
         ("eps", C.c_float), ("logit_softcap", C.c_float), ("final_norm_gain", C.c_float),
         ("embed", C.c_void_p), ("head", C.c_void_p), ("layers", C.POINTER(LayerDesc)), ("exact_f32", C.c_int),
         ("final_norm_w", C.c_void_p), ("embed_scale", C.c_float), ("final_norm_b", C.c_void_p), ("streams", C.c_int),
+        ("pos_embed", C.c_void_p), ("max_positions", C.c_int),
     ]
 
 
@@ -970,6 +1081,52 @@ def _pack_hyper_layer(spec: LayeredSpec, i: int, l: LayerSpec, w: Dict[str, torc
         d.w_down = dev(torch.stack([w[f"{p}mlp.e{e}.down"].to(device) for e in range(l.experts)])).data_ptr()
 
 
+def _pack_prenorm_layer(spec: LayeredSpec, l: LayerSpec, w: Dict[str, torch.Tensor], p: str, d, W: int, device, dev, keep: list) -> None:
+    """Descriptor of a pre-norm layer: q | latent + shared key part | output gate stacked into w_in, the residual multiplier and
+    the layer scale in one gain, the shared expert's gate as one more row of the router."""
+    f32 = torch.float32
+    m, f = p + "mix.", p + "mlp."
+    d.form, d.mixer = LAYER_PRENORM, MIXER_LATENT_ATTENTION
+    for f_ in ("o_q", "o_k", "o_v", "o_dkv", "o_gate", "o_beta", "o_a1", "o_g1", "o_rg1", "o_rg2", "o_router"):
+        setattr(d, f_, -1)
+    d.norm_gain = 1.0
+    vec = lambda name: dev(w[name], f32).data_ptr()
+    gain = lambda name: dev(w[name].double() * spec.residual_mult, f32).data_ptr()
+    d.norm_pre1, d.res_gain[0] = vec(p + "norm1"), gain(p + "ls1")
+    w_in, offs = _stack_inputs([(n, t.to(device)) for n, t in (("q", w[m + "q"]), ("dkv", w[m + "dkv"]), ("gate", w[m + "g"]))], W, device)
+    keep.append(w_in)
+    d.w_in, d.n_in = w_in.data_ptr(), w_in.shape[0]
+    for n, o in offs.items():
+        setattr(d, "o_" + n, o)
+    d.heads, d.dim, d.vdim, d.kv_rank, d.scale, d.rot_dims, d.gate_wide = l.heads, l.dim, l.vdim, l.kv_rank, l.scale, l.rot_dims, 1
+    if l.rot_dims:
+        i2 = torch.arange(l.rot_dims // 2, dtype=torch.float64)
+        d.rot_freq = dev(torch.tensor(l.rot_base, dtype=torch.float64) ** (-2.0 * i2 / l.rot_dims), f32).data_ptr()
+    d.sink = vec(m + "sink")
+    d.w_uk_t = dev(w[m + "uk"].reshape(l.heads, l.dim, l.kv_rank).transpose(1, 2)).data_ptr()      # [heads][kv_rank][dim]
+    d.w_uv = dev(w[m + "uv"]).data_ptr()
+    d.dkv_norm = vec(m + "dkv.norm")
+    d.w_o = dev(w[m + "o"]).data_ptr()
+    d.ff_kind = FF_NONE
+    if not l.ff_kind:
+        return
+    d.norm_pre2, d.res_gain[1] = vec(p + "norm2"), gain(p + "ls2")
+    d.ff_kind, d.ff, d.ff_act, d.experts, d.top, d.groups, d.keep = FF_MOE, l.ff, ACT_SWIGLU, l.experts, l.top, 1, 1
+    d.route_kind, d.route_norm, d.route_scale = ROUTE_SOFTMAX, 1, 1.0        # softmax over all, divided by the chosen ones' sum
+    d.router_bias = vec(f + "router.b")
+    rows = l.experts + (1 if l.shared_ff else 0)
+    router = torch.zeros((rows + 127) // 128 * 128, W, dtype=torch.bfloat16, device=device)
+    router[:l.experts] = w[f + "router"].to(device)
+    paired = lambda q: _interleave(w[q + "gate"].to(device), w[q + "up"].to(device))
+    if l.shared_ff:
+        router[l.experts] = w[f + "shared.sg"][0].to(device)
+        d.shared_ff, d.shared_gate = l.shared_ff, 1
+        d.w_shared_up, d.w_shared_down = dev(paired(f + "shared.")).data_ptr(), dev(w[f + "shared.down"]).data_ptr()
+    d.w_router, d.router_rows = dev(router).data_ptr(), router.shape[0]
+    d.w_gu = dev(torch.stack([paired(f"{f}e{e}.") for e in range(l.experts)])).data_ptr()
+    d.w_down = dev(torch.stack([w[f"{f}e{e}.down"].to(device) for e in range(l.experts)])).data_ptr()
+
+
 def _pack_postnorm_layer(spec: LayeredSpec, i: int, l: LayerSpec, w: Dict[str, torch.Tensor], p: str, d, W: int, device, dev,
                          keep: list, first_mix: int) -> None:
     """Descriptor of a post-norm layer: gains as stored, input convolutions, depth weights, the mixer's projections stacked
@@ -1064,11 +1221,24 @@ def pack(spec: LayeredSpec, w: Dict[str, torch.Tensor], device, exact_f32: bool 
         keep.append(t)
         return t
 
-    descs = (LayerDesc * len(spec.layers))()
+    runs = spec.runs()
+    descs = (LayerDesc * len(runs))()
     W = spec.width
+    if spec.layers and spec.layers[0].form == "prenorm":
+        packed: Dict[int, LayerDesc] = {}
+        for j, (i, t) in enumerate(runs):        # a layer that runs again is the same descriptor once more
+            if i not in packed:
+                packed[i] = LayerDesc()
+                _pack_prenorm_layer(spec, spec.layers[i], w, f"l{i}.", packed[i], W, device, dev, keep)
+            C.memmove(C.byref(descs[j]), C.byref(packed[i]), C.sizeof(LayerDesc))
+            if t is not None:
+                descs[j].re_embed = int(t > 0)
+                descs[j].pre_add = dev(w["loop.step"][t], torch.float32).data_ptr()
     for i, l in enumerate(spec.layers):
         p, d = f"l{i}.", descs[i]
         m = p + "mix."
+        if l.form == "prenorm":
+            continue
         if l.form == "sandwich":
             _pack_sandwich_layer(l, w, p, d, W, device, dev, keep)
             continue
@@ -1130,10 +1300,13 @@ def pack(spec: LayeredSpec, w: Dict[str, torch.Tensor], device, exact_f32: bool 
         else:
             d.ff_kind = FF_NONE
     model = LayeredModel()
-    model.width, model.vocab, model.n_layers = W, spec.vocab, len(spec.layers)
+    model.width, model.vocab, model.n_layers = W, spec.vocab, len(runs)
     model.eps, model.logit_softcap = spec.eps, spec.logit_softcap
     postnorm = bool(spec.layers) and spec.layers[0].form == "postnorm"
     hyper = bool(spec.layers) and spec.layers[0].form == "hyper"
+    prenorm = bool(spec.layers) and spec.layers[0].form == "prenorm"
+    if prenorm:
+        model.pos_embed, model.max_positions = dev(w["pos"]).data_ptr(), spec.max_positions
     if hyper:                                # a layer norm with gain and bias; the logits come from the embedding table
         model.final_norm_gain = 1.0
         model.final_norm_w = dev(w["final.norm"], torch.float32).data_ptr()
@@ -1142,9 +1315,9 @@ def pack(spec: LayeredSpec, w: Dict[str, torch.Tensor], device, exact_f32: bool 
     elif w["final.norm"].dim() == 0:
         model.final_norm_gain = float(w["final.norm"].float().item())
     else:
-        model.final_norm_gain = 1.0          # sandwich models store gain - 1, post-norm models the gain itself
-        model.final_norm_w = dev(w["final.norm"].float() + (0.0 if postnorm else 1.0), torch.float32).data_ptr()
-    model.embed_scale = spec.embed_scale if postnorm or hyper else 1.0
+        model.final_norm_gain = 1.0          # sandwich models store gain - 1, post-norm and pre-norm models the gain itself
+        model.final_norm_w = dev(w["final.norm"].float() + (0.0 if postnorm or prenorm else 1.0), torch.float32).data_ptr()
+    model.embed_scale = spec.embed_scale if postnorm or hyper or prenorm else 1.0
     model.embed = dev(w["embed"]).data_ptr()
     model.head = model.embed if hyper else dev(w["head"]).data_ptr()
     model.layers = C.cast(descs, C.POINTER(LayerDesc))

@@ -205,7 +205,14 @@ enum { FT_FF_NONE = 0, FT_FF_MOE = 1, FT_FF_DENSE = 2 };
  *                      X_t <- sum_s hc_mix[s][t] X_s + hc_out[t] * sublayer(norm(u)).  The model's last norm reads the sum of
  *                      the streams.  streams <= 1 without the hc tensors is the plain x += sublayer(norm(x)).  Takes the
  *                      channel-delta mixer (rank_a == rank_g == 0) or branch mixers, and any feed-forward. */
-enum { FT_LAYER_GATED = 0, FT_LAYER_SANDWICH = 1, FT_LAYER_POSTNORM = 2, FT_LAYER_HYPER = 3 };
+/*   FT_LAYER_PRENORM:  the plain pre-norm layer with a gain per coordinate on the way back (res_gain, a residual multiplier and
+ *                      a layer scale in one): x += res_gain[0] * mixer(rms(x) * norm_pre1);
+ *                      x += res_gain[1] * ff(rms(x) * norm_pre2).  Before the layer the stream may take the embedding output once
+ *                      more and a vector (re_embed, pre_add): what a model that runs some of its layers several times in a row
+ *                      adds ahead of each pass.  Such a model is given as its layer RUNS: a layer that runs twice is two
+ *                      descriptors with the same weights, each with a cache of its own.  Takes latent attention and any
+ *                      feed-forward. */
+enum { FT_LAYER_GATED = 0, FT_LAYER_SANDWICH = 1, FT_LAYER_POSTNORM = 2, FT_LAYER_HYPER = 3, FT_LAYER_PRENORM = 4 };
 enum { FT_ACT_SWIGLU = 0, FT_ACT_RELU2 = 1 };          /* expert: W_down (silu(W_gate h) * W_up h)  |  W_down relu(W_up h)^2 */
 enum { FT_ROUTE_SOFTMAX = 0, FT_ROUTE_SIGMOID = 1 };   /* router scores over all experts */
 
@@ -375,6 +382,22 @@ typedef struct {
     const float* hc_out[2];    /* fp32 [streams]: how its result joins each stream; null = ones */
     const float* hc_mix[2];    /* fp32 [streams][streams], [from][to]; null = identity */
     int route_input;           /* mixture of experts: 1 = a chosen score multiplies its expert's INPUT (sum_e expert_e(s_e h)), not its output */
+    /* ---- FT_LAYER_PRENORM ---- */
+    const float* res_gain[2];  /* fp32 [width] on the mixer's and the feed-forward's result; null = ones */
+    int re_embed;              /* 1: the embedding output is added to the stream before this layer (run) */
+    const float* pre_add;      /* fp32 [width] or null: added to the stream after that */
+    /* ---- latent attention options (any layer form that takes it) ----
+     * rot_dims > 0: a head's query is dim plain | rot_dims rotated columns, the latent projection has kv_rank + rot_dims columns
+     * and its last rot_dims (not normed) are ONE rotated key part shared by the heads; pairs (i, i + rot_dims / 2), angle of pair
+     * i at position p = p * rot_freq[i]; score = (plain . plain + rotated . rotated) * scale.  The cache row is
+     * [normed latent | rotated key part]. */
+    int rot_dims;
+    const float* rot_freq;     /* fp32 [rot_dims / 2] */
+    const float* sink;         /* fp32 [heads] or null: exp(sink_h) joins the softmax denominator, no key, no value, not scaled */
+    int gate_wide;             /* o_gate: 0 = one column per head, 1 = heads * vdim columns that gate the concatenated heads */
+    /* ---- router and shared expert options of the forms whose router is a matrix of its own ---- */
+    const float* router_bias;  /* fp32 [experts] or null: added to the router logits */
+    int shared_gate;           /* 1: row `experts` of w_router gates the shared expert's output by its sigmoid, one number per token */
 } ft_layer_desc;
 
 typedef struct {
@@ -390,9 +413,12 @@ typedef struct {
                                   the tensor cores (tcgen05) from bf16 hi + lo planes of the fp32 activations with fp32
                                   accumulation; norms, scores, softmax, router, recurrence and residual stay fp32 */
     const float* final_norm_w; /* fp32 [width] or null: a gain per coordinate instead of final_norm_gain */
-    float embed_scale;         /* FT_LAYER_POSTNORM / FT_LAYER_HYPER models: the embedding output is embed[token] * embed_scale (0 = 1) */
+    float embed_scale;         /* FT_LAYER_POSTNORM / _HYPER / _PRENORM models: the embedding output is embed[token] * embed_scale (0 = 1) */
     const float* final_norm_b; /* FT_LAYER_HYPER models: the last norm is a layer norm with gain final_norm_w and this bias */
     int streams;               /* FT_LAYER_HYPER models: copies of the stream (0 = 1) */
+    const void* pos_embed;     /* FT_LAYER_PRENORM models: bf16 [max_positions, width] or null, a learned vector per position that the
+                                  embedding output takes (not scaled) */
+    int max_positions;         /* rows of pos_embed: no sequence grows beyond it */
 } ft_layered_model;
 
 /* cfg: vocab, max_batch, max_batched_tokens, num_pages, max_context, max_sessions (= state slots), eos, debug_logit_rows
