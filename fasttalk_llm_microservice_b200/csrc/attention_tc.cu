@@ -57,26 +57,6 @@ struct TcCfg {
     static_assert(256 + 2 * D <= 512, "tensor memory");
 };
 
-__device__ __forceinline__ void tmem_ld16_nowait(uint32_t taddr, uint32_t* r) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x16.b32 "
-        "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
-        : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-          "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
-        : "r"(taddr)
-        : "memory");
-}
-__device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
-__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t* r) {
-    asm volatile(
-        "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
-        "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};" ::"r"(taddr),
-        "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]),
-        "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
-        : "memory");
-}
-__device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
-
 // 3-D tiled tensor-map copy (d, head, token) -> shared memory
 __device__ __forceinline__ void tma_tile_3d(void* dst_smem, const CUtensorMap* map, int c0, int c1, int c2, uint64_t* bar) {
     asm volatile(
@@ -84,34 +64,6 @@ __device__ __forceinline__ void tma_tile_3d(void* dst_smem, const CUtensorMap* m
             smem_u32(dst_smem)),
         "l"(map), "r"(smem_u32(bar)), "r"(c0), "r"(c1), "r"(c2)
         : "memory");
-}
-// MN-major SWIZZLE_128B operand (V slab): 8-row groups (8 keys x 128 B) 1024 B apart along K; one 64-element MN block
-__device__ __forceinline__ uint64_t umma_desc_mn128(uint32_t smem_addr) {
-    uint64_t d = 0;
-    d |= (uint64_t)((smem_addr & 0x3ffff) >> 4);
-    d |= (uint64_t)(TC_SUB_BYTES >> 4) << 16;   // LBO: stride between 64-element MN blocks = one sub-slab (d = 128: two blocks)
-    d |= (uint64_t)(1024 >> 4) << 32;       // SBO: stride between 8-row K groups
-    d |= (uint64_t)1 << 46;
-    d |= (uint64_t)2 << 61;                 // SWIZZLE_128B
-    return d;
-}
-// D[tmem] (+)= A[tmem] * B[smem desc]: the A operand (P, fp16 pairs packed into 32-bit columns, row = lane) is read
-// from tensor memory, so only V crosses the shared-memory port — with both operands in shared memory an
-// M128 N64 product asks for 192 B/clk, more than the port's 128 B/clk
-__device__ __forceinline__ void umma_f16_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc,
-                                            uint32_t accumulate) {
-    asm volatile(
-        "{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-        "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}\n" ::"r"(d_tmem),
-        "r"(a_tmem), "l"(b_desc), "r"(idesc), "r"(accumulate)
-        : "memory");
-}
-// 2^x on the SFU, one instruction: the arguments here are <= 2^8 by construction (lazy rescale) and anything below
-// -126 may flush to zero, so exp2f()'s range fix-up (a compare and two multiplies per element) buys nothing
-__device__ __forceinline__ float ex2_fast(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
 }
 __device__ __forceinline__ void mbar_wait_sleep(uint64_t* bar, uint32_t parity) {
     while (!mbar_try_wait(bar, parity)) __nanosleep(20);

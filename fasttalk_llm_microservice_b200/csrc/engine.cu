@@ -146,6 +146,7 @@ struct Engine {
     int prof_used = 0;
     long long prof_ctx_sum = 0;            // sum of context lengths of the step's decode rows
     cudaEvent_t t0 = nullptr, t1 = nullptr;
+    int* h_kernel_err = nullptr;           // pinned, mapped: a kernel whose wait ran out sets it
     // device time of every step (events on the engine stream around upload .. sampled-token copy)
     cudaEvent_t s0 = nullptr, s1 = nullptr;
     struct StepRec { float gpu_ms, n_decode, n_prefill, host_ms; };
@@ -575,6 +576,7 @@ static int forward(Engine* e, const Batch& b) {
 // as bf16 hi + lo planes (`hi` / `lo` if the producer already wrote them, else staged here), fp32 out.  Otherwise, and always
 // in the exact-fp32 form, the CUDA-core kernels.
 constexpr int kTensorMinRows = 9;
+constexpr int kLatentTcMinTokens = 32;       // portion tokens of a step from which latent attention takes 128-row tiles
 constexpr int kFuseCanonRows = 256;          // steps up to this many rows form the feed-forward's input inside the post-norm kernel
 constexpr int kMoeTensorMinPairs = 256;      // (token, choice) pairs from which the experts run as per-expert tensor-core GEMMs
 static int dense(Engine* e, const float* A, const void* hi, const void* lo, const void* W, float* C, int T, int N, int K,
@@ -947,7 +949,7 @@ static int forward_layered(Engine* e, const Batch& b) {
             la.proj = L.proj; la.ldp = ld; la.o_q = c.o_q; la.o_dkv = c.o_dkv; la.o_gate = c.gate_wide ? -1 : c.o_gate;
             la.norm_w = c.dkv_norm; la.eps = M.eps; la.rot_freq = c.rot_freq; la.sink = c.sink; la.qlat = L.b1; la.out = L.b2;
             la.cache = L.lat_cache ? L.lat_cache + ll.cache_off : nullptr;
-            la.cache16 = L.lat_cache16 ? (uint8_t*)L.lat_cache16 + ll.cache16_off * 2 : nullptr;
+            la.cache16 = L.lat_cache16 && latent_attn_mma_ok(c.kv_rank, R) ? (uint8_t*)L.lat_cache16 + ll.cache16_off * 2 : nullptr;
             la.part = L.attn_part; la.positions = d + m.o_pos; la.seq_rows = d + m.o_rows; la.page_table = d + m.o_pt;
             la.max_pages = e->max_pages; la.H = c.heads; la.dim = c.dim; la.rank = c.kv_rank; la.rot = R; la.scale = c.scale;
             FT_TRY(launch_latent_prep(la, T, st));
@@ -957,7 +959,17 @@ static int forward_layered(Engine* e, const Batch& b) {
             a.C = L.b1; a.ldc = c.heads * kd; a.c_col_stride = kd;
             a.M = T; a.N = c.kv_rank; a.K = c.dim; a.P = c.heads;
             FT_TRY(launch_linear(a, T, st));
-            FT_TRY(launch_latent_attn(la, T, st));
+            // prompt portions on tcgen05, single tokens of running sequences (and steps of a few portion tokens) row by row
+            const bool tc = la.cache16 && b.n_tiles > 0 && T - b.n_decode >= kLatentTcMinTokens && latent_prefill_tc_ok(c.kv_rank, R);
+            if (tc) {
+                WindowTiles tm;
+                tm.tile_req = d + m.o_treq; tm.tile_q0 = d + m.o_tq0; tm.req_q_start = d + m.o_qstart; tm.req_slot = d + m.o_rslot;
+                tm.req_pos0 = d + m.o_rpos0; tm.n_tiles = b.n_tiles;
+                FT_TRY(launch_latent_prefill_tc(la, tm, e->h_kernel_err, st));
+                launched(b.n_decode > 0 ? 1 : 0);
+            }
+            const int rows = tc ? b.n_decode : T;
+            if (rows > 0) FT_TRY(launch_latent_attn(la, rows, st));
             LinearArgs v;                   // values out of latent space: o_h = W_uv_h (sum_j p_j c_j)
             v.A = L.b2; v.lda = c.heads * c.kv_rank; v.a_col_stride = c.kv_rank;
             v.W = (const __nv_bfloat16*)c.w_uv; v.w_stride = (long long)c.vdim * c.kv_rank; v.ldw = c.kv_rank;
@@ -1183,6 +1195,14 @@ static int forward_layered(Engine* e, const Batch& b) {
     return 0;
 }
 
+// After a step's synchronize: did a kernel give up on one of its waits?
+static int check_kernel_err(Engine* e) {
+    if (!e->h_kernel_err || *(volatile int*)e->h_kernel_err == 0) return 0;
+    *e->h_kernel_err = 0;
+    FT_REQUIRE(false, "engine: a kernel of the step gave up waiting for its own copies or products; the step's results are not valid");
+    return -1;
+}
+
 static int upload_meta(Engine* e) {
     FT_CHECK_CUDA(cudaMemcpyAsync(e->meta.d, e->meta.h, e->meta.upload_ints * sizeof(int),
                                   cudaMemcpyHostToDevice, e->stream));
@@ -1393,6 +1413,7 @@ static int engine_step(Engine* e, std::unique_lock<std::mutex>& lk) {
     for (Request* r : dec) r->in_flight = false;
     for (Request* r : pre) r->in_flight = false;
     FT_CHECK_CUDA(sync_rc);
+    FT_TRY(check_kernel_err(e));
     e->st.d2h_bytes += (long long)b.n_logit_rows * sizeof(int);
     {
         float ms = 0.f;
@@ -1859,8 +1880,8 @@ static int engine_init_layered(Engine* e) {
             ll.cache_off = cache_floats;
             cache_floats += (size_t)c.num_pages * kKvTile * (d.kv_rank + d.rot_dims);
             ll.cache16_off = cache16;
-            cache16 += (size_t)c.num_pages * kKvTile * latent_row16(d.kv_rank, d.rot_dims);
-            if (!latent_attn_mma_ok(d.kv_rank, d.rot_dims)) latent_f32 = true;
+            if (latent_attn_mma_ok(d.kv_rank, d.rot_dims)) cache16 += (size_t)c.num_pages * kKvTile * latent_row16(d.kv_rank, d.rot_dims);
+            else latent_f32 = true;
             buf = std::max(buf, (size_t)d.heads * (d.kv_rank + d.rot_dims));
             rank_max = std::max(rank_max, d.kv_rank);
         } else if (d.mixer == FT_MIXER_CHANNEL_DELTA) {
@@ -1908,8 +1929,12 @@ static int engine_init_layered(Engine* e) {
         FT_CHECK_CUDA(cudaMemsetAsync(*p, 0, std::max<size_t>(bytes, 16), e->stream));
         return 0;
     };
+    if (cache16 && M.exact_f32 == 0) {
+        FT_CHECK_CUDA(cudaHostAlloc(&e->h_kernel_err, sizeof(int), cudaHostAllocMapped));
+        *e->h_kernel_err = 0;
+    }
     if (latent_f32) FT_TRY(alloc(&L.lat_cache, cache_floats * 4));
-    if (M.exact_f32 == 0) FT_TRY(alloc(&L.lat_cache16, cache16 * 2));
+    if (cache16 && M.exact_f32 == 0) FT_TRY(alloc(&L.lat_cache16, cache16 * 2));
     FT_TRY(alloc(&L.state, L.slot_stride * (size_t)c.max_sessions * 4));
     if (kv_floats) FT_TRY(alloc(&L.kv_cache, kv_floats * 4));
     if (br_fin) {
@@ -1998,6 +2023,7 @@ static void engine_free(Engine* e) {
     cudaFree(e->attn_scratch); cudaFree(e->meta.d);
     cudaFree(e->w16_qkv); cudaFree(e->w16_o); cudaFree(e->w16_gu); cudaFree(e->w16_d);
     cudaFree(e->x16_xn); cudaFree(e->x16_attn); cudaFree(e->x16_act);
+    if (e->h_kernel_err) cudaFreeHost(e->h_kernel_err);
     if (e->lay) {
         Layered& L = *e->lay;
         cudaFree(L.lat_cache); cudaFree(L.lat_cache16); cudaFree(L.state); cudaFree(L.hn); cudaFree(L.proj); cudaFree(L.b1); cudaFree(L.b2); cudaFree(L.scan_ws);
@@ -2171,6 +2197,7 @@ extern "C" int ft_engine_feed(ft_engine* h, int n_entries, const unsigned long l
         if (!rc) {
             const cudaError_t se = cudaStreamSynchronize(e->stream);
             if (se != cudaSuccess) { set_last_error("ft_engine_feed: %s", cudaGetErrorString(se)); rc = -1; }
+            else rc = check_kernel_err(e);
         }
         if (!rc) {
             for (int i = 0; i < n_entries; ++i)
@@ -2606,6 +2633,7 @@ extern "C" int ft_debug_prefill_logits(ft_engine* h, const int* tokens, int n, i
             set_last_error("ft_debug_prefill_logits: %s", cudaGetErrorString(cudaGetLastError()));
             rc = -1;
         }
+        if (!rc) rc = check_kernel_err(e);
     }
     release_pages_beyond(e, &tmp, 0);
     if (tmp.slot >= 0) e->free_slots.push_back(tmp.slot);

@@ -138,7 +138,7 @@ struct LatentArgs {
     const float* sink = nullptr;                  // [H] or null: exp(sink) joins the softmax denominator
     float* qlat = nullptr;                        // [T][H][rank + rot]
     float* cache = nullptr;                       // this layer's [pages][64][rank + rot] fp32, or null
-    void* cache16 = nullptr;                      // this layer's [pages][64][latent_row16] bf16, or null
+    void* cache16 = nullptr;                      // this layer's bf16 pages (latent_row16), or null
     float* out = nullptr;                         // [T][H][rank] attended latents
     float* part = nullptr;                        // room for split keys (see below), or null
     const int *positions = nullptr, *seq_rows = nullptr, *page_table = nullptr;
@@ -154,8 +154,13 @@ int latent_attn_splits(int T, int H);
 // With cache16 and sizes the tensor-core kernel is built for (latent_attn_mma_ok) the attention runs on mma.sync from bf16
 // operands and `cache` may be null; otherwise on the CUDA cores in fp32.
 bool latent_attn_mma_ok(int rank, int rot);
-int latent_row16(int rank, int rot);              // columns of a bf16 cache row: both parts padded with zeros to multiples of 32
-int launch_latent_attn(const LatentArgs& a, int T, cudaStream_t stream);
+int launch_latent_attn(const LatentArgs& a, int T, cudaStream_t stream);      // the step's first T rows
+// A page of the bf16 cache: [64-column block][64 tokens][64 columns], rows of latent_row16 columns (rank + rot padded with zeros to
+// a multiple of 64), the eight 16-byte chunks of a 128-byte row XOR-swizzled by the token: chunk ch of token j's row lies at
+int latent_row16(int rank, int rot);
+__host__ __device__ inline int latent_chunk16(int j, int ch) {      // elements from the page's start
+    return (ch >> 3) * (kKvTile * 64) + j * 64 + (((ch & 7) ^ (j & 7)) << 3);
+}
 struct DeltaArgs {
     const float* proj = nullptr;      // [T][ldp]: raw q | k | v at column o_q, beta logits at o_beta
     int ldp = 0, o_q = 0, o_beta = 0;
@@ -250,6 +255,11 @@ struct WindowTiles {
 };
 // n_single: how many of the step's first rows are single tokens of running sequences (they precede the portions)
 int launch_window_attention(const WindowArgs& a, int T, int n_single, const WindowTiles& tm, cudaStream_t stream);
+
+// ---- latent_tc.cu: latent attention of the step's prompt portions on tcgen05, from the bf16 cache.  err: set when a wait inside
+// the kernel ran out (never, unless something is broken); mapped host memory or null
+bool latent_prefill_tc_ok(int rank, int rot);
+int launch_latent_prefill_tc(const LatentArgs& a, const WindowTiles& tm, int* err, cudaStream_t stream);
 
 // S <- a_t S + b_t k_t v_t^T, o_t = S^T q_t per (request, head) over the request's rows in order; S [dim][vd] of head h at
 // state + slot * slot_stride + s_off + h * dim * vd, zero at a sequence's start (req_pos0 == 0).

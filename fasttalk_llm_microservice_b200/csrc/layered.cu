@@ -479,9 +479,9 @@ int launch_gather_rows(const float* src, const int* idx, float* dst, int n, int 
 
 // ------------------------------------------------------------------ latent attention
 // Token t: c = raw / sqrt(mean(raw^2) + eps) * w and the rotated shared key part go to page_table[seq_rows[t]][pos / 64], row
-// pos % 64 of the layer's caches ([page][64][rank + rot] fp32; bf16 with both parts padded to multiples of 32); the rotated part
+// pos % 64 of the layer's caches ([page][64][rank + rot] fp32; bf16 as latent_chunk16 lays a page out); the rotated part
 // of every query head goes to qlat.  Pairs (i, i + rot / 2); the angle's sine and cosine are formed once per token.
-__global__ void __launch_bounds__(128) latent_prep_kernel(LatentArgs a, int row16, int rot_at16) {
+__global__ void __launch_bounds__(128) latent_prep_kernel(LatentArgs a, int row16) {
     __shared__ float red[33];
     extern __shared__ float trig[];                        // [rot / 2] cosines, [rot / 2] sines
     const int t = blockIdx.x, rank = a.rank, rot = a.rot, half = rot >> 1;
@@ -494,19 +494,20 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentArgs a, int row1
     ss = block_sum(ss, red);                               // its barriers also publish trig
     const float r = 1.f / sqrtf(ss / (float)rank + a.eps);
     const int page = a.page_table[(size_t)a.seq_rows[t] * a.max_pages + pos / kKvTile];
-    const size_t at = (size_t)page * kKvTile + pos % kKvTile;
-    float* c32 = a.cache ? a.cache + at * (rank + rot) : nullptr;
-    __nv_bfloat16* c16 = a.cache16 ? (__nv_bfloat16*)a.cache16 + at * row16 : nullptr;
+    const int slot = pos % kKvTile;
+    float* c32 = a.cache ? a.cache + ((size_t)page * kKvTile + slot) * (rank + rot) : nullptr;
+    __nv_bfloat16* c16 = a.cache16 ? (__nv_bfloat16*)a.cache16 + (size_t)page * kKvTile * row16 : nullptr;
+    auto at16 = [&](int c) { return latent_chunk16(slot, c >> 3) + (c & 7); };
     for (int c = threadIdx.x; c < rank; c += blockDim.x) {
         const float v = raw[c] * r * a.norm_w[c];
         if (c32) c32[c] = v;
-        if (c16) c16[c] = __float2bfloat16_rn(v);
+        if (c16) c16[at16(c)] = __float2bfloat16_rn(v);
     }
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         const float u = raw[rank + i], v = raw[rank + half + i], cs = trig[i], sn = trig[half + i];
         const float x = u * cs - v * sn, y = v * cs + u * sn;
         if (c32) { c32[rank + i] = x; c32[rank + half + i] = y; }
-        if (c16) { c16[rot_at16 + i] = __float2bfloat16_rn(x); c16[rot_at16 + half + i] = __float2bfloat16_rn(y); }
+        if (c16) { c16[at16(rank + i)] = __float2bfloat16_rn(x); c16[at16(rank + half + i)] = __float2bfloat16_rn(y); }
     }
     const int hd = a.dim + rot, kd = rank + rot;
     for (int j = threadIdx.x; j < a.H * half; j += blockDim.x) {
@@ -652,7 +653,7 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, int n_p
 int launch_latent_prep(const LatentArgs& a, int T, cudaStream_t stream) {
     FT_REQUIRE(a.proj && a.norm_w && (a.cache || a.cache16) && (a.rot == 0 || (a.rot_freq && a.qlat && a.rot % 2 == 0)),
                "latent prep: missing operands");
-    latent_prep_kernel<<<T, 128, (size_t)a.rot * 4, stream>>>(a, latent_row16(a.rank, a.rot), (a.rank + 31) / 32 * 32);
+    latent_prep_kernel<<<T, 128, (size_t)a.rot * 4, stream>>>(a, latent_row16(a.rank, a.rot));
     FT_CHECK_CUDA(cudaGetLastError());
     return 0;
 }
@@ -663,8 +664,8 @@ int launch_latent_prep(const LatentArgs& a, int T, cudaStream_t stream) {
 // (16 latents from the bf16 copy of the cache) is copied into the warp's own double buffer with cp.async one tile ahead,
 // S = Q C^T (ldmatrix fragments of Q and of the tile), online softmax in registers, O += P C with the SAME tile read
 // through ldmatrix.trans — keys and values are one array.  The warps' (max, sum, O) are merged through shared memory.
-// Both parts of a row are padded with zeros to multiples of 32 columns: kc 32-column pieces per row, vc of them the latent.  A
-// CTA sums VC <= 8 of those (O is 4 * VC accumulator tiles per thread).
+// kc 32-column pieces per row, the first vc of them hold the latent (the last of those may hold rotated columns too, whose sums
+// nobody reads).  A CTA sums VC <= 8 pieces (O is 4 * VC accumulator tiles per thread).
 __device__ __forceinline__ void cp_async16(void* dst_smem, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst_smem)), "l"(src) : "memory");
 }
@@ -681,12 +682,11 @@ latent_attn_mma_kernel(LatentArgs a, int kc, int vc, int head_groups, int n_spli
     uint8_t* kbuf = lat_smem + TILE + (size_t)warp * 2 * TILE;
     const int t = blockIdx.x, split = blockIdx.y, h0 = (blockIdx.z % head_groups) * 16;
     const int v_first = (blockIdx.z / head_groups) * VC;   // first 32-column piece of the values this CTA sums
-    const int H = a.H, rank = a.rank, kd = a.rank + a.rot, rot_at = 32 * vc;
+    const int H = a.H, rank = a.rank, kd = a.rank + a.rot;
     const __nv_bfloat16* cache16 = (const __nv_bfloat16*)a.cache16;
     for (int idx = threadIdx.x; idx < 16 * row; idx += 128) {
         const int r = idx / row, c = idx % row;
-        const int src = c < rot_at ? (c < rank ? c : -1) : (c - rot_at < a.rot ? rank + c - rot_at : -1);
-        const float v = h0 + r < H && src >= 0 ? a.qlat[((size_t)t * H + h0 + r) * kd + src] * a.scale : 0.f;
+        const float v = h0 + r < H && c < kd ? a.qlat[((size_t)t * H + h0 + r) * kd + c] * a.scale : 0.f;
         *reinterpret_cast<__nv_bfloat16*>(Qs + r * RS + c * 2) = __float2bfloat16_rn(v);
     }
     __syncthreads();
@@ -705,7 +705,7 @@ latent_attn_mma_kernel(LatentArgs a, int kc, int vc, int head_groups, int n_spli
         for (int i = lane; i < 16 * 4 * kc; i += 32) {          // 16 rows of 4 * kc 16-byte pieces
             const int r = i / (4 * kc), ch = i % (4 * kc);
             const int j = min(key0 + r, j_hi - 1);
-            cp_async16(dst + r * RS + ch * 16, cache16 + ((size_t)pt[j / kKvTile] * kKvTile + j % kKvTile) * row + ch * 8);
+            cp_async16(dst + r * RS + ch * 16, cache16 + (size_t)pt[j / kKvTile] * kKvTile * row + latent_chunk16(j % kKvTile, ch));
         }
         cp_async_commit();
     };
@@ -835,10 +835,11 @@ int latent_attn_splits(int T, int H) {
     return std::max(1, std::min(kLatentMaxSplits, kLatentSplitPairs / std::max(pairs, 1)));
 }
 
-int latent_row16(int rank, int rot) { return (rank + 31) / 32 * 32 + (rot + 31) / 32 * 32; }
+int latent_row16(int rank, int rot) { return (rank + rot + 63) / 64 * 64; }
 // the query tile and the four warps' double-buffered key tiles, 16 rows each
 static size_t latent_mma_smem(int rank, int rot) { return (size_t)9 * 16 * (latent_row16(rank, rot) * 2 + 16); }
-bool latent_attn_mma_ok(int rank, int rot) { return rank >= 1 && latent_mma_smem(rank, rot) <= 224 * 1024; }
+// the serving form keeps latents of whole 32-column pieces in bf16; other sizes stay in fp32 on the CUDA cores
+bool latent_attn_mma_ok(int rank, int rot) { return rank >= 32 && rank % 32 == 0 && latent_mma_smem(rank, rot) <= 224 * 1024; }
 
 int launch_latent_attn(const LatentArgs& a, int T, cudaStream_t stream) {
     const int n_pairs = T * a.H;

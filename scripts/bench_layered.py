@@ -4,6 +4,7 @@
     python bench.py --design gedelorn [--sizes s,m] [--arms gedelorn,gitozen,llama] [--steps K] [--warmup W]
     python bench.py --design vonedra  [--sizes s,m] [--arms vonedra,gedelorn,gitozen,llama] [--steps K] [--warmup W]
     python bench.py --design lotinex  [--sizes s,m] [--arms lotinex,vonedra,gedelorn,llama] [--steps K] [--warmup W]
+    python bench.py --design gedalix  [--sizes s,m,l] [--arms gedalix,gitozen,vonedra,llama] [--steps K] [--warmup W]
 
 For every size all arms get the same width, depth, heads x head size, active feed-forward width (top x expert ff =
 Llama's ffn) and vocabulary.  Gedelorn's closest relative in the framework is Gitozen (the same engine path: stacked
@@ -32,6 +33,7 @@ DECODE_CTX = 1024
 SIZES = {
     "s": dict(width=1024, order="ladl", heads=8, dim=128, kv_rank=128, experts=8, top=2, ff=512, vocab=16384),
     "m": dict(width=2048, order="ladl", heads=16, dim=128, kv_rank=256, experts=16, top=2, ff=1024, vocab=32768),
+    "l": dict(width=4096, order="ladl", heads=32, dim=128, kv_rank=512, experts=16, top=2, ff=2048, vocab=32768),
 }
 
 
@@ -114,6 +116,20 @@ def lotinex_spec(name, c):
     return spec_from_config(cfg, name=f"lotinex-{name}")
 
 
+def gedalix_spec(name, c):
+    """Four pre-norm layer runs: three layers of latent attention (64 rotated coordinates beside every head's plain part) + experts
+    with a shared expert, the middle one run twice.  Heads x head size, latent size and experts as in the other arms."""
+    from fasttalk_llm_microservice_b200.layered import spec_from_config
+    W, H, D = c["width"], c["heads"], c["dim"]
+    mixer = {"dim": D, "heads": H, "kv_rank": c["kv_rank"], "rot": {"base": 1e4, "dims": 64}, "rot_dim": 64, "scale": (D + 64) ** -0.5,
+             "vdim": D}
+    moe = {"expert": {"ff": c["ff"]}, "kind": "moe", "router": {"experts": c["experts"], "top": c["top"]}, "shared": {"ff": c["ff"]}}
+    layers = [{"type": "latent_attention", "mixer": dict(mixer), "mlp": dict(moe)} for _ in range(3)]
+    cfg = {"architecture": "Gedalix", "embedding": {"scale": 1.0}, "layers": layers, "loop": {"start": 1, "stop": 2, "times": 2},
+           "max_positions": 2 * PREFILL, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "vocab": c["vocab"], "width": W}
+    return spec_from_config(cfg, name=f"gedalix-{name}")
+
+
 def llama_spec(name, c):
     from fasttalk_llm_microservice_b200.model_spec import ModelSpec
     return ModelSpec(name=f"llama-{name}", hidden=c["width"], ffn=c["top"] * c["ff"], layers=len(c["order"]),
@@ -176,11 +192,12 @@ def run(args) -> None:
         c = SIZES[name]
         row = {"config": c}
         design = getattr(args, "design", "") or "gitozen"
-        default_arms = {"lotinex": "lotinex,vonedra,gedelorn,llama", "vonedra": "vonedra,gedelorn,gitozen,llama",
+        default_arms = {"gedalix": "gedalix,gitozen,vonedra,llama", "lotinex": "lotinex,vonedra,gedelorn,llama", "vonedra": "vonedra,gedelorn,gitozen,llama",
                         "gedelorn": "gedelorn,gitozen,llama"}.get(design, "gitozen,llama")
         for arm in (getattr(args, "arms", "") or default_arms).split(","):
-            if arm in ("gitozen", "gedelorn", "vonedra", "lotinex"):
-                spec = {"gitozen": gitozen_spec, "gedelorn": gedelorn_spec, "vonedra": vonedra_spec, "lotinex": lotinex_spec}[arm](name, c)
+            specs = {"gitozen": gitozen_spec, "gedelorn": gedelorn_spec, "vonedra": vonedra_spec, "lotinex": lotinex_spec, "gedalix": gedalix_spec}
+            if arm in specs:
+                spec = specs[arm](name, c)
                 w = init_layered(spec, seed=0, device="cuda")
             else:
                 spec = llama_spec(name, c)
