@@ -608,6 +608,12 @@ static int dense(Engine* e, const float* A, const void* hi, const void* lo, cons
     return 0;
 }
 
+// Projections of every head side by side: as dense(), one launch for all heads.
+static int heads(Engine* e, const LinearArgs& a) {
+    if (e->lay->tensor && a.M >= kTensorMinRows && linear_heads_ok(a)) return launch_linear_heads(a, e->h_kernel_err, e->stream);
+    return launch_linear(a, a.M, e->stream);
+}
+
 // layer forms whose feed-forward reads a normed input of its own: its projections (the router among them) are not part of w_in
 static bool own_ff(const ft_layer_desc& c) {
     return c.form == FT_LAYER_SANDWICH || c.form == FT_LAYER_HYPER || c.form == FT_LAYER_PRENORM;
@@ -958,7 +964,7 @@ static int forward_layered(Engine* e, const Batch& b) {
             a.W = (const __nv_bfloat16*)c.w_uk_t; a.w_stride = (long long)c.kv_rank * c.dim; a.ldw = c.dim;
             a.C = L.b1; a.ldc = c.heads * kd; a.c_col_stride = kd;
             a.M = T; a.N = c.kv_rank; a.K = c.dim; a.P = c.heads;
-            FT_TRY(launch_linear(a, T, st));
+            FT_TRY(heads(e, a));
             // prompt portions on tcgen05, single tokens of running sequences (and steps of a few portion tokens) row by row
             const bool tc = la.cache16 && b.n_tiles > 0 && T - b.n_decode >= kLatentTcMinTokens && latent_prefill_tc_ok(c.kv_rank, R);
             if (tc) {
@@ -976,7 +982,7 @@ static int forward_layered(Engine* e, const Batch& b) {
             v.C = L.b3; v.ldc = c.heads * c.vdim; v.c_col_stride = c.vdim;
             v.M = T; v.N = c.vdim; v.K = c.kv_rank; v.P = c.heads;
             if (c.gate_wide) { v.gate = L.proj + c.o_gate; v.ldg = ld; }
-            FT_TRY(launch_linear(v, T, st));
+            FT_TRY(heads(e, v));
             launched(4);
             mixed = L.b3;
         } else {
@@ -1929,7 +1935,7 @@ static int engine_init_layered(Engine* e) {
         FT_CHECK_CUDA(cudaMemsetAsync(*p, 0, std::max<size_t>(bytes, 16), e->stream));
         return 0;
     };
-    if (cache16 && M.exact_f32 == 0) {
+    if (M.exact_f32 == 0) {
         FT_CHECK_CUDA(cudaHostAlloc(&e->h_kernel_err, sizeof(int), cudaHostAllocMapped));
         *e->h_kernel_err = 0;
     }

@@ -113,6 +113,10 @@ struct LinearArgs {
 };
 // rows_bound: M when batched; an upper bound of seg[P] when grouped
 int launch_linear(const LinearArgs& a, int rows_bound, cudaStream_t stream);
+// ---- heads_tc.cu: a batched LinearArgs (seg, a_rows null) on tcgen05, fp32 activations as bf16 hi + lo planes; K and N whole
+// 32-column pieces.  err as for launch_latent_prefill_tc
+bool linear_heads_ok(const LinearArgs& a);
+int launch_linear_heads(const LinearArgs& a, int* err, cudaStream_t stream);
 // hi / lo (may be null): the normed row once more as bf16 planes, the input form of the tensor-core projections
 // gain_w (may be null): a gain per coordinate instead of the single `gain`
 int launch_embed_norm(const int* tokens, const void* embed, float* x, float* hn, void* hi, void* lo, int T, int W, float eps,

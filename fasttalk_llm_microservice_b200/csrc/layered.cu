@@ -626,27 +626,26 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(LatentArgs a, int n_pa
     }
 }
 
-// The shares of one (token, head) put together: one warp each.
-__global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, int n_pairs, int n_split) {
-    const int pair = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (pair >= n_pairs) return;
-    const int rank = a.rank;
+// The shares of one (token, head) put together: one CTA each.
+__global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, int n_split) {
+    __shared__ float share[kLatentMaxSplits];              // what a share's sums count in the result
+    const int pair = blockIdx.x, rank = a.rank;
     const float* p = a.part + (size_t)pair * n_split * (rank + 2);
-    float m = -INFINITY;
-    for (int s = 0; s < n_split; ++s) m = fmaxf(m, p[(size_t)s * (rank + 2)]);
-    float l = 0.f;
-    for (int s = 0; s < n_split; ++s) {
-        const float ms = p[(size_t)s * (rank + 2)];
-        if (ms > -INFINITY) l += p[(size_t)s * (rank + 2) + 1] * expf(ms - m);
+    if (threadIdx.x < 32) {
+        const int s = threadIdx.x;
+        const float ms = s < n_split ? p[(size_t)s * (rank + 2)] : -INFINITY;
+        const float m = warp_max(ms);
+        const float w = ms > -INFINITY ? expf(ms - m) : 0.f;
+        const float l = warp_sum(w > 0.f ? p[(size_t)s * (rank + 2) + 1] * w : 0.f);
+        if (s < n_split) share[s] = w * latent_finish(m, l, a, pair / a.H, pair % a.H);
     }
-    const float g = latent_finish(m, l, a, pair / a.H, pair % a.H);
-    for (int c = lane; c < rank; c += 32) {
+    __syncthreads();
+    for (int c = threadIdx.x; c < rank; c += blockDim.x) {
         float v = 0.f;
-        for (int s = 0; s < n_split; ++s) {
-            const float ms = p[(size_t)s * (rank + 2)];
-            if (ms > -INFINITY) v = fmaf(p[(size_t)s * (rank + 2) + 2 + c], expf(ms - m), v);
-        }
-        a.out[(size_t)pair * rank + c] = v * g;
+#pragma unroll
+        for (int s = 0; s < kLatentMaxSplits; ++s)
+            if (s < n_split && share[s] > 0.f) v = fmaf(p[(size_t)s * (rank + 2) + 2 + c], share[s], v);
+        a.out[(size_t)pair * rank + c] = v;
     }
 }
 
@@ -880,7 +879,7 @@ int launch_latent_attn(const LatentArgs& a, int T, cudaStream_t stream) {
     }
     FT_CHECK_CUDA(cudaGetLastError());
     if (n_split > 1) {
-        latent_merge_kernel<<<(n_pairs + 3) / 4, 128, 0, stream>>>(a, n_pairs, n_split);
+        latent_merge_kernel<<<n_pairs, 128, 0, stream>>>(a, n_split);
         FT_CHECK_CUDA(cudaGetLastError());
     }
     return 0;
