@@ -336,7 +336,9 @@ def run_plan(eng, seqs, plan):
 def test_pages_are_used_again(exact):
     """A pool of 6 pages serves six sequences, one after the other and two at a time: what an ended session left in its pages
     (of every layer run) must not reach the next one."""
-    layers = [layer(latent(heads=2, dim=16, vdim=16, kv_rank=32, rot=8, scale=1.0), moe()), layer(latent(heads=3, kv_rank=64, rot=4, scale=1.0))]
+    # every expert chosen: bf16 attention must not meet a close choice
+    layers = [layer(latent(heads=2, dim=16, vdim=16, kv_rank=32, rot=8, scale=1.0), moe(experts=3, top=3)),
+              layer(latent(heads=3, kv_rank=64, rot=4, scale=1.0))]
     spec, w = make(layers, seed=17, loop=(0, 1, 3))
     tol = TOL if exact else TOL16
     eng = engine(spec, w, max_batch=2, max_sessions=2, num_pages=6, max_context=384, max_batched_tokens=384, debug_logit_rows=384,
@@ -402,7 +404,8 @@ def test_latent_attention_on_tensor_cores(heads, rank, rot, dim, vdim, sharp):
 def test_unequal_requests_on_tensor_cores():
     """Portions of several requests in one step (query tiles of 64 tokens that start anywhere in a page, partly filled ones, a
     later one of the same step that sees another request's pages nowhere) beside single tokens of others."""
-    layers = [layer(latent(heads=6, dim=32, vdim=32, kv_rank=64, rot=16, scale=0.5), moe(ff=64, shared=64)), layer(latent(heads=3, dim=32, vdim=64, kv_rank=96, rot=8))]
+    layers = [layer(latent(heads=6, dim=32, vdim=32, kv_rank=64, rot=16, scale=0.5), moe(ff=64, experts=4, top=4, shared=64)),
+              layer(latent(heads=3, dim=32, vdim=64, kv_rank=96, rot=8))]
     spec, w = make(layers, width=128, vocab=128, seed=47, loop=(0, 2, 2))
     eng = engine(spec, w, exact_f32=False, num_pages=24, max_batched_tokens=704, debug_logit_rows=704)
     try:
