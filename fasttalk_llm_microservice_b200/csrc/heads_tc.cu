@@ -129,19 +129,25 @@ __global__ void __launch_bounds__(HT_THREADS) linear_heads_kernel(LinearArgs a, 
             const uint32_t lanes = tmem + ((uint32_t)((warp & 3) * 32) << 16);
             for (int c = (warp >> 2) * 16; c < NT; c += 32) {
                 if (t0 + c >= a.M) break;                              // uniform
-                float v[16];
+                const int nt = min(16, a.M - t0 - c);
+                const size_t col = (size_t)p * a.c_col_stride + f;
+                float v[16], g[16];
+                if (a.gate && f < a.N) {                               // all of them on the way before the first is used
+                    const float* gp = a.gate + (size_t)(t0 + c) * a.ldg + col;
+#pragma unroll
+                    for (int i = 0; i < 16; ++i) g[i] = i < nt ? gp[(size_t)i * a.ldg] : 0.f;
+                }
+                __syncwarp();
                 tmem_ld16(lanes + c, v);
                 if (f < a.N) {
+                    if (a.gate) {
 #pragma unroll
-                    for (int i = 0; i < 16; ++i) {
-                        const int t = t0 + c + i;
-                        if (t < a.M) {
-                            const size_t col = (size_t)p * a.c_col_stride + f;
-                            float y = v[i];
-                            if (a.gate) y *= 1.f / (1.f + expf(-a.gate[(size_t)t * a.ldg + col]));
-                            a.C[(size_t)t * a.ldc + col] = y;
-                        }
+                        for (int i = 0; i < 16; ++i) v[i] *= 1.f / (1.f + expf(-g[i]));
                     }
+                    float* cp = a.C + (size_t)(t0 + c) * a.ldc + col;
+#pragma unroll
+                    for (int i = 0; i < 16; ++i)
+                        if (i < nt) cp[(size_t)i * a.ldc] = v[i];
                 }
                 __syncwarp();
             }
