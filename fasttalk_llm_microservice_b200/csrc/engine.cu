@@ -953,16 +953,19 @@ static int forward_layered(Engine* e, const Batch& b) {
             const int R = c.rot_dims, kd = c.kv_rank + R, hd = c.dim + R;
             LatentArgs la;
             la.proj = L.proj; la.ldp = ld; la.o_q = c.o_q; la.o_dkv = c.o_dkv; la.o_gate = c.gate_wide ? -1 : c.o_gate;
-            la.norm_w = c.dkv_norm; la.eps = M.eps; la.rot_freq = c.rot_freq; la.sink = c.sink; la.qlat = L.b1; la.out = L.b2;
-            la.cache = L.lat_cache ? L.lat_cache + ll.cache_off : nullptr;
+            la.norm_w = c.dkv_norm; la.eps = M.eps; la.rot_freq = c.rot_freq; la.sink = c.sink; la.out = L.b2;
             la.cache16 = L.lat_cache16 && latent_attn_mma_ok(c.kv_rank, R) ? (uint8_t*)L.lat_cache16 + ll.cache16_off * 2 : nullptr;
+            // one work buffer holds the queries in the form the attention reads
+            if (la.cache16) la.qlat16 = (__nv_bfloat16*)L.b1;
+            else { la.cache = L.lat_cache + ll.cache_off; la.qlat = L.b1; }
             la.part = L.attn_part; la.positions = d + m.o_pos; la.seq_rows = d + m.o_rows; la.page_table = d + m.o_pt;
             la.max_pages = e->max_pages; la.H = c.heads; la.dim = c.dim; la.rank = c.kv_rank; la.rot = R; la.scale = c.scale;
             FT_TRY(launch_latent_prep(la, T, st));
             LinearArgs a;                   // plain query parts into latent space, head by head: qlat_h = W_uk_h^T q_h
             a.A = L.proj + c.o_q; a.lda = ld; a.a_col_stride = hd;
             a.W = (const __nv_bfloat16*)c.w_uk_t; a.w_stride = (long long)c.kv_rank * c.dim; a.ldw = c.dim;
-            a.C = L.b1; a.ldc = c.heads * kd; a.c_col_stride = kd;
+            a.c_col_stride = la.qlat16 ? latent_row16(c.kv_rank, R) : kd;
+            a.C = la.qlat; a.C16 = la.qlat16; a.c16_scale = c.scale; a.ldc = c.heads * a.c_col_stride;
             a.M = T; a.N = c.kv_rank; a.K = c.dim; a.P = c.heads;
             FT_TRY(heads(e, a));
             // prompt portions on tcgen05, single tokens of running sequences (and steps of a few portion tokens) row by row

@@ -110,6 +110,8 @@ struct LinearArgs {
     float cap = 0.f;
     const float* gate = nullptr;
     int ldg = 0;
+    __nv_bfloat16* C16 = nullptr;                 // the result as bf16(C * c16_scale) instead (plain epilogue; C is not written)
+    float c16_scale = 1.f;
 };
 // rows_bound: M when batched; an upper bound of seg[P] when grouped
 int launch_linear(const LinearArgs& a, int rows_bound, cudaStream_t stream);
@@ -140,7 +142,8 @@ struct LatentArgs {
     float eps = 0.f;
     const float* rot_freq = nullptr;              // [rot / 2]
     const float* sink = nullptr;                  // [H] or null: exp(sink) joins the softmax denominator
-    float* qlat = nullptr;                        // [T][H][rank + rot]
+    float* qlat = nullptr;                        // [T][H][rank + rot] fp32, read with `cache`
+    __nv_bfloat16* qlat16 = nullptr;              // [T][H][latent_row16]: bf16(query * scale), zeros behind; read with `cache16`
     float* cache = nullptr;                       // this layer's [pages][64][rank + rot] fp32, or null
     void* cache16 = nullptr;                      // this layer's bf16 pages (latent_row16), or null
     float* out = nullptr;                         // [T][H][rank] attended latents
@@ -149,7 +152,7 @@ struct LatentArgs {
     int max_pages = 0, H = 0, dim = 0, rank = 0, rot = 0;
     float scale = 1.f;
 };
-// Latent normed, shared key part rotated -> the caches; the rotated part of every query -> qlat.
+// Latent normed, shared key part rotated -> the caches; the rotated part of every query -> qlat or qlat16.
 int launch_latent_prep(const LatentArgs& a, int T, cudaStream_t stream);
 // With fewer than kLatentSplitPairs (token, head) pairs in a step the keys of each are cut into up to kLatentMaxSplits
 // shares that run side by side; `part` then holds pairs x shares x (rank + 2) floats (null: never split).

@@ -144,10 +144,16 @@ __global__ void __launch_bounds__(HT_THREADS) linear_heads_kernel(LinearArgs a, 
 #pragma unroll
                         for (int i = 0; i < 16; ++i) v[i] *= 1.f / (1.f + expf(-g[i]));
                     }
-                    float* cp = a.C + (size_t)(t0 + c) * a.ldc + col;
+                    const size_t at = (size_t)(t0 + c) * a.ldc + col;
+                    if (a.C16) {
 #pragma unroll
-                    for (int i = 0; i < 16; ++i)
-                        if (i < nt) cp[(size_t)i * a.ldc] = v[i];
+                        for (int i = 0; i < 16; ++i)
+                            if (i < nt) a.C16[at + (size_t)i * a.ldc] = __float2bfloat16_rn(v[i] * a.c16_scale);
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 16; ++i)
+                            if (i < nt) a.C[at + (size_t)i * a.ldc] = v[i];
+                    }
                 }
                 __syncwarp();
             }

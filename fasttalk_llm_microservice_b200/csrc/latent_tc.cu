@@ -8,7 +8,7 @@
 // K-major 128-byte-swizzled operand of the scores and, block by block, the MN-major one of the values — ONE bulk copy per page,
 // one array in shared memory for both products.
 //
-//   S  = Q C^T   tcgen05.mma  M128 N64, K in steps of 16 over all columns.  Q sits in TENSOR MEMORY as far as there is room (4 or
+//   S  = Q C^T   tcgen05.mma  M128 N64, over all columns.  Q sits in TENSOR MEMORY as far as there is room (4 or
 //                8 blocks of 64 columns): with both operands in shared memory an M128 N64 product asks for more than the port's
 //                128 B/clk.  Further blocks lie in shared memory.
 //   softmax      4 warps, one thread per row, running maximum and sum in fp32, exp2; the rescale of O is lazy (the reference
@@ -35,17 +35,18 @@ constexpr int LT_MAX_STAGES = 6;
 constexpr int LT_COL_O = 0, LT_COL_S = 256, LT_COL_Q = 384, LT_COL_Q2 = 128;
 constexpr float LT_RESCALE = 8.f;                      // log2 units
 constexpr int LT_SPIN = 1 << 20;
+constexpr float LOG2E = 1.4426950408889634f;
+constexpr int LT_OUT_LD = 36;                          // floats per row of a warp's output staging (32 columns)
 constexpr size_t LT_SMEM_MAX = 227 * 1024;
 
 struct LatentTcCfg {
-    int nblk, ksteps, tq, stages, nv, groups;          // 64-column blocks, K steps, blocks of Q in TMEM, ring, value columns per CTA
+    int nblk, tq, stages, nv, groups;                  // 64-column blocks, blocks of Q in TMEM, ring, value columns per CTA, groups of them
     size_t smem;
 };
 
 bool latent_tc_cfg(int rank, int rot, LatentTcCfg& c) {
     const int vblk = (rank + 63) / 64;
     c.nblk = latent_row16(rank, rot) / 64;
-    c.ksteps = (rank + rot + 15) / 16;
     c.groups = (vblk + 3) / 4;
     c.nv = (vblk + c.groups - 1) / c.groups * 64;
     c.tq = std::min(c.nblk, c.nv <= 128 ? 8 : 4);
@@ -74,12 +75,11 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
     uint8_t* kv_s = smem;                                              // [stages][nblk] slabs
     uint8_t* q_s = kv_s + (size_t)cfg.stages * page_bytes;             // blocks of Q that TMEM has no room for
     uint64_t* kv_full = reinterpret_cast<uint64_t*>(q_s + (size_t)(cfg.nblk - cfg.tq) * LT_QBLK);      // [6]
-    uint64_t* kv_empty = kv_full + LT_MAX_STAGES;                      // [6]
+    uint64_t* kv_empty = kv_full + LT_MAX_STAGES;                      // [6] the products of the page have retired: O holds its share
     uint64_t* q_full = kv_empty + LT_MAX_STAGES;
     uint64_t* s_full = q_full + 1;                                     // [2]
     uint64_t* p_full = s_full + 2;                                     // [2]
-    uint64_t* pv_done = p_full + 2;                                    // [2]
-    uint64_t* drain = pv_done + 2;
+    uint64_t* drain = p_full + 2;
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(drain + 1);
     volatile int* dead = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
@@ -102,7 +102,6 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
         for (int b = 0; b < 2; ++b) {
             mbar_init(&s_full[b], 1);
             mbar_init(&p_full[b], LT_ROWS / 32);
-            mbar_init(&pv_done[b], 1);
         }
         mbar_init(drain, 1);
         *dead = 0;
@@ -153,15 +152,19 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
             auto stage_at = [&](int j) { return kv_addr + (uint32_t)(j % cfg.stages) * page_bytes; };
             auto issue_qk = [&](int j) {
                 const uint32_t k_addr = stage_at(j), d = tmem + LT_COL_S + (j & 1) * 64;
-                for (int s = 0; s < cfg.ksteps; ++s) {
-                    const int blk = s >> 2, k = s & 3;
-                    const uint64_t b = umma_desc_k128(k_addr + blk * LT_SLAB) + 2 * k;
-                    if (blk < cfg.tq) {
-                        const uint32_t qa = tmem + (blk < 4 ? LT_COL_Q + 32 * blk : LT_COL_Q2 + 32 * (blk - 4)) + 8 * k;
-                        umma_f16_ts(d, qa, b, idesc_qk, s != 0);
-                    } else {
-                        umma_bf16(d, umma_desc_k128(q_addr + (blk - cfg.tq) * LT_QBLK) + 2 * k, b, idesc_qk, s != 0);
-                    }
+                uint64_t b = umma_desc_k128(k_addr);
+                uint32_t acc = 0;
+                // whole blocks: columns beyond the row's end are zeros on both sides.  Little besides the products in here: one
+                // thread issues them all
+                for (int blk = 0; blk < cfg.tq; ++blk, b += LT_SLAB >> 4) {
+                    const uint32_t qa = tmem + (blk < 4 ? LT_COL_Q : LT_COL_Q2 - 128) + 32 * blk;
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) { umma_f16_ts(d, qa + 8 * k, b + 2 * k, idesc_qk, acc); acc = 1; }
+                }
+                uint64_t qd = umma_desc_k128(q_addr);
+                for (int blk = cfg.tq; blk < cfg.nblk; ++blk, b += LT_SLAB >> 4, qd += LT_QBLK >> 4) {
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) umma_bf16(d, qd + 2 * k, b + 2 * k, idesc_qk, 1);
                 }
                 umma_commit(&s_full[j & 1]);
             };
@@ -172,18 +175,20 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
                 tc_fence_after();
                 if (ok) issue_qk(j);
             }
+            const bool ahead = cfg.stages >= 3;                        // page j + 2 does not wait for the products of page j
             for (int j = 0; j < n_tiles && ok; ++j) {
-                ok = wait_limited(&p_full[j & 1], (j >> 1) & 1, dead);      // P(j) written, S(j) consumed, O rescaled if needed
+                if (ahead && j + 2 < n_tiles) ok = wait_limited(&kv_full[(j + 2) % cfg.stages], ((j + 2) / cfg.stages) & 1, dead);
+                ok = ok && wait_limited(&p_full[j & 1], (j >> 1) & 1, dead);      // P(j) written, S(j) consumed, O rescaled if needed
                 if (!ok) break;
                 tc_fence_after();
                 const uint32_t p = tmem + LT_COL_S + (j & 1) * 64, v_addr = stage_at(j) + (v0 >> 6) * LT_SLAB;
+                const uint64_t vd = umma_desc_mn128(v_addr);
 #pragma unroll
                 for (int k = 0; k < kKvTile / 16; ++k)
-                    umma_f16_ts(tmem + LT_COL_O, p + 8 * k, umma_desc_mn128(v_addr + k * 2048), idesc_pv, (j | k) != 0);
-                umma_commit(&pv_done[j & 1]);
+                    umma_f16_ts(tmem + LT_COL_O, p + 8 * k, vd + k * (2048 >> 4), idesc_pv, (j | k) != 0);
                 umma_commit(&kv_empty[j % cfg.stages]);
                 if (j + 2 < n_tiles) {
-                    ok = wait_limited(&kv_full[(j + 2) % cfg.stages], ((j + 2) / cfg.stages) & 1, dead);
+                    if (!ahead) ok = wait_limited(&kv_full[(j + 2) % cfg.stages], ((j + 2) / cfg.stages) & 1, dead);
                     tc_fence_after();
                     if (ok) issue_qk(j + 2);                           // behind the product that reads P out of this buffer
                 }
@@ -199,42 +204,27 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
         const int pair = first + row, tok = pair / a.H, head = pair % a.H;
         const bool valid = tok < ntok;
         const int pos = valid ? p0 + tok : p0 + last_tok;
-        const int kd = a.rank + a.rot;
         const uint32_t lanes = tmem + ((uint32_t)(quarter * 32) << 16);
-        const float to_log2 = a.scale * 1.4426950408889634f;
-        const float* q = a.qlat + ((size_t)row0 * a.H + first + row) * kd;
-        const bool vec = (kd & 3) == 0;
-        for (int blk = 0; blk < cfg.nblk; ++blk) {
+        const uint4* q = reinterpret_cast<const uint4*>(a.qlat16 + ((size_t)row0 * a.H + pair) * (cfg.nblk * 64));
+        constexpr int QB = 5;                                          // blocks of a row on their way at a time
+        for (int b0 = 0; b0 < cfg.nblk; b0 += QB) {
+            uint4 v[QB][8];
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                uint32_t pk[16];
+            for (int i = 0; i < QB; ++i)
 #pragma unroll
-                for (int e4 = 0; e4 < 8; ++e4) {
-                    const int c = blk * 64 + half * 32 + 4 * e4;
-                    float v[4] = {0.f, 0.f, 0.f, 0.f};
-                    if (valid) {
-                        if (vec) {
-                            if (c < kd) {
-                                const float4 t = *reinterpret_cast<const float4*>(q + c);
-                                v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
-                            }
-                        } else {
+                for (int ch = 0; ch < 8; ++ch) v[i][ch] = valid && b0 + i < cfg.nblk ? q[(b0 + i) * 8 + ch] : make_uint4(0u, 0u, 0u, 0u);
+            __syncwarp();
 #pragma unroll
-                            for (int i = 0; i < 4; ++i) if (c + i < kd) v[i] = q[c + i];
-                        }
-                    }
-                    pk[2 * e4] = pack_bf16(v[0] * to_log2, v[1] * to_log2);
-                    pk[2 * e4 + 1] = pack_bf16(v[2] * to_log2, v[3] * to_log2);
-                }
-                __syncwarp();
+            for (int i = 0; i < QB; ++i) {
+                const int blk = b0 + i;
                 if (blk < cfg.tq) {
-                    tmem_st16(lanes + (blk < 4 ? LT_COL_Q + 32 * blk : LT_COL_Q2 + 32 * (blk - 4)) + 16 * half, pk);
-                } else {
+                    const uint32_t dst = lanes + (blk < 4 ? LT_COL_Q : LT_COL_Q2 - 128) + 32 * blk;
+                    tmem_st16(dst, &v[i][0].x);
+                    tmem_st16(dst + 16, &v[i][4].x);
+                } else if (blk < cfg.nblk) {
                     uint8_t* dst = q_s + (size_t)(blk - cfg.tq) * LT_QBLK + row * 128;
 #pragma unroll
-                    for (int ch = 0; ch < 4; ++ch)
-                        *reinterpret_cast<uint4*>(dst + (((half * 4 + ch) ^ (row & 7)) << 4)) =
-                            make_uint4(pk[4 * ch], pk[4 * ch + 1], pk[4 * ch + 2], pk[4 * ch + 3]);
+                    for (int ch = 0; ch < 8; ++ch) *reinterpret_cast<uint4*>(dst + ((ch ^ (row & 7)) << 4)) = v[i][ch];
                 }
             }
         }
@@ -267,11 +257,11 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
 #pragma unroll
                 for (int c = 0; c < 64; ++c) t4[c & 3] = fmaxf(t4[c & 3], __uint_as_float(sr[c]));
             }
-            const float m_new = fmaxf(m_ref, fmaxf(fmaxf(t4[0], t4[1]), fmaxf(t4[2], t4[3])));
+            const float m_new = fmaxf(m_ref, fmaxf(fmaxf(t4[0], t4[1]), fmaxf(t4[2], t4[3])) * LOG2E);
             if (j == 0) {
                 m_ref = m_new;                                         // finite: position 0 is visible to every row
             } else if (__any_sync(0xffffffffu, m_new > m_ref + LT_RESCALE)) {      // tcgen05.ld / st move whole warps
-                ok = __all_sync(0xffffffffu, wait_limited(&pv_done[(j - 1) & 1], ((j - 1) >> 1) & 1, dead));
+                ok = __all_sync(0xffffffffu, wait_limited(&kv_empty[(j - 1) % cfg.stages], ((j - 1) / cfg.stages) & 1, dead));
                 if (!ok) break;
                 tc_fence_after();
                 const float alpha = exp2f(m_ref - m_new);
@@ -293,8 +283,8 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
                 uint32_t pk[16];
 #pragma unroll
                 for (int e = 0; e < 16; ++e) {
-                    const float x = ex2_fast(__uint_as_float(sr[half * 32 + 2 * e]) - m_ref);
-                    const float y = ex2_fast(__uint_as_float(sr[half * 32 + 2 * e + 1]) - m_ref);
+                    const float x = ex2_fast(fmaf(__uint_as_float(sr[half * 32 + 2 * e]), LOG2E, -m_ref));
+                    const float y = ex2_fast(fmaf(__uint_as_float(sr[half * 32 + 2 * e + 1]), LOG2E, -m_ref));
                     ps[(2 * e) & 3] += x;
                     ps[(2 * e + 1) & 3] += y;
                     pk[e] = pack_bf16(x, y);
@@ -307,39 +297,37 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
             __syncwarp();
             if (lane == 0) mbar_arrive(&p_full[j & 1]);
         }
-        if (ok) ok = __all_sync(0xffffffffu, wait_limited(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, dead));
+        if (ok) ok = __all_sync(0xffffffffu, wait_limited(&kv_empty[(n_tiles - 1) % cfg.stages], ((n_tiles - 1) / cfg.stages) & 1, dead));
         if (ok) {
             tc_fence_after();
             float f = 1.f;
             if (a.sink && valid) {                                     // relative to the larger of maximum and sink
-                const float s = a.sink[head] * 1.4426950408889634f, top = fmaxf(m_ref, s);
+                const float s = a.sink[head] * LOG2E, top = fmaxf(m_ref, s);
                 f = exp2f(m_ref - top);
                 l_run = l_run * f + exp2f(s - top);
             }
             if (a.o_gate >= 0 && valid) f *= 1.f / (1.f + expf(-a.proj[(size_t)(row0 + tok) * a.ldp + a.o_gate + head]));
             f /= l_run;
-            float* out = a.out + ((size_t)row0 * a.H + first + row) * a.rank;
-            const bool vec_o = (a.rank & 3) == 0;
-            for (int c = 0; c < nv && v0 + c < a.rank; c += 16) {
-                uint32_t o[16];
-                __syncwarp();
+            // 32 columns at a time through shared memory (the ring is idle now), so that a store covers whole 128-byte runs
+            float* stage = reinterpret_cast<float*>(kv_s) + quarter * 32 * LT_OUT_LD;
+            float* out = a.out + ((size_t)row0 * a.H + first + quarter * 32) * a.rank + v0;
+            const int rows = min(32, ntok * a.H - first - quarter * 32);      // valid rows of this warp (may be <= 0)
+            for (int c = 0; c < nv && v0 + c < a.rank; c += 32) {
+                uint32_t o[32];
                 tmem_ld16_nowait(lanes + LT_COL_O + c, o);
+                tmem_ld16_nowait(lanes + LT_COL_O + c + 16, o + 16);
                 tmem_ld_wait();
-                if (valid) {
 #pragma unroll
-                    for (int k = 0; k < 16; k += 4) {
-                        const int col = v0 + c + k;
-                        float v[4];
+                for (int k = 0; k < 32; k += 4)
+                    *reinterpret_cast<float4*>(stage + lane * LT_OUT_LD + k) =
+                        make_float4(__uint_as_float(o[k]) * f, __uint_as_float(o[k + 1]) * f, __uint_as_float(o[k + 2]) * f, __uint_as_float(o[k + 3]) * f);
+                __syncwarp();
 #pragma unroll
-                        for (int i = 0; i < 4; ++i) v[i] = __uint_as_float(o[k + i]) * f;
-                        if (vec_o) {
-                            if (col < a.rank) *reinterpret_cast<float4*>(out + col) = make_float4(v[0], v[1], v[2], v[3]);
-                        } else {
-#pragma unroll
-                            for (int i = 0; i < 4; ++i) if (col + i < a.rank) out[col + i] = v[i];
-                        }
-                    }
+                for (int r0 = 0; r0 < 32; r0 += 4) {
+                    const int r = r0 + (lane >> 3), k = (lane & 7) * 4;
+                    if (r < rows) *reinterpret_cast<float4*>(out + (size_t)r * a.rank + c + k) = *reinterpret_cast<const float4*>(stage + r * LT_OUT_LD + k);
                 }
+                __syncwarp();
             }
         }
     }
@@ -361,7 +349,7 @@ bool latent_prefill_tc_ok(int rank, int rot) {
 
 int launch_latent_prefill_tc(const LatentArgs& a, const WindowTiles& tm, int* err, cudaStream_t stream) {
     LatentTcCfg c;
-    FT_REQUIRE(a.cache16 && latent_tc_cfg(a.rank, a.rot, c), "latent attention (tcgen05): sizes %d + %d do not fit", a.rank, a.rot);
+    FT_REQUIRE(a.cache16 && a.qlat16 && a.rank % 32 == 0 && latent_tc_cfg(a.rank, a.rot, c), "latent attention (tcgen05): sizes %d + %d do not fit", a.rank, a.rot);
     static PerDeviceFlag attr;
     if (!attr.done()) {
         FT_CHECK_CUDA(cudaFuncSetAttribute(latent_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LT_SMEM_MAX));

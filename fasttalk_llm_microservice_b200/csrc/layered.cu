@@ -167,7 +167,8 @@ __global__ void __launch_bounds__(LTHREADS) linear_tile_kernel(LinearArgs a) {
                     if (a.epi == LIN_SOFTCAP) v = a.cap * tanhf(v / a.cap);
                     else if (a.epi == LIN_RELU2) { v = fmaxf(v, 0.f); v *= v; }
                     if (a.gate) v *= sigmoid_exact(a.gate[(size_t)r * a.ldg + (size_t)p * a.c_col_stride + n]);
-                    C[(size_t)r * a.ldc + n] = v;
+                    if (a.C16) a.C16[(size_t)r * a.ldc + (size_t)p * a.c_col_stride + n] = __float2bfloat16_rn(v * a.c16_scale);
+                    else C[(size_t)r * a.ldc + n] = v;
                 }
             }
         }
@@ -278,7 +279,10 @@ __global__ void __launch_bounds__(LWARPS * 32) linear_rows_kernel(LinearArgs a) 
                     if (a.gate && lane == 0 && col0 + c < cols)
                         v *= sigmoid_exact(a.gate[(size_t)(rb + i) * a.ldg + (size_t)p * a.c_col_stride + col0 + c]);
                 }
-                if (lane == 0 && col0 + c < cols) C[(size_t)(rb + i) * a.ldc + col0 + c] = v;
+                if (lane == 0 && col0 + c < cols) {
+                    if (a.C16) a.C16[(size_t)(rb + i) * a.ldc + (size_t)p * a.c_col_stride + col0 + c] = __float2bfloat16_rn(v * a.c16_scale);
+                    else C[(size_t)(rb + i) * a.ldc + col0 + c] = v;
+                }
             }
         }
     }
@@ -514,10 +518,20 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentArgs a, int row1
         const int h = j / half, i = j % half;
         const float* q = pr + a.o_q + h * hd + a.dim;
         const float u = q[i], v = q[half + i], cs = trig[i], sn = trig[half + i];
-        float* dst = a.qlat + ((size_t)t * a.H + h) * kd + rank;
-        dst[i] = u * cs - v * sn;
-        dst[half + i] = v * cs + u * sn;
+        const float x = u * cs - v * sn, y = v * cs + u * sn;
+        if (a.qlat16) {
+            __nv_bfloat16* dst = a.qlat16 + ((size_t)t * a.H + h) * row16 + rank;
+            dst[i] = __float2bfloat16_rn(x * a.scale);
+            dst[half + i] = __float2bfloat16_rn(y * a.scale);
+        } else {
+            float* dst = a.qlat + ((size_t)t * a.H + h) * kd + rank;
+            dst[i] = x;
+            dst[half + i] = y;
+        }
     }
+    if (a.qlat16 && kd < row16)
+        for (int j = threadIdx.x; j < a.H * (row16 - kd); j += blockDim.x)
+            a.qlat16[((size_t)t * a.H + j / (row16 - kd)) * row16 + kd + j % (row16 - kd)] = __float2bfloat16_rn(0.f);
 }
 
 // One warp per (token, head, key range): the query in latent space stays in registers (NR values per lane), keys = values =
@@ -650,7 +664,7 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, int n_s
 }
 
 int launch_latent_prep(const LatentArgs& a, int T, cudaStream_t stream) {
-    FT_REQUIRE(a.proj && a.norm_w && (a.cache || a.cache16) && (a.rot == 0 || (a.rot_freq && a.qlat && a.rot % 2 == 0)),
+    FT_REQUIRE(a.proj && a.norm_w && (a.cache || a.cache16) && (a.rot == 0 || (a.rot_freq && (a.qlat || a.qlat16) && a.rot % 2 == 0)),
                "latent prep: missing operands");
     latent_prep_kernel<<<T, 128, (size_t)a.rot * 4, stream>>>(a, latent_row16(a.rank, a.rot));
     FT_CHECK_CUDA(cudaGetLastError());
@@ -681,12 +695,13 @@ latent_attn_mma_kernel(LatentArgs a, int kc, int vc, int head_groups, int n_spli
     uint8_t* kbuf = lat_smem + TILE + (size_t)warp * 2 * TILE;
     const int t = blockIdx.x, split = blockIdx.y, h0 = (blockIdx.z % head_groups) * 16;
     const int v_first = (blockIdx.z / head_groups) * VC;   // first 32-column piece of the values this CTA sums
-    const int H = a.H, rank = a.rank, kd = a.rank + a.rot;
+    const int H = a.H, rank = a.rank;
     const __nv_bfloat16* cache16 = (const __nv_bfloat16*)a.cache16;
-    for (int idx = threadIdx.x; idx < 16 * row; idx += 128) {
-        const int r = idx / row, c = idx % row;
-        const float v = h0 + r < H && c < kd ? a.qlat[((size_t)t * H + h0 + r) * kd + c] * a.scale : 0.f;
-        *reinterpret_cast<__nv_bfloat16*>(Qs + r * RS + c * 2) = __float2bfloat16_rn(v);
+    for (int idx = threadIdx.x; idx < 16 * 4 * kc; idx += 128) {
+        const int r = idx / (4 * kc), ch = idx % (4 * kc);
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (h0 + r < H) v = *reinterpret_cast<const uint4*>(a.qlat16 + ((size_t)t * H + h0 + r) * row + ch * 8);
+        *reinterpret_cast<uint4*>(Qs + r * RS + ch * 16) = v;
     }
     __syncthreads();
     const int n_keys = a.positions[t] + 1;
@@ -844,6 +859,7 @@ int launch_latent_attn(const LatentArgs& a, int T, cudaStream_t stream) {
     const int n_pairs = T * a.H;
     const int n_split = a.part ? latent_attn_splits(T, a.H) : 1;
     if (a.cache16 && latent_attn_mma_ok(a.rank, a.rot)) {
+        FT_REQUIRE(a.qlat16, "latent attention: no bf16 queries");
         const int vc = (a.rank + 31) / 32, kc = latent_row16(a.rank, a.rot) / 32;
         const int groups = (vc + 7) / 8, per = (vc + groups - 1) / groups, hg = (a.H + 15) / 16;
         const dim3 grid(T, n_split, hg * groups);
@@ -865,7 +881,7 @@ int launch_latent_attn(const LatentArgs& a, int T, cudaStream_t stream) {
         }
 #undef FT_LATM
     } else {
-        FT_REQUIRE(a.cache, "latent attention: no fp32 cache");
+        FT_REQUIRE(a.cache && a.qlat, "latent attention: no fp32 cache or queries");
         const int kd = a.rank + a.rot;
         const dim3 grid((n_pairs + 3) / 4, n_split);
 #define FT_LAT(NR_, KB_) latent_attn_kernel<NR_, KB_><<<grid, 128, 0, stream>>>(a, n_pairs, n_split)
