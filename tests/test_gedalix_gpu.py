@@ -404,7 +404,7 @@ def test_latent_attention_on_tensor_cores(heads, rank, rot, dim, vdim, sharp):
 def test_unequal_requests_on_tensor_cores():
     """Portions of several requests in one step (query tiles of 64 tokens that start anywhere in a page, partly filled ones, a
     later one of the same step that sees another request's pages nowhere) beside single tokens of others."""
-    layers = [layer(latent(heads=6, dim=32, vdim=32, kv_rank=64, rot=16, scale=0.5), moe(ff=64, experts=4, top=4, shared=64)),
+    layers = [layer(latent(heads=5, dim=64, vdim=32, kv_rank=64, rot=24, scale=0.5), moe(ff=64, experts=4, top=4, shared=64)),
               layer(latent(heads=3, dim=32, vdim=64, kv_rank=96, rot=8))]
     spec, w = make(layers, width=128, vocab=128, seed=47, loop=(0, 2, 2))
     eng = engine(spec, w, exact_f32=False, num_pages=24, max_batched_tokens=704, debug_logit_rows=704)
