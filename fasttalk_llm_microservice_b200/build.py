@@ -41,6 +41,8 @@ def _digest() -> str:
         with open(os.path.join(CSRC, f), "rb") as fh:
             h.update(f.encode())
             h.update(fh.read())
+    with open(os.path.join(HERE, os.pardir, "include", "fasttalk_b200.h"), "rb") as fh:      # the descriptors' layout
+        h.update(fh.read())
     h.update(" ".join(NVCC_FLAGS).encode())
     return h.hexdigest()
 

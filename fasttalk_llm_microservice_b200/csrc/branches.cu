@@ -1,20 +1,19 @@
-// Kernels of the branch mixers and of the sandwich layer form (ft_branch_desc, FT_LAYER_SANDWICH).  Everything here is
+// Kernels of the branch mixers (ft_branch_desc).  Everything here is
 // fp32: positions and angles, scores and softmax, norms, gates, decays and the recurrent state; the projections that feed
 // these kernels come from the linear / tensor-core GEMMs of the layered family.
 //
-//   sandwich norm        x += rms(y) * post_gain;  hn = rms(x) * next_gain   (y = scaled sum of up to two branch results, or
-//                        the experts' weighted sum plus the shared expert): one kernel between any two GEMMs of a layer
 //   window attention     biases + rotary pairs, rotated keys and values into the paged cache; one CTA per (token, head),
 //                        its warps take key blocks of the window in turn (one key per lane for the scores, one value column
 //                        per lane for the sum), online softmax, merged through shared memory; prompt portions on a tiled
 //                        kernel.  Options, each off by default: queries and keys divided by their root mean square, a bias
 //                        by distance, first positions that stay visible beyond the window, a sink in the softmax denominator,
-//                        values mixed with those an earlier layer kept for the step, values that are columns of the keys
+//                        values mixed with those an earlier layer kept for the step, values that are columns of the keys, a
+//                        temperature that grows with the position, an element-wise gate on the result
 //   scalar-decay rule    S <- a_t S + b_t k_t v_t^T, o_t = S^T q_t for a request's tokens in order; one CTA per (request,
 //                        head, block of value columns), LPC lanes share a column and hold a run of key channels of its
 //                        state in registers.  Decay attention, the gated matrix memory and the state-space mixer all run
 //                        on it; they differ in how a, b, q, k, v are prepared and in the read-out that follows
-//   preparation          SiLU in place; gate pre-activations and the running-maximum scan of the matrix memory; short causal
+//   preparation          SiLU in place; rotation of q and k in place; gate pre-activations and the running-maximum scan of the matrix memory; short causal
 //                        convolution over a step's rows and the slot's tail, step sizes and decays of the state space
 //   read-out             normaliser, skip, gates and group-wise RMS norm, one CTA per (token, norm group)
 #include "common.cuh"
@@ -43,57 +42,6 @@ __device__ __forceinline__ float cta_sum(float v, float* red) {      // red: >= 
     return red[32];
 }
 
-__device__ __forceinline__ void put_planes(__nv_bfloat16* hi, __nv_bfloat16* lo, size_t i, float v) {
-    const __nv_bfloat16 h = __float2bfloat16_rn(v);
-    hi[i] = h;
-    lo[i] = __float2bfloat16_rn(v - __bfloat162float(h));
-}
-
-// ------------------------------------------------------------------ sandwich norm
-__global__ void __launch_bounds__(256) sandwich_norm_kernel(SandwichArgs a) {
-    __shared__ float red[33];
-    extern __shared__ float row[];
-    const int t = blockIdx.x, W = a.W;
-    float ss = 0.f;
-    for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        float y = 0.f;
-        if (a.y0) y = a.s0 * a.y0[(size_t)t * W + c];
-        if (a.y1) y = fmaf(a.s1, a.y1[(size_t)t * W + c], y);
-        if (a.top > 0) {
-            float f = 0.f;
-            for (int k = 0; k < a.top; ++k)
-                f = fmaf(a.wt[(size_t)t * a.top + k], a.eout[(size_t)a.slot_pos[(size_t)t * a.top + k] * W + c], f);
-            y += f;
-        }
-        row[c] = y;
-        ss += y * y;
-    }
-    ss = cta_sum(ss, red);
-    const float r1 = 1.f / sqrtf(ss / (float)W + a.eps);
-    float s2 = 0.f;
-    for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        const float v = a.x[(size_t)t * W + c] + row[c] * r1 * a.post_w[c];
-        a.x[(size_t)t * W + c] = v;
-        row[c] = v;
-        s2 += v * v;
-    }
-    s2 = cta_sum(s2, red);
-    const float r2 = 1.f / sqrtf(s2 / (float)W + a.eps);
-    __nv_bfloat16 *hi = (__nv_bfloat16*)a.hi, *lo = (__nv_bfloat16*)a.lo;
-    for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        const float v = row[c] * r2 * a.next_w[c];
-        a.hn[(size_t)t * W + c] = v;
-        if (hi) put_planes(hi, lo, (size_t)t * W + c, v);
-    }
-}
-
-int launch_sandwich_norm(const SandwichArgs& a, int T, cudaStream_t stream) {
-    FT_REQUIRE(a.x && a.hn && a.post_w && a.next_w && (a.y0 || a.y1 || a.top > 0), "sandwich norm: missing operands");
-    sandwich_norm_kernel<<<T, 256, (size_t)a.W * 4, stream>>>(a);
-    FT_CHECK_CUDA(cudaGetLastError());
-    return 0;
-}
-
 // ------------------------------------------------------------------ elementwise preparation
 // x[t][c0 .. c0 + n) <- silu(x) in place, rows of stride ld
 __global__ void silu_cols_kernel(float* __restrict__ x, int ld, int c0, int n) {
@@ -102,6 +50,32 @@ __global__ void silu_cols_kernel(float* __restrict__ x, int ld, int c0, int n) {
 }
 int launch_silu_cols(float* x, int ld, int c0, int n, int T, cudaStream_t stream) {
     silu_cols_kernel<<<T, 256, 0, stream>>>(x, ld, c0, n);
+    FT_CHECK_CUDA(cudaGetLastError());
+    return 0;
+}
+__global__ void turn_qk_kernel(TurnArgs a) {
+    const int t = blockIdx.x, half = a.rot_dims >> 1, per = half + a.dim - a.rot_dims;      // pairs, then single coordinates of a head
+    const float pos = (float)a.positions[t];
+    for (int i = threadIdx.x; i < (a.heads + a.kv_heads) * per; i += blockDim.x) {
+        const int hh = i / per, j = i % per;
+        const bool isq = hh < a.heads;
+        if (isq && j >= half) continue;                       // a query's other coordinates stay
+        float* x = a.proj + (size_t)t * a.ldp + (isq ? a.o_q + hh * a.dim : a.o_k + (hh - a.heads) * a.dim);
+        const float s = isq ? 1.f : a.k_scale;
+        if (j >= half) { x[a.rot_dims + j - half] *= s; continue; }
+        float sn, cs;
+        sincosf(pos * a.rot_freq[j], &sn, &cs);
+        float* p = x + (a.rot_half ? j : 2 * j);
+        float* q = x + (a.rot_half ? j + half : 2 * j + 1);
+        const float u = *p, v = *q;
+        *p = (u * cs - v * sn) * s;
+        *q = (v * cs + u * sn) * s;
+    }
+}
+int launch_turn_qk(const TurnArgs& a, int T, cudaStream_t stream) {
+    FT_REQUIRE(a.rot_dims >= 0 && a.rot_dims <= a.dim && (a.rot_dims & 1) == 0 && (a.rot_dims == 0 || a.rot_freq),
+               "rotation: bad sizes (dim %d, rotated %d)", a.dim, a.rot_dims);
+    turn_qk_kernel<<<T, 256, 0, stream>>>(a);
     FT_CHECK_CUDA(cudaGetLastError());
     return 0;
 }
@@ -183,10 +157,11 @@ __global__ void __launch_bounds__(128) window_write_kernel(WindowArgs a) {
         __syncthreads();
     }
     const RotSpec rs = {a.rot_freq, a.rot_dims, a.rot_half, a.rot_mag};
+    const float qt = a.temp_every > 0 ? fmaf(a.temp_coef, logf((float)((p + 1) / a.temp_every + 1)), 1.f) : 1.f;
     const bool wide = a.qk_norm == 2;             // gains per (head, coordinate) instead of per coordinate
     for (int i = threadIdx.x; i < nq; i += blockDim.x)
-        a.q_out[(size_t)t * nq + i] = rotated(pr + a.o_q, a.q_bias, a.q_gain, wide ? i - i % a.dim : 0, i, i % a.dim, rs, pos,
-                                              a.qk_norm ? inv[i / a.dim] : 1.f);
+        a.q_out[(size_t)t * nq + i] = qt * rotated(pr + a.o_q, a.q_bias, a.q_gain, wide ? i - i % a.dim : 0, i, i % a.dim, rs, pos,
+                                                   a.qk_norm ? inv[i / a.dim] : 1.f);
     if (a.no_kv) return;
     const int* pt = a.page_table + (size_t)a.seq_rows[t] * a.max_pages;
     const bool alias = a.v_in_key >= 0;                // the values are columns of the keys: the row holds the keys only
@@ -324,7 +299,9 @@ __global__ void __launch_bounds__(kWinWarps * 32) window_attn_kernel(WindowArgs 
     for (int c = threadIdx.x; c < a.vdim; c += blockDim.x) {
         float num = 0.f;
         for (int w = 0; w < kWinWarps; ++w) num += sacc[(size_t)w * a.vdim + c] * expf(sm[w] - mm);
-        a.out[((size_t)t * a.H + h) * a.vdim + c] = num / den;
+        float r = num / den;
+        if (a.gate) r *= sigmoid_f(a.gate[(size_t)t * a.ldg + h * a.vdim + c]);
+        a.out[((size_t)t * a.H + h) * a.vdim + c] = r;
     }
 }
 
@@ -517,6 +494,7 @@ __global__ void __launch_bounds__(WT_THREADS) window_tile_kernel(WindowArgs a, W
         if (row >= rows_used) continue;
         const float inv = cr[row];
         float* orow = a.out + ((size_t)(row_base + row / grp) * a.H + g * grp + row % grp) * a.vdim;
+        const float* gate = a.gate ? a.gate + (size_t)(row_base + row / grp) * a.ldg + (g * grp + row % grp) * a.vdim : nullptr;
 #pragma unroll
         for (int k = 0; k < VK; ++k) {
             const int col = 4 * ox + 128 * k;
@@ -524,6 +502,7 @@ __global__ void __launch_bounds__(WT_THREADS) window_tile_kernel(WindowArgs a, W
                 float o0, o1, o2, o3;
                 unpack2(acc[r][k][0], o0, o1);
                 unpack2(acc[r][k][1], o2, o3);
+                if (gate) { o0 *= sigmoid_f(gate[col]); o1 *= sigmoid_f(gate[col + 1]); o2 *= sigmoid_f(gate[col + 2]); o3 *= sigmoid_f(gate[col + 3]); }
                 *reinterpret_cast<float4*>(orow + col) = make_float4(o0 * inv, o1 * inv, o2 * inv, o3 * inv);
             }
         }
@@ -990,7 +969,7 @@ int launch_space_prep(const SpaceArgs& a, int T, int n_req, cudaStream_t stream)
 //   / (max(|o[t][h * vd + vdim] * q_scale|, floor[t][h]) + 1e-6)      with a normaliser
 //   + skip[h] * x[t][c]                                      with a skip
 //   * silu(gate[t][c])                                       gate_kind 1 (before the norm)
-// then divided by the root mean square of its group, times gain[c], times sigmoid(gate[t][c]) for gate_kind 2.
+// then divided by the root mean square of its group, times gain[c], times sigmoid (gate_kind 2) or silu (3) of gate[t][c].
 __device__ __forceinline__ float readout_value(const ReadoutArgs& a, int t, int c) {
     const int h = c / a.vdim, j = c % a.vdim;
     const float* orow = a.o + (size_t)t * a.ldo + (size_t)h * a.vd;
@@ -1017,8 +996,10 @@ __global__ void __launch_bounds__(256) readout_kernel(ReadoutArgs a) {
     const float rr = 1.f / sqrtf(ss / (float)n + a.eps);
     i = 0;
     for (int c = threadIdx.x; c < n; c += blockDim.x, ++i) {
-        float v = (i < kReadoutKeep ? keep[i] : readout_value(a, t, c0 + c)) * rr * a.gain[c0 + c];
+        float v = (i < kReadoutKeep ? keep[i] : readout_value(a, t, c0 + c)) * rr;
+        if (a.gain) v *= a.gain[c0 + c];
         if (a.gate_kind == 2) v *= sigmoid_f(a.gate[(size_t)t * a.ldg + c0 + c]);
+        else if (a.gate_kind == 3) v *= silu_f(a.gate[(size_t)t * a.ldg + c0 + c]);
         a.out[(size_t)t * a.heads * a.vdim + c0 + c] = v;
     }
 }
@@ -1028,21 +1009,6 @@ int launch_readout(const ReadoutArgs& a, int T, cudaStream_t stream) {
     const int n = a.heads * a.vdim / a.norm_groups;
     const int threads = n <= 64 ? 32 : n <= 256 ? 64 : n <= 1024 ? 128 : 256;
     readout_kernel<<<T * a.norm_groups, threads, 0, stream>>>(a);
-    FT_CHECK_CUDA(cudaGetLastError());
-    return 0;
-}
-
-// ------------------------------------------------------------------ activations between the two halves of a feed-forward
-// SwiGLU: gu [rows][2 ff] with columns (2j, 2j+1) = (gate_j, up_j) -> out [rows][ff]; squared ReLU: [rows][ff] -> [rows][ff]
-__global__ void ff_act_kernel(const float* __restrict__ in, float* __restrict__ out, size_t n, int act) {
-    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
-        if (act == FT_ACT_RELU2) { const float v = fmaxf(in[i], 0.f); out[i] = v * v; }
-        else { const float2 v = reinterpret_cast<const float2*>(in)[i]; out[i] = silu_f(v.x) * v.y; }
-    }
-}
-int launch_ff_act(const float* in, float* out, size_t n, int act, cudaStream_t stream) {
-    const int blocks = (int)std::min<size_t>((n + 255) / 256, 148 * 16);
-    ff_act_kernel<<<blocks, 256, 0, stream>>>(in, out, n, act);
     FT_CHECK_CUDA(cudaGetLastError());
     return 0;
 }

@@ -217,6 +217,9 @@ struct Layered {
     float* streams = nullptr;
     bool hyper = false;
     bool prenorm = false;
+    // sandwich models whose looped layers read [stream | embedding output]: rows of 2 * width, fp32 and as planes
+    float* cat = nullptr;
+    void *cat_hi = nullptr, *cat_lo = nullptr;
     float* trail = nullptr;            // debug: residual stream after every layer [n_layers][t_max][width]
     bool trail_on = false;
 };
@@ -619,6 +622,13 @@ static bool own_ff(const ft_layer_desc& c) {
     return c.form == FT_LAYER_SANDWICH || c.form == FT_LAYER_HYPER || c.form == FT_LAYER_PRENORM;
 }
 
+// The activation of a layer's feed-forward with its constants; bias: of a dense feed-forward's pairs.
+static GluSpec glu_of(const ft_layer_desc& c, int act, const float* bias) {
+    GluSpec g;
+    g.kind = act; g.limit = c.act_limit; g.alpha = c.act_alpha; g.shift = c.act_shift; g.bias = bias;
+    return g;
+}
+
 // The mixture of experts of one layer: routing from `logits` (row stride ldl, first column o_router), then every (token,
 // choice) pair through its expert, grouped by expert.  Reads the rows of L.hn; leaves the pairs' outputs in L.eout and their
 // weights / places in L.wts / L.slot_pos (the caller's residual kernel gathers them).
@@ -629,7 +639,8 @@ static int run_experts(Engine* e, const ft_layer_desc& c, const float* logits, i
     auto launched = [&](int n = 1) { e->st.kernel_launches += n; };
     const bool sandwich = own_ff(c);                                  // forms whose router is a matrix of its own
     const int act = sandwich ? c.ff_act : FT_ACT_SWIGLU;
-    const int n_up = act == FT_ACT_SWIGLU ? 2 * c.ff : c.ff;          // rows of an expert's first matrix
+    const int n_up = act == FT_ACT_RELU2 ? c.ff : 2 * c.ff;           // rows of an expert's first matrix
+    const GluSpec glu = glu_of(c, act, nullptr);
     const bool scaled_in = c.route_input != 0;                        // the experts read score * row, in sorted order
     const int top = c.top;
     FT_TRY(launch_route(logits, ldl, o_router, c.experts, c.top, sandwich ? 1 : c.groups, sandwich ? 1 : c.keep, L.ids, L.wts,
@@ -668,7 +679,7 @@ static int run_experts(Engine* e, const ft_layer_desc& c, const float* logits, i
             launched();
         }
         FT_TRY(join());
-        FT_TRY(launch_swiglu_planes(L.gu, L.ax_hi, L.ax_lo, (size_t)pairs * c.ff, st, act));
+        FT_TRY(launch_act_planes(L.gu, L.ax_hi, L.ax_lo, pairs, c.ff, act, glu, st));
         FT_CHECK_CUDA(cudaEventRecord(L.main_ready, st));
         for (int i = 0; i < Layered::kSide; ++i) FT_CHECK_CUDA(cudaStreamWaitEvent(L.side[i], L.main_ready, 0));
         k = 0;
@@ -691,7 +702,7 @@ static int run_experts(Engine* e, const ft_layer_desc& c, const float* logits, i
             gu.A = L.eout; gu.a_rows = nullptr;
         }
         gu.w_stride = (long long)n_up * W; gu.ldw = W; gu.C = L.act; gu.ldc = c.ff; gu.seg = L.seg;
-        gu.N = n_up; gu.K = W; gu.P = c.experts; gu.epi = act == FT_ACT_SWIGLU ? LIN_SWIGLU_PAIR : LIN_RELU2;
+        gu.N = n_up; gu.K = W; gu.P = c.experts; gu.epi = act == FT_ACT_RELU2 ? LIN_RELU2 : LIN_SWIGLU_PAIR; gu.glu = glu;
         FT_TRY(launch_linear(gu, T * top, st));
         LinearArgs dn;
         dn.A = L.act; dn.lda = c.ff; dn.W = (const __nv_bfloat16*)c.w_down; dn.w_stride = (long long)W * c.ff;
@@ -705,20 +716,20 @@ static int run_experts(Engine* e, const ft_layer_desc& c, const float* logits, i
 // out [T][width] = W_down act(W_up in) for every row: the dense feed-forward and the shared expert of a sandwich layer.
 // `in` is the normed stream L.hn (hi / lo: its planes when the step has them).
 static int run_mlp(Engine* e, const void* hi, const void* lo, const void* w_up, const void* w_down, int ff, int act, float* out,
-                   int T) {
+                   int T, const GluSpec& glu = GluSpec()) {
     Layered& L = *e->lay;
     const int W = L.m.width;
-    const int n_up = act == FT_ACT_SWIGLU ? 2 * ff : ff;
+    const int n_up = act == FT_ACT_RELU2 ? ff : 2 * ff;
     cudaStream_t st = e->stream;
     if (L.tensor && T >= kTensorMinRows && n_up % 128 == 0 && W % 64 == 0 && W % 128 == 0 && ff % 64 == 0) {
         FT_TRY(dense(e, L.hn, hi, lo, w_up, L.ffa, T, n_up, W));
-        FT_TRY(launch_swiglu_planes(L.ffa, L.ax_hi, L.ax_lo, (size_t)T * ff, st, act));
+        FT_TRY(launch_act_planes(L.ffa, L.ax_hi, L.ax_lo, T, ff, act, glu, st));
         e->st.kernel_launches++;
         return dense(e, nullptr, L.ax_hi, L.ax_lo, w_down, out, T, W, ff);
     }
     LinearArgs up;
     up.A = L.hn; up.lda = W; up.W = (const __nv_bfloat16*)w_up; up.ldw = W; up.C = L.ffb; up.ldc = ff; up.M = T; up.N = n_up;
-    up.K = W; up.epi = act == FT_ACT_SWIGLU ? LIN_SWIGLU_PAIR : LIN_RELU2;
+    up.K = W; up.epi = act == FT_ACT_RELU2 ? LIN_RELU2 : LIN_SWIGLU_PAIR; up.glu = glu;
     FT_TRY(launch_linear(up, T, st));
     e->st.kernel_launches++;
     return dense(e, L.ffb, nullptr, nullptr, w_down, out, T, W, ff);
@@ -766,6 +777,8 @@ static int run_branch(Engine* e, const Batch& b, const LayeredLayer& ll, int k, 
             a.q_bias = c.q_bias; a.k_bias = c.k_bias;
             a.G = c.kv_heads; a.dim = c.dim; a.vdim = c.vdim;
             a.qk_norm = c.qk_norm; a.eps = M.eps; a.keep_first = c.keep_first; a.sink = c.sink; a.rel = c.rel; a.rel_n = c.rel_n;
+            if (c.o_g >= 0) { a.gate = L.proj + c.o_g; a.ldg = ld; }
+            a.temp_coef = c.q_temp_coef; a.temp_every = c.q_temp_every;
             a.v_bias = c.v_bias; a.v_role = c.v_role; a.v_mix = c.v_mix; a.v_first = L.v_first;
         } else {
             // One shared key head: cached key [rotated part | normed latent], the value is its latent part.  The plain query
@@ -835,12 +848,23 @@ static int run_branch(Engine* e, const Batch& b, const LayeredLayer& ll, int k, 
         ReadoutArgs o;
         o.o = L.bo; o.vd = c.vdim; o.vdim = c.vdim; o.heads = c.heads; o.gain = c.out_norm; o.eps = M.eps; o.out = L.bfin;
         if (c.kind == FT_BRANCH_DECAY_ATTENTION) {
-            // q | k | v are adjacent columns of the projection: SiLU in place, then the rule reads them where they are
-            FT_TRY(launch_silu_cols(L.proj, ld, c.o_q, 2 * c.kv_heads * c.dim + c.heads * c.vdim, T, st));
+            // q | k | v are adjacent columns of the projection: SiLU or rotation in place, then the rule reads them where they are
+            if (!c.plain_qkv) {
+                FT_TRY(launch_silu_cols(L.proj, ld, c.o_q, 2 * c.kv_heads * c.dim + c.heads * c.vdim, T, st));
+                launched();
+            }
+            if (c.rot_dims > 0 || (c.k_scale != 0.f && c.k_scale != 1.f)) {
+                TurnArgs tq;
+                tq.proj = L.proj; tq.ldp = ld; tq.o_q = c.o_q; tq.o_k = c.o_k; tq.heads = c.heads; tq.kv_heads = c.kv_heads; tq.dim = c.dim;
+                tq.rot_dims = c.rot_dims; tq.rot_half = c.rot_half; tq.rot_freq = c.rot_freq; tq.k_scale = c.k_scale != 0.f ? c.k_scale : 1.f;
+                tq.positions = d + m.o_pos;
+                FT_TRY(launch_turn_qk(tq, T, st));
+                launched();
+            }
             FT_TRY(launch_const_decay(c.decay, L.ab, c.heads, T, st));
             r.q = L.proj + c.o_q; r.k = L.proj + c.o_k; r.v = L.proj + c.o_v; r.ldq = r.ldk = r.ldv = ld;
-            o.gate = L.proj + c.o_g; o.ldg = ld; o.gate_kind = 2; o.norm_groups = 1;
-            launched(2);
+            o.gate = L.proj + c.o_g; o.ldg = ld; o.gate_kind = c.gate_act ? 3 : 2; o.norm_groups = c.head_norm ? c.heads : 1;
+            launched();
         } else if (c.kind == FT_BRANCH_MATRIX_MEMORY) {
             MemoryArgs g;
             g.proj = L.proj; g.ldp = ld; g.o_v = c.o_v; g.o_i = c.o_i; g.o_f = c.o_f; g.gate_bias = c.gate_bias; g.cap = c.gate_cap;
@@ -901,6 +925,14 @@ static int forward_layered(Engine* e, const Batch& b) {
         p.embed_scale = M.embed_scale != 0.f ? M.embed_scale : 1.f;
         if (to) { p.re_embed = to->re_embed; p.pre_add = to->pre_add; }
     };
+    // what a sandwich joint leaves for the next reader: the stream ahead of layer run `to` (null: the head, or the same layer's
+    // feed-forward), normed by nw; ahead of a pass over looped layers the row [x | x0] instead
+    auto sandwich_next = [&](SandwichArgs& s, const ft_layer_desc* to, const float* nw) {
+        s.x = e->resid; s.W = W; s.eps = M.eps; s.hn = L.hn; s.hi = hn_hi; s.lo = hn_lo;
+        s.cat = L.cat; s.cat_hi = hn_hi ? L.cat_hi : nullptr; s.cat_lo = hn_hi ? L.cat_lo : nullptr;
+        if (to && to->pass_in) s.cat_x = 1;
+        else s.next_w = nw;
+    };
     if (L.prenorm) {
         PreNormArgs p;
         prenorm_next(p, &L.layers[0].d, L.layers[0].d.norm_pre1);
@@ -914,9 +946,14 @@ static int forward_layered(Engine* e, const Batch& b) {
         FT_TRY(launch_hyper_joint(h, T, st));
     } else if (L.postnorm)
         FT_TRY(launch_embed_scale(d + m.o_tokens, M.embed, M.embed_scale != 0.f ? M.embed_scale : 1.f, e->resid, L.hist, T, W, st));
-    else
-        FT_TRY(launch_embed_norm(d + m.o_tokens, M.embed, e->resid, L.hn, hn_hi, hn_lo, T, W, M.eps, L.layers[0].d.norm_gain,
-                                 L.layers[0].d.form == FT_LAYER_SANDWICH ? L.layers[0].d.norm_pre1 : nullptr, st));
+    else if (L.layers[0].d.form == FT_LAYER_SANDWICH) {
+        SandwichArgs s;
+        sandwich_next(s, &L.layers[0].d, L.layers[0].d.norm_pre1);
+        s.tokens = d + m.o_tokens; s.embed = M.embed; s.embed_scale = M.embed_scale != 0.f ? M.embed_scale : 1.f;
+        s.cat_x0 = L.cat != nullptr;
+        FT_TRY(launch_sandwich_joint(s, T, st));
+    } else
+        FT_TRY(launch_embed_norm(d + m.o_tokens, M.embed, e->resid, L.hn, hn_hi, hn_lo, T, W, M.eps, L.layers[0].d.norm_gain, nullptr, st));
     launched();
     // what the mixer of a post-norm layer reads: the stream plus its short convolution over time
     auto canon = [&](const LayeredLayer& ll) -> int {
@@ -936,6 +973,13 @@ static int forward_layered(Engine* e, const Batch& b) {
         const bool sandwich = c.form == FT_LAYER_SANDWICH;
         const int ld = c.n_in;              // row stride of this layer's projection outputs
         if (c.form == FT_LAYER_POSTNORM) FT_TRY(canon(ll));
+        if (c.pass_in) {                    // a pass over looped layers begins: x <- W [x; x0], then the layer's own norm
+            FT_TRY(dense(e, L.cat, hn_hi ? L.cat_hi : nullptr, hn_hi ? L.cat_lo : nullptr, c.pass_in, e->resid, T, W, 2 * W));
+            SandwichArgs s;
+            sandwich_next(s, nullptr, c.norm_pre1);
+            FT_TRY(launch_sandwich_joint(s, T, st));
+            launched();
+        }
         FT_TRY(dense(e, L.hn, hn_hi, hn_lo, c.w_in, L.proj, T, c.n_in, W));
         const float *y0 = L.mix, *y1 = nullptr;      // the mixer's result: s0 * y0 + s1 * y1, each [T][width]
         float s0 = 1.f, s1 = 1.f;
@@ -1144,18 +1188,18 @@ static int forward_layered(Engine* e, const Batch& b) {
         } else if (sandwich) {
             FT_REQUIRE(gain_next_w, "engine: layer %d: a sandwich layer needs per-coordinate gains in what follows it", l);
             SandwichArgs sa;
-            sa.x = e->resid; sa.hn = L.hn; sa.hi = hn_hi; sa.lo = hn_lo; sa.W = W; sa.eps = M.eps;
+            if (c.ff_kind != FT_FF_NONE) sandwich_next(sa, nullptr, c.norm_pre2);
+            else sandwich_next(sa, nx, gain_next_w);
             sa.y0 = y0; sa.s0 = s0; sa.y1 = y1; sa.s1 = s1; sa.post_w = c.norm_post1;
-            sa.next_w = c.ff_kind != FT_FF_NONE ? c.norm_pre2 : gain_next_w;
-            FT_TRY(launch_sandwich_norm(sa, T, st));
+            FT_TRY(launch_sandwich_joint(sa, T, st));
             launched();
             if (c.ff_kind != FT_FF_NONE) {
                 SandwichArgs sf;
-                sf.x = e->resid; sf.hn = L.hn; sf.hi = hn_hi; sf.lo = hn_lo; sf.W = W; sf.eps = M.eps;
-                sf.post_w = c.norm_post2; sf.next_w = gain_next_w;
+                sandwich_next(sf, nx, gain_next_w);
+                sf.post_w = c.norm_post2;
                 if (c.ff_kind == FT_FF_DENSE) {
-                    FT_TRY(run_mlp(e, hn_hi, hn_lo, c.w_gu, c.w_down, c.ff, c.ff_act, L.mix, T));
-                    sf.y0 = L.mix;
+                    FT_TRY(run_mlp(e, hn_hi, hn_lo, c.w_gu, c.w_down, c.ff, c.ff_act, L.mix, T, glu_of(c, c.ff_act, c.gu_bias)));
+                    sf.y0 = L.mix; sf.b0 = c.down_bias;
                 } else {
                     // router logits: fp32 accumulation over fp32 activations (CUDA cores), or over their bf16 hi + lo planes
                     // on the tensor cores when the step is large; the router's rows are padded to whole tiles for that
@@ -1164,11 +1208,11 @@ static int forward_layered(Engine* e, const Batch& b) {
                     FT_TRY(run_experts(e, c, L.rlog, ldl, 0, T));
                     sf.eout = L.eout; sf.wt = L.wts; sf.slot_pos = L.slot_pos; sf.top = c.top;
                     if (c.shared_ff > 0) {
-                        FT_TRY(run_mlp(e, hn_hi, hn_lo, c.w_shared_up, c.w_shared_down, c.shared_ff, c.ff_act, L.mix, T));
+                        FT_TRY(run_mlp(e, hn_hi, hn_lo, c.w_shared_up, c.w_shared_down, c.shared_ff, c.ff_act, L.mix, T, glu_of(c, c.ff_act, nullptr)));
                         sf.y0 = L.mix;
                     }
                 }
-                FT_TRY(launch_sandwich_norm(sf, T, st));
+                FT_TRY(launch_sandwich_joint(sf, T, st));
                 launched();
             }
         } else {
@@ -1722,7 +1766,7 @@ static int engine_init_layered(Engine* e) {
     size_t kv_floats = 0, br_q = 0, br_v = 0, br_o = 0, br_fin = 0, br_heads = 0, e_max_s = 1, scan_cn = 0;
     int n_in_max = 1, top_max = 1, heads_max = 1, rank_max = 0;
     size_t vfirst_cols = 0, lstage_cols = 0;
-    bool use_hist = false;
+    bool use_hist = false, has_pass = false;
     for (int l = 0; l < M.n_layers; ++l) {
         LayeredLayer& ll = L.layers[l];
         const ft_layer_desc& d = ll.d;
@@ -1765,6 +1809,10 @@ static int engine_init_layered(Engine* e) {
         } else {
             FT_REQUIRE(d.form == FT_LAYER_GATED && d.rg_bias && d.o_rg1 >= 0 && d.mixer != FT_MIXER_BRANCHES,
                        "engine: gated layer %d is incomplete (it takes latent attention or channel delta)", l);
+        }
+        if (d.pass_in) {
+            FT_REQUIRE(d.form == FT_LAYER_SANDWICH, "engine: layer %d: the projection ahead of a pass belongs to the sandwich form", l);
+            has_pass = true;
         }
         n_in_max = std::max(n_in_max, d.n_in);
         if (d.mixer != FT_MIXER_BRANCHES) {
@@ -1833,8 +1881,8 @@ static int engine_init_layered(Engine* e) {
                     lstage_cols = std::max(lstage_cols, (size_t)c.heads * kd + kd);
                     buf = std::max(buf, std::max((size_t)c.q_rank, (size_t)c.heads * (c.dim + c.rot_dims)));
                 } else if (c.kind == FT_BRANCH_DECAY_ATTENTION) {
-                    FT_REQUIRE(c.kv_heads == c.heads && c.decay && c.out_norm && c.o_v >= 0 && c.o_g >= 0 &&
-                                   c.o_k == c.o_q + c.heads * c.dim && c.o_v == c.o_k + c.heads * c.dim,
+                    FT_REQUIRE(c.kv_heads == c.heads && c.decay && (c.out_norm || c.head_norm) && c.o_v >= 0 && c.o_g >= 0 &&
+                                   (c.rot_dims == 0 || c.rot_freq) && c.o_k == c.o_q + c.heads * c.dim && c.o_v == c.o_k + c.heads * c.dim,
                                "engine: decay-attention layer %d branch %d is incomplete", l, k);
                     ll.br_s_off[k] = L.slot_stride;
                     L.slot_stride += (size_t)c.heads * c.dim * c.vdim;
@@ -1927,6 +1975,9 @@ static int engine_init_layered(Engine* e) {
             FT_REQUIRE(d.ff_kind == FT_FF_NONE, "engine: layer %d has an unknown feed-forward %d", l, d.ff_kind);
         }
     }
+    if (has_pass)
+        for (const LayeredLayer& ll : L.layers)
+            FT_REQUIRE(ll.d.form == FT_LAYER_SANDWICH, "engine: a model whose passes take the embedding output again has sandwich layers only");
     L.ld_proj = (n_in_max + 3) & ~3;
     L.tensor = M.exact_f32 == 0;
     L.top_max = top_max;
@@ -1961,6 +2012,13 @@ static int engine_init_layered(Engine* e) {
     if (vfirst_cols) FT_TRY(alloc(&L.v_first, T * vfirst_cols * 4));
     if (lstage_cols) FT_TRY(alloc(&L.lstage, T * lstage_cols * 4));
     if (L.postnorm) FT_TRY(alloc(&L.resid2, T * W * 4));
+    if (has_pass) {
+        FT_TRY(alloc(&L.cat, T * 2 * W * 4));
+        if (L.tensor) {
+            FT_TRY(alloc(&L.cat_hi, T * 2 * W * 2));
+            FT_TRY(alloc(&L.cat_lo, T * 2 * W * 2));
+        }
+    }
     if (L.hyper) FT_TRY(alloc(&L.streams, T * (size_t)std::max(M.streams, 1) * W * 4));
     FT_TRY(alloc(&L.ffa, T * act_cols * 2 * 4));
     FT_TRY(alloc(&L.ffb, T * act_cols * 4));
@@ -2039,6 +2097,7 @@ static void engine_free(Engine* e) {
         cudaFree(L.b3); cudaFree(L.b4); cudaFree(L.beta); cudaFree(L.attn_part); cudaFree(L.mix); cudaFree(L.act); cudaFree(L.eout);
         cudaFree(L.kv_cache); cudaFree(L.bq); cudaFree(L.bv); cudaFree(L.bo); cudaFree(L.bfin); cudaFree(L.ab); cudaFree(L.gates);
         cudaFree(L.hist); cudaFree(L.v_first); cudaFree(L.lstage); cudaFree(L.resid2); cudaFree(L.streams);
+        cudaFree(L.cat); cudaFree(L.cat_hi); cudaFree(L.cat_lo);
         cudaFree(L.floor); cudaFree(L.mix2); cudaFree(L.ffa); cudaFree(L.ffb); cudaFree(L.rlog);
         cudaFree(L.wts); cudaFree(L.xlast); cudaFree(L.ids); cudaFree(L.seg); cudaFree(L.slot_token);
         cudaFree(L.slot_pos); cudaFree(L.trail); cudaFree(L.pl_hi); cudaFree(L.pl_lo); cudaFree(L.hn_hi); cudaFree(L.hn_lo);

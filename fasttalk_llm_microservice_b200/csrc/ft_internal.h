@@ -89,12 +89,32 @@ int launch_attn_prefill_tc(const void* q, int q_rows, const void* kv_layer, cons
                            cudaStream_t stream);
 
 // ---- layered.cu (the layered model family: every size is a run-time value, activations fp32, weights bf16)
+// How a (gate, up) pair of a feed-forward becomes one number.  bias (may be null): added to the pairs first, paired like them.
+// kind FT_ACT_SWIGLU: silu(g) * u.  FT_ACT_CLIPPED_GLU: g <- min(g, limit), u <- clamp(u, -limit, limit), then
+// g * sigmoid(alpha * g) * (u + shift).
+struct GluSpec {
+    int kind = FT_ACT_SWIGLU;
+    float limit = 0.f, alpha = 0.f, shift = 0.f;
+    const float* bias = nullptr;
+};
+#ifdef __CUDACC__
+__device__ __forceinline__ float glu_value(const GluSpec& s, float g, float u, int j) {
+    if (s.bias) { g += s.bias[2 * j]; u += s.bias[2 * j + 1]; }
+    if (s.kind == FT_ACT_CLIPPED_GLU) {
+        g = fminf(g, s.limit);
+        u = fminf(fmaxf(u, -s.limit), s.limit);
+        return g / (1.f + expf(-s.alpha * g)) * (u + s.shift);
+    }
+    return g / (1.f + expf(-g)) * u;
+}
+#endif
 enum { LIN_PLAIN = 0, LIN_SWIGLU_PAIR = 1, LIN_SOFTCAP = 2, LIN_RELU2 = 3 };
 // C[r, n] = sum_k A[row(r), k] * W[p][n, k] for problems p = 0..P-1.
 //   batched (seg == null): every problem has rows 0..M-1; problem p reads A + p * a_col_stride, W + p * w_stride and
 //                          writes C + p * c_col_stride (heads side by side in the columns of one buffer)
 //   grouped (seg != null): problem p owns rows seg[p]..seg[p+1]-1 of C; row r reads A row a_rows[r] (or r)
 // LIN_SWIGLU_PAIR: W rows (2j, 2j+1) are (gate_j, up_j); C[r, j] = silu(gate) * up, ldc counts those N/2 columns.
+//                  (or what `glu` says: see GluSpec)
 // LIN_SOFTCAP:     C = cap * tanh(C / cap).
 // LIN_RELU2:       C = max(C, 0)^2.
 // gate (plain epilogue): C = C * sigmoid(gate[r * ldg + p * c_col_stride + n]), the gate's columns laid out as those of C.
@@ -112,6 +132,7 @@ struct LinearArgs {
     int ldg = 0;
     __nv_bfloat16* C16 = nullptr;                 // the result as bf16(C * c16_scale) instead (plain epilogue; C is not written)
     float c16_scale = 1.f;
+    GluSpec glu;                                  // LIN_SWIGLU_PAIR
 };
 // rows_bound: M when batched; an upper bound of seg[P] when grouped
 int launch_linear(const LinearArgs& a, int rows_bound, cudaStream_t stream);
@@ -126,8 +147,8 @@ int launch_embed_norm(const int* tokens, const void* embed, float* x, float* hn,
 int launch_to_planes(const float* x, void* hi, void* lo, size_t n, cudaStream_t stream);
 int launch_softcap(float* x, size_t n, float cap, cudaStream_t stream);
 int launch_gather_planes_rows(const float* src, const int* idx, void* hi, void* lo, int n, int W, cudaStream_t stream);
-// act FT_ACT_SWIGLU: gu holds (gate, up) pairs, n counts pairs; FT_ACT_RELU2: gu holds n plain values
-int launch_swiglu_planes(const float* gu, void* hi, void* lo, size_t n, cudaStream_t stream, int act = FT_ACT_SWIGLU);
+// bf16 planes of an activation, [rows][ff].  act FT_ACT_RELU2: gu holds plain values; otherwise (gate, up) pairs and glu says the rest
+int launch_act_planes(const float* gu, void* hi, void* lo, int rows, int ff, int act, const GluSpec& glu, cudaStream_t stream);
 int launch_combine_norm(float* x, float* hn, const float* proj, int ldp, int o_rg1, int o_rg2, const float* rg_bias,
                         const float* mix, const float* eout, const float* wt, const int* slot_pos, int top, int T, int W,
                         float eps, float gain, void* hi, void* lo, cudaStream_t stream);
@@ -197,9 +218,12 @@ int launch_route(const float* proj, int ldp, int o_router, int E, int top, int g
                  int* seg, int* slot_token, int* slot_pos, int T, cudaStream_t stream, int route_kind = FT_ROUTE_SOFTMAX,
                  int normalise = 0, float scale = 1.f, const float* bias = nullptr);
 
-// ---- branches.cu (branch mixers and the sandwich layer form: ft_branch_desc, FT_LAYER_SANDWICH; everything fp32)
-// x += rms(y) * post_w;  hn = rms(x) * next_w  with  y = s0 * y0 + s1 * y1 + sum_k wt[t, k] * eout[slot_pos[t, k]]
-// (each of the three parts optional); hi / lo (may be null): hn once more as bf16 planes.
+// ---- sandwich.cu (FT_LAYER_SANDWICH: the joint between two sublayers)
+// One CTA per row.  With `tokens`: x = embed[token] * embed_scale (a step's first joint).  With any of the parts of y:
+//   x += rms(y) * post_w,   y = s0 * y0 + b0 + s1 * y1 + sum_k wt[t, k] * eout[slot_pos[t, k]]   (each part optional)
+// otherwise x stays.  Then hn = rms(x) * next_w with its bf16 planes (hi / lo may be null; next_w null: neither is formed).
+// cat (rows [x | x0] of 2 W, with planes cat_hi / cat_lo when given): cat_x writes the stream into the first half, cat_x0 the
+// embedding output into the second (a step's first joint).
 struct SandwichArgs {
     float* x = nullptr;
     float* hn = nullptr;
@@ -213,11 +237,29 @@ struct SandwichArgs {
     const float *post_w = nullptr, *next_w = nullptr;
     int W = 0;
     float eps = 0.f;
+    const float* b0 = nullptr;
+    const int* tokens = nullptr;
+    const void* embed = nullptr;
+    float embed_scale = 1.f;
+    float* cat = nullptr;
+    void *cat_hi = nullptr, *cat_lo = nullptr;
+    int cat_x = 0, cat_x0 = 0;
 };
-int launch_sandwich_norm(const SandwichArgs& a, int T, cudaStream_t stream);
+int launch_sandwich_joint(const SandwichArgs& a, int T, cudaStream_t stream);
+
+// ---- branches.cu (branch mixers: ft_branch_desc; everything fp32)
+// q (heads x dim at o_q) and k (at o_k) of the projection in place: rotation of the first rot_dims coordinates of a head (pairs
+// (2i, 2i + 1), or (i, i + rot_dims / 2) with rot_half), then k times k_scale
+struct TurnArgs {
+    float* proj = nullptr;
+    int ldp = 0, o_q = 0, o_k = 0, heads = 0, kv_heads = 0, dim = 0, rot_dims = 0, rot_half = 0;
+    const float* rot_freq = nullptr;
+    float k_scale = 1.f;
+    const int* positions = nullptr;
+};
+int launch_turn_qk(const TurnArgs& a, int T, cudaStream_t stream);
 int launch_silu_cols(float* x, int ld, int c0, int n, int T, cudaStream_t stream);
 int launch_const_decay(const float* decay, float* ab, int heads, int T, cudaStream_t stream);
-int launch_ff_act(const float* in, float* out, size_t n, int act, cudaStream_t stream);
 
 // Softmax attention over the last `window` positions (0 = all) of a paged cache whose rows hold, per position,
 // [G * dim rotated keys | G * vdim values].  launch_window_attention writes the step's rows first, then attends.
@@ -253,6 +295,10 @@ struct WindowArgs {
     float rot_mag = 1.f;                          // factor on cos and sin
     int chunked = 0;                              // position p sees the keys from (p / window) * window on, not the last `window`
     int no_kv = 0;                                // the cache belongs to another layer, which has written the step's rows: queries only
+    const float* gate = nullptr;                  // rows of stride ldg, H * vdim numbers: out *= sigmoid(gate)
+    int ldg = 0;
+    float temp_coef = 0.f;                        // q *= 1 + temp_coef * ln(1 + floor((p + 1) / temp_every)); temp_every 0: no
+    int temp_every = 0;
 };
 // The step's prompt portions as the batch builder lists them: 64-token query tiles (request, first token), and per request
 // its first row in the step, its page-table row and the position of its first token.
@@ -323,9 +369,9 @@ struct ReadoutArgs {
     const float* x = nullptr;
     int ldx = 0;
     const float* gate = nullptr;                  // rows of stride ldg
-    int ldg = 0, gate_kind = 0;                   // 0 none, 1 silu before the norm, 2 sigmoid after it
+    int ldg = 0, gate_kind = 0;                   // 0 none, 1 silu before the norm, 2 sigmoid after it, 3 silu after it
     int norm_groups = 1;
-    const float* gain = nullptr;                  // [heads * vdim]
+    const float* gain = nullptr;                  // [heads * vdim] or null (ones)
     float eps = 0.f;
     float* out = nullptr;                         // [T][heads * vdim]
 };

@@ -153,10 +153,7 @@ __global__ void __launch_bounds__(LTHREADS) linear_tile_kernel(LinearArgs a) {
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
                 const int n = n0 + tx * 4 + j;
-                if (n + 1 < a.N) {
-                    const float g = acc[i][j];
-                    C[(size_t)r * a.ldc + (n >> 1)] = g / (1.f + expf(-g)) * acc[i][j + 1];
-                }
+                if (n + 1 < a.N) C[(size_t)r * a.ldc + (n >> 1)] = glu_value(a.glu, acc[i][j], acc[i][j + 1], n >> 1);
             }
         } else {
 #pragma unroll
@@ -271,7 +268,7 @@ __global__ void __launch_bounds__(LWARPS * 32) linear_rows_kernel(LinearArgs a) 
                 float v;
                 if (PAIR) {
                     const float g = warp_sum(acc[2 * c][i]), u = warp_sum(acc[2 * c + 1][i]);
-                    v = g / (1.f + expf(-g)) * u;
+                    v = lane == 0 && col0 + c < cols ? glu_value(a.glu, g, u, col0 + c) : 0.f;
                 } else {
                     v = warp_sum(acc[c][i]);
                     if (a.epi == LIN_SOFTCAP) v = a.cap * tanhf(v / a.cap);
@@ -350,12 +347,12 @@ __global__ void gather_planes_kernel2(const float* __restrict__ src, const int* 
     for (int c = threadIdx.x; c < W; c += blockDim.x) store_planes(hi, lo, i * W + c, r[c]);
 }
 
-// gu [rows][2 ff] with columns (2j, 2j+1) = (gate_j, up_j)  ->  planes of silu(gate) * up, [rows][ff]
-__global__ void swiglu_planes_kernel(const float* __restrict__ gu, __nv_bfloat16* __restrict__ hi, __nv_bfloat16* __restrict__ lo,
-                                     size_t n) {
+// gu [rows][2 ff] with columns (2j, 2j+1) = (gate_j, up_j)  ->  planes of their gated product (GluSpec), [rows][ff]
+__global__ void glu_planes_kernel(const float* __restrict__ gu, __nv_bfloat16* __restrict__ hi, __nv_bfloat16* __restrict__ lo, size_t n,
+                                  int ff, GluSpec glu) {
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
         const float2 v = reinterpret_cast<const float2*>(gu)[i];
-        store_planes(hi, lo, i, v.x / (1.f + expf(-v.x)) * v.y);
+        store_planes(hi, lo, i, glu_value(glu, v.x, v.y, glu.bias ? (int)(i % ff) : 0));
     }
 }
 
@@ -373,10 +370,11 @@ int launch_gather_planes_rows(const float* src, const int* idx, void* hi, void* 
     FT_CHECK_CUDA(cudaGetLastError());
     return 0;
 }
-int launch_swiglu_planes(const float* gu, void* hi, void* lo, size_t n, cudaStream_t stream, int act) {
+int launch_act_planes(const float* gu, void* hi, void* lo, int rows, int ff, int act, const GluSpec& glu, cudaStream_t stream) {
+    const size_t n = (size_t)rows * ff;
     const int blocks = (int)std::min<size_t>((n + 255) / 256, 148 * 16);
     if (act == FT_ACT_RELU2) relu2_planes_kernel<<<blocks, 256, 0, stream>>>(gu, (__nv_bfloat16*)hi, (__nv_bfloat16*)lo, n);
-    else swiglu_planes_kernel<<<blocks, 256, 0, stream>>>(gu, (__nv_bfloat16*)hi, (__nv_bfloat16*)lo, n);
+    else glu_planes_kernel<<<blocks, 256, 0, stream>>>(gu, (__nv_bfloat16*)hi, (__nv_bfloat16*)lo, n, ff, glu);
     FT_CHECK_CUDA(cudaGetLastError());
     return 0;
 }

@@ -33,6 +33,12 @@ the softmax and an element-wise output gate, a mixture of experts with biased so
 shared expert under a gate of its own, learned position vectors, and a run of layers that is repeated with the same weights: a
 pass takes the embedding output again and a vector of its own.  The engine sees the repeated layers as further layer RUNS.
 
+The sixth design is Fedutar: sandwich layers again, with plain gains; every mixer is "parallel" — a causal grouped-query attention
+without rotation (per-head RMS-normed queries and keys with gains, a query temperature that grows with the position, an
+element-wise output gate) beside a retention (the decay attention with rotated queries and keys, heads normed apart and a SiLU
+gate) — and the feed-forward is a dense SwiGLU with biases or a mixture of clipped gated experts.  A run of layers is repeated;
+each pass starts from one projection of the stream beside the embedding output.  Its logits come from the embedding table.
+
 The reference names models by tag only and owns no model code (app/utils/config.py:86, docker-compose.vllm.yml:39); this
 module is the model side of what its engine container would load: config.json -> LayeredSpec, model.safetensors -> the
 tensors by their names in the file, pack() -> the device arrays and descriptors the native engine reads.
@@ -50,7 +56,8 @@ import torch
 MIXER_LATENT_ATTENTION, MIXER_CHANNEL_DELTA, MIXER_BRANCHES = 1, 2, 3
 FF_NONE, FF_MOE, FF_DENSE = 0, 1, 2
 LAYER_GATED, LAYER_SANDWICH, LAYER_POSTNORM, LAYER_HYPER, LAYER_PRENORM = 0, 1, 2, 3, 4
-ACT_SWIGLU, ACT_RELU2 = 0, 1
+ACT_SWIGLU, ACT_RELU2, ACT_CLIPPED_GLU = 0, 1, 2
+CLIPPED_ALPHA, CLIPPED_SHIFT = 1.702, 1.0          # Fedutar's experts: g * sigmoid(1.702 g) * (u + 1)
 ROUTE_SOFTMAX, ROUTE_SIGMOID = 0, 1
 BRANCH_WINDOW_ATTENTION, BRANCH_DECAY_ATTENTION, BRANCH_MATRIX_MEMORY, BRANCH_STATE_SPACE, BRANCH_LATENT_WINDOW = 1, 2, 3, 4, 5
 BRANCH_SELECTIVE_SCAN = 6
@@ -103,6 +110,11 @@ class BranchSpec:
     kv_from: int = -1               # layer whose keys and values this one reads
     out_norm_width: bool = False    # the projected output is RMS-normed over the width (gain '<side>out')
     dt_rank: int = 0                # selective scan (heads = channels, dim = states per channel)
+    # window attention options (left side of Fedutar's mixer)
+    out_gate: bool = False          # the concatenated heads are gated element by element
+    q_temp: Tuple[float, ...] = ()  # (coef, every): q *= 1 + coef * ln(1 + floor((p + 1) / every))
+    # decay attention as a retention: no SiLU, rotation (rot_dims, rot_base, halves), k * dim^-1/2, heads normed apart, SiLU gate
+    retention: bool = False
 
 
 @dataclass(frozen=True)
@@ -131,6 +143,10 @@ class LayerSpec:
     # latent attention of pre-norm layers (Gedalix): rotated size (query and shared key part) and its base
     rot_dims: int = 0
     rot_base: float = 10000.0
+    # sandwich layers of Fedutar
+    plain_gain: bool = False        # the norms' weights are the gains themselves (Gedelorn stores gain - 1)
+    ff_bias: bool = False           # dense: biases on all three projections
+    act_limit: Optional[float] = None       # experts: the clipped gated activation with this limit (None: the other activations)
 
 
 @dataclass(frozen=True)
@@ -142,13 +158,14 @@ class LayeredSpec:
     eps: float
     logit_softcap: float
     layers: Tuple[LayerSpec, ...] = field(default_factory=tuple)
-    embed_scale: float = 1.0        # post-norm and hyper-connected models
+    embed_scale: float = 1.0        # post-norm, hyper-connected, pre-norm and looped sandwich models
     canon_taps: int = 0             # post-norm models: taps of the input convolutions
     streams: int = 0                # hyper-connected models: copies of the stream (0: one, and no mixing tensors)
     # pre-norm models
     residual_mult: float = 1.0
     max_positions: int = 0          # rows of the position table
-    loop: Tuple[int, int, int] = () # (start, stop, times): layers start .. stop - 1 run `times` times in a row
+    loop: Tuple[int, int, int] = () # (start, stop, times): layers start .. stop - 1 run `times` times in a row (also sandwich models)
+    logit_scale: float = 1.0        # models whose logits come from the embedding table
 
     def runs(self) -> List[Tuple[int, Optional[int]]]:
         """(layer, pass) in the order the layers run; the pass number stands only at the first layer of a pass over the loop."""
@@ -182,6 +199,15 @@ class LayeredSpec:
                    "width": self.width}
             if self.streams:
                 cfg["streams"] = self.streams
+            return cfg
+        if self.architecture == "Fedutar":
+            cfg = {"architecture": self.architecture, "embedding": {"scale": self.embed_scale},
+                   "layers": [_retentive_layer_config(l) for l in self.layers], "logit_scale": self.logit_scale,
+                   "norm": {"eps": self.eps}, "vocab": self.vocab, "width": self.width}
+            if self.logit_softcap:
+                cfg["logit_softcap"] = self.logit_softcap
+            if self.loop:
+                cfg["loop"] = dict(zip(("start", "stop", "times"), self.loop))
             return cfg
         for l in self.layers:
             if l.form == "sandwich":
@@ -479,16 +505,66 @@ def _sandwich_layer_from_config(i: int, l: Dict) -> LayerSpec:
     return LayerSpec(**kw)
 
 
+def _retentive_layer_config(l: LayerSpec) -> Dict:
+    left, right = l.branches
+    a = {"dim": left.dim, "heads": left.heads, "kv_heads": left.kv_heads, "scale": left.scale, "vdim": left.vdim}
+    if left.q_temp:
+        a["q_temp"] = {"coef": left.q_temp[0], "every": int(left.q_temp[1])}
+    r = {"decay": list(right.decay), "dim": right.dim, "heads": right.heads, "vdim": right.vdim}
+    if right.rot_dims:
+        r["rot"] = {"base": right.rot_base, "dims": right.rot_dims}
+    mlp = None
+    if l.ff_kind == "dense":
+        mlp = {"ff": l.ff, "kind": "dense"}
+    elif l.ff_kind == "moe":
+        mlp = {"expert": {"ff": l.ff, "limit": l.act_limit}, "kind": "moe", "router": {"experts": l.experts, "top": l.top}}
+    return {"mixer": {"left": a, "left_scale": left.out_scale, "right": r, "right_scale": right.out_scale}, "mlp": mlp, "type": l.mixer}
+
+
+def _retentive_layer_from_config(i: int, l: Dict) -> LayerSpec:
+    kind, m, mlp = l["type"], l["mixer"], l.get("mlp")
+    if kind != "parallel":
+        raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+    a, r = m["left"], m["right"]
+    qt, rot = a.get("q_temp") or {}, r.get("rot") or {}
+    heads, dims = int(r["heads"]), int(rot.get("dims", 0))
+    decay = tuple(float(x) for x in r["decay"])
+    if len(decay) != heads:
+        raise ValueError(f"layer {i}: {len(decay)} decays for {heads} heads")
+    if dims % 2 or dims > int(r["dim"]):
+        raise ValueError(f"layer {i}: {dims} rotated coordinates of {r['dim']}")
+    left = BranchSpec(kind="window_attention", heads=int(a["heads"]), kv_heads=int(a.get("kv_heads", a["heads"])), dim=int(a["dim"]),
+                      vdim=int(a.get("vdim", a["dim"])), prefix="left.", out_scale=float(m.get("left_scale", 1.0)), scale=float(a["scale"]),
+                      qk_norm=True, qk_gain="head", out_gate=True, q_temp=(float(qt["coef"]), float(qt["every"])) if qt else ())
+    right = BranchSpec(kind="decay_attention", heads=heads, kv_heads=heads, dim=int(r["dim"]), vdim=int(r["vdim"]), prefix="right.",
+                       out_scale=float(m.get("right_scale", 1.0)), decay=decay, rot_dims=dims, rot_base=float(rot.get("base", 10000.0)),
+                       rot_half=True, retention=True)
+    kw = dict(mixer=kind, form="sandwich", branches=(left, right), plain_gain=True)
+    if mlp:
+        if mlp.get("kind") == "dense":
+            kw.update(ff_kind="dense", ff=int(mlp["ff"]), ff_bias=True)
+        elif mlp.get("kind") == "moe":
+            kw.update(ff_kind="moe", ff=int(mlp["expert"]["ff"]), act_limit=float(mlp["expert"]["limit"]),
+                      experts=int(mlp["router"]["experts"]), top=int(mlp["router"]["top"]))
+        else:
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+    return LayerSpec(**kw)
+
+
 def spec_from_config(cfg: Dict, shapes: Optional[Dict[str, Tuple[int, ...]]] = None, name: str = "checkpoint") -> LayeredSpec:
     """config.json (+ tensor shapes, for the sizes only a shape gives) -> LayeredSpec."""
     layers = []
     postnorm = cfg.get("architecture") == "Vonedra"
     hyper = cfg.get("architecture") == "Lotinex"
     prenorm = cfg.get("architecture") == "Gedalix"
+    retentive = cfg.get("architecture") == "Fedutar"
     for i, l in enumerate(cfg["layers"]):
         kind, m = l["type"], l["mixer"]
         if prenorm:
             layers.append(_prenorm_layer_from_config(i, l))
+            continue
+        if retentive:
+            layers.append(_retentive_layer_from_config(i, l))
             continue
         if hyper:
             layers.append(_hyper_layer_from_config(i, l))
@@ -525,7 +601,7 @@ def spec_from_config(cfg: Dict, shapes: Optional[Dict[str, Tuple[int, ...]]] = N
                        layers=tuple(layers), embed_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)),
                        canon_taps=int((cfg.get("canon") or {}).get("taps", 0)), streams=int(cfg.get("streams") or 0) if hyper else 0,
                        residual_mult=float(cfg.get("residual_mult", 1.0)), max_positions=int(cfg["max_positions"]) if prenorm else 0,
-                       loop=_loop_from_config(cfg) if prenorm else ())
+                       loop=_loop_from_config(cfg) if prenorm or retentive else (), logit_scale=float(cfg.get("logit_scale", 1.0)))
 
 
 def tensor_shapes(spec: LayeredSpec) -> Dict[str, Tuple[int, ...]]:
@@ -545,6 +621,9 @@ def tensor_shapes(spec: LayeredSpec) -> Dict[str, Tuple[int, ...]]:
             out.update(_hyper_shapes(f"l{i}.", l, W, spec.streams))
         out.update({"final.norm": (W,), "final.norm.b": (W,)})      # no head: the logits come from the embedding table
         return out
+    tied = spec.architecture == "Fedutar"        # the logits come from the embedding table
+    if tied and spec.loop:
+        out["loop.in"] = (W, 2 * W)
     for i, l in enumerate(spec.layers):
         p = f"l{i}."
         if l.form == "sandwich":
@@ -573,7 +652,8 @@ def tensor_shapes(spec: LayeredSpec) -> Dict[str, Tuple[int, ...]]:
             out.update({p + "rg2": (W, W), p + "rg2.b": (W,)})
         out.update({p + "rg1": (W, W), p + "rg1.b": (W,)})
     out["final.norm"] = (W,) if spec.layers and spec.layers[-1].form in ("sandwich", "postnorm") else ()
-    out["head"] = (spec.vocab, W)
+    if not tied:
+        out["head"] = (spec.vocab, W)
     return out
 
 
@@ -667,9 +747,15 @@ def _sandwich_shapes(p: str, l: LayerSpec, W: int) -> Dict[str, Tuple[int, ...]]
     for b in l.branches:
         m = p + "mix." + b.prefix
         hv = b.heads * b.vdim
-        if b.kind == "window_attention":
+        if b.kind == "window_attention" and b.out_gate:
+            out.update({m + "q": (b.heads * b.dim, W), m + "k": (b.kv_heads * b.dim, W), m + "v": (b.kv_heads * b.vdim, W),
+                        m + "q.norm": (b.dim,), m + "k.norm": (b.dim,), m + "g": (hv, W), m + "o": (W, hv)})
+        elif b.kind == "window_attention":
             out.update({m + "q": (b.heads * b.dim, W), m + "q.b": (b.heads * b.dim,), m + "k": (b.kv_heads * b.dim, W),
                         m + "k.b": (b.kv_heads * b.dim,), m + "o": (W, hv)})
+        elif b.kind == "decay_attention" and b.retention:
+            out.update({m + "q": (b.heads * b.dim, W), m + "k": (b.heads * b.dim, W), m + "v": (hv, W), m + "g": (hv, W),
+                        m + "o": (W, hv)})
         elif b.kind == "decay_attention":
             out.update({m + "q": (b.heads * b.dim, W), m + "k": (b.heads * b.dim, W), m + "v": (hv, W), m + "g": (hv, W),
                         m + "o": (W, hv), m + "norm": (hv,)})
@@ -686,8 +772,12 @@ def _sandwich_shapes(p: str, l: LayerSpec, W: int) -> Dict[str, Tuple[int, ...]]
         out.update({p + "norm2": (W,), p + "norm2b": (W,)})
     if l.ff_kind == "dense":
         out.update({p + "mlp.gate": (l.ff, W), p + "mlp.up": (l.ff, W), p + "mlp.down": (W, l.ff)})
+        if l.ff_bias:
+            out.update({p + "mlp.gate.b": (l.ff,), p + "mlp.up.b": (l.ff,), p + "mlp.down.b": (W,)})
     elif l.ff_kind == "moe":
         for e in range(l.experts):
+            if l.act_limit is not None:
+                out[f"{p}mlp.e{e}.gate"] = (l.ff, W)
             out.update({f"{p}mlp.e{e}.up": (l.ff, W), f"{p}mlp.e{e}.down": (W, l.ff)})
         out[p + "mlp.router"] = (l.experts, W)
         if l.shared_ff:
@@ -705,6 +795,7 @@ def init_weights(spec: LayeredSpec, seed: int = 0, device: str = "cpu") -> Dict[
     postnorm = bool(spec.layers) and spec.layers[-1].form == "postnorm"
     hyper = bool(spec.layers) and spec.layers[-1].form == "hyper"
     prenorm = bool(spec.layers) and spec.layers[-1].form == "prenorm"
+    plain = sandwich and spec.layers[-1].plain_gain
     for name, shape in tensor_shapes(spec).items():
         leaf = name.split(".")[-1]
         part = name.split(".")[-2] if "." in name else ""
@@ -726,6 +817,8 @@ def init_weights(spec: LayeredSpec, seed: int = 0, device: str = "cpu") -> Dict[
             t = 1.0 + 0.2 * torch.randn(shape, generator=g)
         elif prenorm and (name in ("pos", "loop.step") or leaf in ("sink", "b")):
             t = 0.5 * torch.randn(shape, generator=g)
+        elif plain and (leaf in ("norm1", "norm1b", "norm2", "norm2b") or leaf == "norm"):
+            t = 1.0 + 0.2 * torch.randn(shape, generator=g)
         elif postnorm and leaf in ("canon1", "canon2"):
             t = 0.3 * torch.randn(shape, generator=g)
         elif postnorm and leaf == "dwa":
@@ -821,6 +914,8 @@ class BranchDesc(C.Structure):
         ("rot_half", C.c_int), ("chunked", C.c_int), ("kv_lender", C.c_int), ("rot_mag", C.c_float),
         ("q_gain", C.c_void_p), ("k_gain", C.c_void_p), ("out_gain", C.c_void_p),
         ("dt_rank", C.c_int), ("w_x", C.c_void_p), ("w_dt", C.c_void_p), ("x_rows", C.c_int),
+        ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int), ("plain_qkv", C.c_int), ("head_norm", C.c_int), ("gate_act", C.c_int),
+        ("k_scale", C.c_float),
     ]
 
 
@@ -849,6 +944,8 @@ class LayerDesc(C.Structure):
         ("res_gain", C.c_void_p * 2), ("re_embed", C.c_int), ("pre_add", C.c_void_p),
         ("rot_dims", C.c_int), ("rot_freq", C.c_void_p), ("sink", C.c_void_p), ("gate_wide", C.c_int),
         ("router_bias", C.c_void_p), ("shared_gate", C.c_int),
+        ("act_limit", C.c_float), ("act_alpha", C.c_float), ("act_shift", C.c_float), ("gu_bias", C.c_void_p), ("down_bias", C.c_void_p),
+        ("pass_in", C.c_void_p),
     ]
 
 
@@ -887,20 +984,22 @@ def _interleave(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
 
 
 def _pack_sandwich_layer(l: LayerSpec, w: Dict[str, torch.Tensor], p: str, d, W: int, device, dev, keep: list) -> None:
-    """Descriptor of a sandwich layer: its branches' projections stacked into w_in, norm gains as 1 + stored weight."""
+    """Descriptor of a sandwich layer: its branches' projections stacked into w_in, norm gains as 1 + stored weight (or as stored)."""
     f32 = torch.float32
     d.form, d.mixer, d.n_branches = LAYER_SANDWICH, MIXER_BRANCHES, len(l.branches)
     for f_ in ("o_q", "o_k", "o_v", "o_dkv", "o_gate", "o_beta", "o_a1", "o_g1", "o_rg1", "o_rg2", "o_router"):
         setattr(d, f_, -1)
     d.norm_gain = 1.0
-    gain = lambda name: dev(1.0 + w[name].float(), f32).data_ptr()
+    gain = lambda name: dev(w[name].float() + (0.0 if l.plain_gain else 1.0), f32).data_ptr()
     d.norm_pre1, d.norm_post1 = gain(p + "norm1"), gain(p + "norm1b")
     parts: List[Tuple[str, torch.Tensor]] = []
     for k, b in enumerate(l.branches):
         m = p + "mix." + b.prefix
         if b.kind == "window_attention":
             parts += [(f"{k}q", w[m + "q"]), (f"{k}k", w[m + "k"])]
-        elif b.kind == "decay_attention":      # q | k | v adjacent: one SiLU pass covers them
+            if b.out_gate:
+                parts += [(f"{k}v", w[m + "v"]), (f"{k}g", w[m + "g"])]
+        elif b.kind == "decay_attention":      # q | k | v adjacent: one SiLU or rotation pass covers them
             parts += [(f"{k}q", torch.cat([w[m + "q"], w[m + "k"], w[m + "v"]], 0)), (f"{k}g", w[m + "g"])]
         elif b.kind == "matrix_memory":
             parts += [(f"{k}q", w[m + "q"]), (f"{k}k", w[m + "k"]), (f"{k}v", w[m + "v"]), (f"{k}g", w[m + "g"]),
@@ -927,13 +1026,25 @@ def _pack_sandwich_layer(l: LayerSpec, w: Dict[str, torch.Tensor], p: str, d, W:
                 c.rot_freq = dev(torch.tensor(b.rot_base, dtype=torch.float64) ** (-2.0 * i2 / b.rot_dims), f32).data_ptr()
             if m + "q.b" in w:
                 c.q_bias, c.k_bias = dev(w[m + "q.b"], f32).data_ptr(), dev(w[m + "k.b"], f32).data_ptr()
+            if b.out_gate:
+                c.o_v, c.o_g = offs[f"{k}v"], offs[f"{k}g"]
+                c.qk_norm = 1
+                c.q_gain, c.k_gain = dev(w[m + "q.norm"], f32).data_ptr(), dev(w[m + "k.norm"], f32).data_ptr()
+            if b.q_temp:
+                c.q_temp_coef, c.q_temp_every = b.q_temp[0], int(b.q_temp[1])
         elif b.kind == "decay_attention":
             c.o_q = offs[f"{k}q"]
             c.o_k = c.o_q + b.heads * b.dim
             c.o_v = c.o_k + b.heads * b.dim
             c.o_g = offs[f"{k}g"]
             c.decay = dev(torch.tensor(b.decay, dtype=torch.float64), f32).data_ptr()
-            c.out_norm = dev(w[m + "norm"], f32).data_ptr()
+            if b.retention:
+                c.plain_qkv = c.head_norm = c.gate_act = c.rot_half = 1
+                c.k_scale, c.rot_dims = b.dim ** -0.5, b.rot_dims
+                if b.rot_dims:
+                    c.rot_freq = dev(torch.tensor(rotary_frequencies(b)[0], dtype=torch.float64), f32).data_ptr()
+            else:
+                c.out_norm = dev(w[m + "norm"], f32).data_ptr()
         elif b.kind == "matrix_memory":
             c.o_q, c.o_k, c.o_v, c.o_g, c.o_i, c.o_f = (offs[f"{k}{x}"] for x in "qkvgif")
             c.gate_cap = b.gate_cap
@@ -961,13 +1072,20 @@ def _pack_sandwich_layer(l: LayerSpec, w: Dict[str, torch.Tensor], p: str, d, W:
         d.ff_kind, d.ff_act = FF_DENSE, ACT_SWIGLU
         d.w_gu = dev(_interleave(w[p + "mlp.gate"].to(device), w[p + "mlp.up"].to(device))).data_ptr()
         d.w_down = dev(w[p + "mlp.down"]).data_ptr()
+        if l.ff_bias:
+            d.gu_bias = dev(torch.stack([w[p + "mlp.gate.b"], w[p + "mlp.up.b"]], 1).reshape(-1), f32).data_ptr()
+            d.down_bias = dev(w[p + "mlp.down.b"], f32).data_ptr()
     elif l.ff_kind == "moe":
         d.ff_kind, d.ff_act, d.experts, d.top, d.groups, d.keep = FF_MOE, ACT_RELU2, l.experts, l.top, 1, 1
         d.route_kind, d.route_norm, d.route_scale = ROUTE_SIGMOID, 1, l.route_scale
+        if l.act_limit is not None:             # clipped gated experts; softmax over the chosen logits
+            d.ff_act, d.act_limit, d.act_alpha, d.act_shift = ACT_CLIPPED_GLU, l.act_limit, CLIPPED_ALPHA, CLIPPED_SHIFT
+            d.route_kind, d.route_scale = ROUTE_SOFTMAX, 1.0
         router = torch.zeros((l.experts + 127) // 128 * 128, W, dtype=torch.bfloat16, device=device)
         router[:l.experts] = w[p + "mlp.router"].to(device)
         d.w_router, d.router_rows = dev(router).data_ptr(), router.shape[0]
-        d.w_gu = dev(torch.stack([w[f"{p}mlp.e{e}.up"].to(device) for e in range(l.experts)])).data_ptr()
+        up = lambda q: _interleave(w[q + "gate"].to(device), w[q + "up"].to(device)) if l.act_limit is not None else w[q + "up"].to(device)
+        d.w_gu = dev(torch.stack([up(f"{p}mlp.e{e}.") for e in range(l.experts)])).data_ptr()
         d.w_down = dev(torch.stack([w[f"{p}mlp.e{e}.down"].to(device) for e in range(l.experts)])).data_ptr()
         if l.shared_ff:
             d.shared_ff = l.shared_ff
@@ -1234,13 +1352,20 @@ def pack(spec: LayeredSpec, w: Dict[str, torch.Tensor], device, exact_f32: bool 
             if t is not None:
                 descs[j].re_embed = int(t > 0)
                 descs[j].pre_add = dev(w["loop.step"][t], torch.float32).data_ptr()
+    if spec.layers and spec.layers[0].form == "sandwich":
+        packed = {}
+        pass_in = dev(w["loop.in"]) if spec.loop else None
+        for j, (i, t) in enumerate(runs):
+            if i not in packed:
+                packed[i] = LayerDesc()
+                _pack_sandwich_layer(spec.layers[i], w, f"l{i}.", packed[i], W, device, dev, keep)
+            C.memmove(C.byref(descs[j]), C.byref(packed[i]), C.sizeof(LayerDesc))
+            if t is not None:
+                descs[j].pass_in = pass_in.data_ptr()
     for i, l in enumerate(spec.layers):
         p, d = f"l{i}.", descs[i]
         m = p + "mix."
-        if l.form == "prenorm":
-            continue
-        if l.form == "sandwich":
-            _pack_sandwich_layer(l, w, p, d, W, device, dev, keep)
+        if l.form in ("prenorm", "sandwich"):
             continue
         if l.form == "hyper":
             _pack_hyper_layer(spec, i, l, w, p, d, W, device, dev, keep)
@@ -1305,6 +1430,8 @@ def pack(spec: LayeredSpec, w: Dict[str, torch.Tensor], device, exact_f32: bool 
     postnorm = bool(spec.layers) and spec.layers[0].form == "postnorm"
     hyper = bool(spec.layers) and spec.layers[0].form == "hyper"
     prenorm = bool(spec.layers) and spec.layers[0].form == "prenorm"
+    plain = bool(spec.layers) and spec.layers[0].plain_gain
+    tied = hyper or spec.architecture == "Fedutar"
     if prenorm:
         model.pos_embed, model.max_positions = dev(w["pos"]).data_ptr(), spec.max_positions
     if hyper:                                # a layer norm with gain and bias; the logits come from the embedding table
@@ -1316,10 +1443,12 @@ def pack(spec: LayeredSpec, w: Dict[str, torch.Tensor], device, exact_f32: bool 
         model.final_norm_gain = float(w["final.norm"].float().item())
     else:
         model.final_norm_gain = 1.0          # sandwich models store gain - 1, post-norm and pre-norm models the gain itself
-        model.final_norm_w = dev(w["final.norm"].float() + (0.0 if postnorm or prenorm else 1.0), torch.float32).data_ptr()
-    model.embed_scale = spec.embed_scale if postnorm or hyper or prenorm else 1.0
+        # (a factor on the logits goes into it: the head is linear)
+        gain = w["final.norm"].double() + (0.0 if postnorm or prenorm or plain else 1.0)
+        model.final_norm_w = dev(gain * spec.logit_scale, torch.float32).data_ptr()
+    model.embed_scale = spec.embed_scale if postnorm or hyper or prenorm or plain else 1.0
     model.embed = dev(w["embed"]).data_ptr()
-    model.head = model.embed if hyper else dev(w["head"]).data_ptr()
+    model.head = model.embed if tied else dev(w["head"]).data_ptr()
     model.layers = C.cast(descs, C.POINTER(LayerDesc))
     model.exact_f32 = int(exact_f32)
     keep.append(descs)

@@ -193,6 +193,9 @@ enum { FT_FF_NONE = 0, FT_FF_MOE = 1, FT_FF_DENSE = 2 };
  *   FT_LAYER_GATED:    the form above (one scalar-gain norm feeds both sublayers, sigmoid gates on the way back).
  *   FT_LAYER_SANDWICH: x += post1(mixer(pre1(x))); x += post2(ff(pre2(x))), each of the four an RMS norm with a gain per
  *                      coordinate, given as the gain itself (a checkpoint that stores gain - 1 is converted at load time). */
+/*                      Before a layer (run) with pass_in the stream is first projected together with the embedding output,
+ *                      x <- pass_in [x; x0]: what a model that runs some of its layers several times in a row does ahead of each
+ *                      pass (given as layer runs, see FT_LAYER_PRENORM). */
 /*   FT_LAYER_POSTNORM: the sublayers read the stream itself, through a short causal convolution over time per coordinate
  *                      (h = x + conv(x), taps canon_taps, the last column of the [width][taps] table weighs the current
  *                      token; the last taps - 1 stream rows of each sublayer live in the session's state slot), and only
@@ -213,7 +216,9 @@ enum { FT_FF_NONE = 0, FT_FF_MOE = 1, FT_FF_DENSE = 2 };
  *                      descriptors with the same weights, each with a cache of its own.  Takes latent attention and any
  *                      feed-forward. */
 enum { FT_LAYER_GATED = 0, FT_LAYER_SANDWICH = 1, FT_LAYER_POSTNORM = 2, FT_LAYER_HYPER = 3, FT_LAYER_PRENORM = 4 };
-enum { FT_ACT_SWIGLU = 0, FT_ACT_RELU2 = 1 };          /* expert: W_down (silu(W_gate h) * W_up h)  |  W_down relu(W_up h)^2 */
+/* a feed-forward's activation: W_down (silu(W_gate h) * W_up h)  |  W_down relu(W_up h)^2  |  with g = min(W_gate h, act_limit) and
+ * u = W_up h clamped to +- act_limit: W_down (g * sigmoid(act_alpha * g) * (u + act_shift)) */
+enum { FT_ACT_SWIGLU = 0, FT_ACT_RELU2 = 1, FT_ACT_CLIPPED_GLU = 2 };
 enum { FT_ROUTE_SOFTMAX = 0, FT_ROUTE_SIGMOID = 1 };   /* router scores over all experts */
 
 /* Branch mixers (mixer == FT_MIXER_BRANCHES): one or two token mixers side by side on the same normed input, each with
@@ -254,6 +259,12 @@ enum { FT_ROUTE_SOFTMAX = 0, FT_ROUTE_SIGMOID = 1 };   /* router scores over all
  * token, no bias; the last conv - 1 projected rows live in the session's state slot); kv_lender (n > 0: the branch has no
  * keys and values of its own and attends over the cache of layer n - 1's first window-attention branch, which has the same
  * key heads and sizes).
+ * Further options of window attention: o_g (heads * vdim columns: the concatenated heads are multiplied element by element by their
+ * sigmoid before the output projection); q_temp_coef, q_temp_every (the query at position p is multiplied by
+ * 1 + q_temp_coef * ln(1 + floor((p + 1) / q_temp_every)), after norm, gain and rotation).
+ * Options of decay attention: plain_qkv (no SiLU on q, k, v), rot_dims + rot_freq + rot_half (q and k rotated as in window
+ * attention), k_scale (k is multiplied by it; 0 = 1), head_norm (every head is divided by its own root mean square; out_norm may
+ * then be null), gate_act 1 (the gate is silu(g) instead of sigmoid(g)).
  *   FT_BRANCH_SELECTIVE_SCAN    heads = channels, dim = N states per channel, vdim = 1.  x (columns o_v) passes a short causal
  *                               convolution with bias and SiLU; w_x x = [dt_rank | N | N] = (low, B, C); dt = softplus(w_dt low +
  *                               dt_bias) per channel; S[c][n] <- exp(-exp(a_log[c][n]) dt_c) S[c][n] + dt_c x_c B_n;
@@ -315,6 +326,12 @@ typedef struct {
     const void* w_dt;          /* bf16 [heads][dt_rank] */
     int x_rows;                /* 0, or the rows of w_x when it is padded with zero rows to whole GEMM tiles; w_dt is then
                                   [heads][x_rows] with zeros beyond column dt_rank (it reads the whole low-rank row) */
+    /* further window-attention options (see above) */
+    float q_temp_coef;
+    int q_temp_every;          /* 0 = no temperature */
+    /* decay-attention options (see above) */
+    int plain_qkv, head_norm, gate_act;
+    float k_scale;
 } ft_branch_desc;
 
 typedef struct {
@@ -398,6 +415,11 @@ typedef struct {
     /* ---- router and shared expert options of the forms whose router is a matrix of its own ---- */
     const float* router_bias;  /* fp32 [experts] or null: added to the router logits */
     int shared_gate;           /* 1: row `experts` of w_router gates the shared expert's output by its sigmoid, one number per token */
+    /* ---- activation constants (FT_ACT_CLIPPED_GLU) and biases of a sandwich layer's dense feed-forward ---- */
+    float act_limit, act_alpha, act_shift;
+    const float* gu_bias;      /* fp32 [2 * ff], paired like the rows of w_gu, or null */
+    const float* down_bias;    /* fp32 [width] or null */
+    const void* pass_in;       /* FT_LAYER_SANDWICH: bf16 [width][2 * width] or null */
 } ft_layer_desc;
 
 typedef struct {
@@ -413,7 +435,7 @@ typedef struct {
                                   the tensor cores (tcgen05) from bf16 hi + lo planes of the fp32 activations with fp32
                                   accumulation; norms, scores, softmax, router, recurrence and residual stay fp32 */
     const float* final_norm_w; /* fp32 [width] or null: a gain per coordinate instead of final_norm_gain */
-    float embed_scale;         /* FT_LAYER_POSTNORM / _HYPER / _PRENORM models: the embedding output is embed[token] * embed_scale (0 = 1) */
+    float embed_scale;         /* FT_LAYER_SANDWICH / _POSTNORM / _HYPER / _PRENORM models: the embedding output is embed[token] * embed_scale (0 = 1) */
     const float* final_norm_b; /* FT_LAYER_HYPER models: the last norm is a layer norm with gain final_norm_w and this bias */
     int streams;               /* FT_LAYER_HYPER models: copies of the stream (0 = 1) */
     const void* pos_embed;     /* FT_LAYER_PRENORM models: bf16 [max_positions, width] or null, a learned vector per position that the
