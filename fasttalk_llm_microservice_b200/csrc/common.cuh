@@ -292,10 +292,11 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t* r) {
 }
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 // MN-major SWIZZLE_128B operand (V slab): 8-row groups (8 keys x 128 B) 1024 B apart along K; one 64-element MN block
-__device__ __forceinline__ uint64_t umma_desc_mn128(uint32_t smem_addr) {
+// (block_bytes: from one block of 64 MN elements to the next)
+__device__ __forceinline__ uint64_t umma_desc_mn128(uint32_t smem_addr, uint32_t block_bytes = kKvTile * 128) {
     uint64_t d = 0;
     d |= (uint64_t)((smem_addr & 0x3ffff) >> 4);
-    d |= (uint64_t)((kKvTile * 128) >> 4) << 16;      // LBO: stride between 64-element MN blocks = one [64 keys][64 columns] slab
+    d |= (uint64_t)(block_bytes >> 4) << 16;          // LBO: stride between 64-element MN blocks (of the cache: one [64 keys][64 columns] slab)
     d |= (uint64_t)(1024 >> 4) << 32;       // SBO: stride between 8-row K groups
     d |= (uint64_t)1 << 46;
     d |= (uint64_t)2 << 61;                 // SWIZZLE_128B

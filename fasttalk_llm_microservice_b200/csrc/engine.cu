@@ -173,6 +173,8 @@ struct LayeredLayer {
     size_t s_off = 0, tail_off = 0;    // floats inside a state slot: S [heads][dim][vdim], tails [channels][conv - 1]
     // branch mixers: per branch its block in kv_cache (window attention), its S inside a state slot, and what else it keeps
     // there (the running maximum of a matrix memory, the convolution tails of a state space)
+    size_t br_cache16_off[2] = {0, 0}; // bf16: the branch's block in kv_cache16 (br_tensor)
+    bool br_tensor[2] = {false, false};
     size_t br_cache_off[2] = {0, 0}, br_s_off[2] = {0, 0}, br_x_off[2] = {0, 0};
     size_t canon_off[2] = {0, 0};      // post-norm layers: the tails [taps - 1][width] of the two input convolutions in a slot
     int lender_branch[2] = {0, 0};     // window attention over another layer's cache: which branch of that layer owns it
@@ -184,6 +186,9 @@ struct Layered {
     void* lat_cache16 = nullptr;       // serving form: the latents in bf16 for the tensor-core attention (lat_cache is then only
                                        // there when a layer's sizes are beyond that kernel)
     float* kv_cache = nullptr;         // window-attention branches: per layer [num_pages][64][kv_heads * (dim + vdim)] fp32
+    void* kv_cache16 = nullptr;        // branches whose serving form keeps keys and values in bf16 (Paged16Args)
+    void *r16 = nullptr;               // packed rows of a retention's portions
+    float* ret_ws = nullptr;           // states at the starts of their runs
     float* state = nullptr;
     size_t slot_stride = 0;            // floats per state slot
     int n_stateful = 0;                // layers whose mixer carries state from token to token
@@ -579,13 +584,15 @@ static int forward(Engine* e, const Batch& b) {
 // as bf16 hi + lo planes (`hi` / `lo` if the producer already wrote them, else staged here), fp32 out.  Otherwise, and always
 // in the exact-fp32 form, the CUDA-core kernels.
 constexpr int kTensorMinRows = 9;
-constexpr int kLatentTcMinTokens = 32;       // portion tokens of a step from which latent attention takes 128-row tiles
+static bool dense_tiles(const Engine* e, int T, int N, int K) { return e->lay->tensor && T >= kTensorMinRows && N % 128 == 0 && K % 64 == 0; }
+constexpr int kAttnTcMinTokens = 32;         // portion tokens of a step from which attention over a bf16 cache takes 128-row tiles
+constexpr int kRetentionTcMinTokens = 32;    // portion tokens of a step from which a retention runs on the tensor cores
 constexpr int kFuseCanonRows = 256;          // steps up to this many rows form the feed-forward's input inside the post-norm kernel
 constexpr int kMoeTensorMinPairs = 256;      // (token, choice) pairs from which the experts run as per-expert tensor-core GEMMs
 static int dense(Engine* e, const float* A, const void* hi, const void* lo, const void* W, float* C, int T, int N, int K,
                  float softcap = 0.f) {
     Layered& L = *e->lay;
-    if (L.tensor && T >= kTensorMinRows && N % 128 == 0 && K % 64 == 0) {
+    if (dense_tiles(e, T, N, K)) {
         if (!hi) {
             FT_TRY(launch_to_planes(A, L.pl_hi, L.pl_lo, (size_t)T * K, e->stream));
             e->st.kernel_launches++;
@@ -735,6 +742,22 @@ static int run_mlp(Engine* e, const void* hi, const void* lo, const void* w_up, 
     return dense(e, L.ffb, nullptr, nullptr, w_down, out, T, W, ff);
 }
 
+// The sizes of a window-attention branch whose serving form keeps keys and values in bf16.
+static void branch_paged(const ft_branch_desc& c, Paged16Args& p) {
+    p.H = c.heads; p.G = c.kv_heads; p.dim = c.dim; p.vdim = c.vdim;
+    p.key_blocks = p.v_block = (c.dim + 63) / 64;
+    p.blocks = p.key_blocks + (c.vdim + 63) / 64;
+}
+static bool branch_on_tensor(const ft_layered_model& M, const ft_branch_desc& c) {
+    Paged16Args p;
+    branch_paged(c, p);
+    return M.exact_f32 == 0 && c.kind == FT_BRANCH_WINDOW_ATTENTION && c.tensor_cache && c.window == 0 && c.softcap == 0.f && !c.rel &&
+           c.keep_first == 0 && c.qk_norm <= 1 && c.o_v >= 0 && c.v_role == 0 && c.kv_lender == 0 && c.dim <= 512 && c.vdim <= 512 &&
+           paged16_mma_ok(p) && paged16_tc_ok(p);
+}
+// Decay attention in the form retention.cu computes.
+static bool retention_branch(const ft_branch_desc& c) { return c.plain_qkv && c.head_norm && !c.out_norm && c.kv_heads == c.heads; }
+
 // One branch of a branch mixer: from the layer's stacked projection L.proj to `y` [T][width] (before its out_scale).
 static int run_branch(Engine* e, const Batch& b, const LayeredLayer& ll, int k, float* y) {
     Layered& L = *e->lay;
@@ -747,6 +770,10 @@ static int run_branch(Engine* e, const Batch& b, const LayeredLayer& ll, int k, 
     auto launched = [&](int n = 1) { e->st.kernel_launches += n; };
     const float* fin = L.bfin;
     int fin_cols = c.heads * c.vdim;
+    // a branch whose kernels can leave their result as the planes the output projection reads
+    void *fin_hi = nullptr, *fin_lo = nullptr;
+    const bool tiles = dense_tiles(e, T, M.width, fin_cols);
+    const int n_rows = T - b.n_decode;           // rows of prompt portions
     if (c.kind == FT_BRANCH_WINDOW_ATTENTION || c.kind == FT_BRANCH_LATENT_WINDOW) {
         WindowArgs a;
         a.q_out = L.bq; a.cache = L.kv_cache + ll.br_cache_off[k];
@@ -799,8 +826,23 @@ static int run_branch(Engine* e, const Batch& b, const LayeredLayer& ll, int k, 
         WindowTiles tm;
         tm.tile_req = d + m.o_treq; tm.tile_q0 = d + m.o_tq0; tm.req_q_start = d + m.o_qstart; tm.req_slot = d + m.o_rslot;
         tm.req_pos0 = d + m.o_rpos0; tm.n_tiles = b.n_tiles;
-        FT_TRY(launch_window_attention(a, T, b.n_decode, tm, st));
-        launched(b.n_tiles > 0 && b.n_decode > 0 ? 3 : 2);
+        if (ll.br_tensor[k]) {
+            Paged16Args p;
+            p.q = (const __nv_bfloat16*)L.bq; p.cache = (const uint8_t*)L.kv_cache16 + ll.br_cache16_off[k] * 2;
+            p.positions = a.positions; p.seq_rows = a.seq_rows; p.page_table = a.page_table; p.max_pages = a.max_pages;
+            branch_paged(c, p);
+            p.sink = a.sink; p.gate = a.gate; p.ldg = a.ldg; p.gate_wide = 1; p.out = L.bfin; p.part = L.attn_part;
+            if (tiles) { p.out_hi = fin_hi = L.pl_hi; p.out_lo = fin_lo = L.pl_lo; }
+            FT_TRY(launch_paged16_write(a, (__nv_bfloat16*)L.bq, (uint8_t*)L.kv_cache16 + ll.br_cache16_off[k] * 2, T, st));
+            const bool tc = n_rows >= kAttnTcMinTokens;
+            if (tc) FT_TRY(launch_paged16_tc(p, tm, e->h_kernel_err, st));
+            const int rows = tc ? b.n_decode : T;
+            if (rows > 0) FT_TRY(launch_paged16_mma(p, rows, st));
+            launched(1 + (tc ? 1 : 0) + (rows > 0 ? 2 : 0));
+        } else {
+            FT_TRY(launch_window_attention(a, T, b.n_decode, tm, st));
+            launched(b.n_tiles > 0 && b.n_decode > 0 ? 3 : 2);
+        }
         if (c.kind == FT_BRANCH_LATENT_WINDOW) {
             LinearArgs v;                   // values out of latent space: o_h = W_uv_h (sum_j p_j c_j)
             v.A = L.bfin; v.lda = c.heads * c.kv_rank; v.a_col_stride = c.kv_rank;
@@ -847,24 +889,53 @@ static int run_branch(Engine* e, const Batch& b, const LayeredLayer& ll, int k, 
         r.heads = c.heads; r.qk_heads = c.kv_heads; r.dim = c.dim; r.vd = c.vdim; r.ldo = c.heads * c.vdim;
         ReadoutArgs o;
         o.o = L.bo; o.vd = c.vdim; o.vdim = c.vdim; o.heads = c.heads; o.gain = c.out_norm; o.eps = M.eps; o.out = L.bfin;
+        int q0 = 0, r0 = 0;                      // first row and request that still go through the rule
+        if (c.kind == FT_BRANCH_DECAY_ATTENTION && retention_branch(c)) {
+            // single tokens in one pass over their states; portions in runs on the tensor cores where the sizes allow it
+            RetentionArgs a;
+            a.proj = L.proj; a.ldp = ld; a.o_q = c.o_q; a.o_k = c.o_k; a.o_v = c.o_v; a.o_g = c.o_g; a.heads = c.heads; a.dim = c.dim;
+            a.vdim = c.vdim; a.rot_dims = c.rot_dims; a.rot_half = c.rot_half; a.gate_act = c.gate_act; a.rot_freq = c.rot_freq; a.decay = c.decay;
+            a.k_scale = c.k_scale != 0.f ? c.k_scale : 1.f; a.eps = M.eps; a.positions = d + m.o_pos; a.state = L.state;
+            a.slot_stride = r.slot_stride; a.s_off = r.s_off; a.req_start = r.req_start; a.req_pos0 = r.req_pos0; a.req_slot = r.req_slot;
+            a.out = L.bfin;
+            const bool tc = L.ret_ws && n_rows >= kRetentionTcMinTokens && retention_tc_ok(c.dim, c.vdim), one = retention_one_pass(c.vdim);
+            if (tiles && (n_rows == 0 || (tc && one))) { a.out_hi = fin_hi = L.pl_hi; a.out_lo = fin_lo = L.pl_lo; }
+            FT_TRY(launch_retention_step(a, b.n_decode, st));
+            launched(b.n_decode > 0 ? 1 : 0);
+            q0 = b.n_decode; r0 = b.n_decode;
+            if (tc) {
+                WindowTiles tm;
+                tm.tile_req = d + m.o_treq; tm.tile_q0 = d + m.o_tq0; tm.req_q_start = d + m.o_qstart; tm.req_slot = d + m.o_rslot;
+                tm.req_pos0 = d + m.o_rpos0; tm.n_tiles = b.n_tiles;
+                const size_t qn = (size_t)n_rows * c.heads * retention_padded(c.dim);
+                a.q16 = L.r16; a.k16 = (uint8_t*)L.r16 + qn * 2; a.v16 = (uint8_t*)L.r16 + qn * 4; a.ws = L.ret_ws;
+                if (!one) a.out = L.bo;          // before norm and gate
+                FT_TRY(launch_retention_tc(a, tm, b.n_decode, b.n_decode, n_rows, b.n_req - b.n_decode, e->h_kernel_err, st));
+                launched(4);
+                r0 = b.n_req;
+                if (one) q0 = T;
+            }
+        }
         if (c.kind == FT_BRANCH_DECAY_ATTENTION) {
             // q | k | v are adjacent columns of the projection: SiLU or rotation in place, then the rule reads them where they are
-            if (!c.plain_qkv) {
+            if (!c.plain_qkv && r0 < b.n_req) {
                 FT_TRY(launch_silu_cols(L.proj, ld, c.o_q, 2 * c.kv_heads * c.dim + c.heads * c.vdim, T, st));
                 launched();
             }
-            if (c.rot_dims > 0 || (c.k_scale != 0.f && c.k_scale != 1.f)) {
+            if (r0 < b.n_req && (c.rot_dims > 0 || (c.k_scale != 0.f && c.k_scale != 1.f))) {
                 TurnArgs tq;
-                tq.proj = L.proj; tq.ldp = ld; tq.o_q = c.o_q; tq.o_k = c.o_k; tq.heads = c.heads; tq.kv_heads = c.kv_heads; tq.dim = c.dim;
+                tq.proj = L.proj + (size_t)q0 * ld; tq.ldp = ld; tq.o_q = c.o_q; tq.o_k = c.o_k; tq.heads = c.heads; tq.kv_heads = c.kv_heads; tq.dim = c.dim;
                 tq.rot_dims = c.rot_dims; tq.rot_half = c.rot_half; tq.rot_freq = c.rot_freq; tq.k_scale = c.k_scale != 0.f ? c.k_scale : 1.f;
-                tq.positions = d + m.o_pos;
-                FT_TRY(launch_turn_qk(tq, T, st));
+                tq.positions = d + m.o_pos + q0;
+                FT_TRY(launch_turn_qk(tq, T - q0, st));
                 launched();
             }
-            FT_TRY(launch_const_decay(c.decay, L.ab, c.heads, T, st));
+            if (r0 < b.n_req) {
+                FT_TRY(launch_const_decay(c.decay, L.ab, c.heads, T, st));
+                launched();
+            }
             r.q = L.proj + c.o_q; r.k = L.proj + c.o_k; r.v = L.proj + c.o_v; r.ldq = r.ldk = r.ldv = ld;
             o.gate = L.proj + c.o_g; o.ldg = ld; o.gate_kind = c.gate_act ? 3 : 2; o.norm_groups = c.head_norm ? c.heads : 1;
-            launched();
         } else if (c.kind == FT_BRANCH_MATRIX_MEMORY) {
             MemoryArgs g;
             g.proj = L.proj; g.ldp = ld; g.o_v = c.o_v; g.o_i = c.o_i; g.o_f = c.o_f; g.gate_bias = c.gate_bias; g.cap = c.gate_cap;
@@ -892,11 +963,21 @@ static int run_branch(Engine* e, const Batch& b, const LayeredLayer& ll, int k, 
             launched(2);
         }
         o.ldo = r.ldo;
-        FT_TRY(launch_decay_rule(r, b.n_req, T, st));
-        FT_TRY(launch_readout(o, T, st));
-        launched(2);
+        if (r0 < b.n_req) {
+            r.req_start += r0; r.req_pos0 += r0; r.req_slot += r0;
+            FT_TRY(launch_decay_rule(r, b.n_req - r0, T - q0, st));
+            launched();
+        }
+        if (q0 < T) {
+            o.o += (size_t)q0 * o.ldo; o.out += (size_t)q0 * fin_cols;
+            if (o.gate) o.gate += (size_t)q0 * o.ldg;
+            if (o.x) o.x += (size_t)q0 * o.ldx;
+            if (o.floor) o.floor += (size_t)q0 * o.heads;
+            FT_TRY(launch_readout(o, T - q0, st));
+            launched();
+        }
     }
-    return dense(e, fin, nullptr, nullptr, c.w_o, y, T, M.width, fin_cols);
+    return dense(e, fin, fin_hi, fin_lo, c.w_o, y, T, M.width, fin_cols);
 }
 
 // Forward pass of a layered model.  Per layer: ONE projection of the normed input into all the parts that read it
@@ -1013,12 +1094,12 @@ static int forward_layered(Engine* e, const Batch& b) {
             a.M = T; a.N = c.kv_rank; a.K = c.dim; a.P = c.heads;
             FT_TRY(heads(e, a));
             // prompt portions on tcgen05, single tokens of running sequences (and steps of a few portion tokens) row by row
-            const bool tc = la.cache16 && b.n_tiles > 0 && T - b.n_decode >= kLatentTcMinTokens && latent_prefill_tc_ok(c.kv_rank, R);
+            const bool tc = la.cache16 && b.n_tiles > 0 && T - b.n_decode >= kAttnTcMinTokens && paged16_tc_ok(latent_paged(la, c.kv_rank, R));
             if (tc) {
                 WindowTiles tm;
                 tm.tile_req = d + m.o_treq; tm.tile_q0 = d + m.o_tq0; tm.req_q_start = d + m.o_qstart; tm.req_slot = d + m.o_rslot;
                 tm.req_pos0 = d + m.o_rpos0; tm.n_tiles = b.n_tiles;
-                FT_TRY(launch_latent_prefill_tc(la, tm, e->h_kernel_err, st));
+                FT_TRY(launch_paged16_tc(latent_paged(la, c.kv_rank, R), tm, e->h_kernel_err, st));
                 launched(b.n_decode > 0 ? 1 : 0);
             }
             const int rows = tc ? b.n_decode : T;
@@ -1765,7 +1846,8 @@ static int engine_init_layered(Engine* e) {
     bool latent_f32 = M.exact_f32 != 0;
     size_t kv_floats = 0, br_q = 0, br_v = 0, br_o = 0, br_fin = 0, br_heads = 0, e_max_s = 1, scan_cn = 0;
     int n_in_max = 1, top_max = 1, heads_max = 1, rank_max = 0;
-    size_t vfirst_cols = 0, lstage_cols = 0;
+    size_t vfirst_cols = 0, lstage_cols = 0, kv16 = 0, r16_cols = 0, ret_cols = 0;
+    int part_cols = 0;
     bool use_hist = false, has_pass = false;
     for (int l = 0; l < M.n_layers; ++l) {
         LayeredLayer& ll = L.layers[l];
@@ -1850,8 +1932,18 @@ static int engine_init_layered(Engine* e) {
                                    "engine: layer %d: layer %d has no keys and values of its sizes to lend", l, c.kv_lender - 1);
                         ll.lender_branch[k] = found;
                     } else {
-                        ll.br_cache_off[k] = kv_floats;
-                        kv_floats += (size_t)e->cfg.num_pages * kKvTile * c.kv_heads * (c.dim + c.vdim);
+                        if (branch_on_tensor(M, c)) {
+                            Paged16Args p;
+                            branch_paged(c, p);
+                            ll.br_tensor[k] = true;
+                            ll.br_cache16_off[k] = kv16;
+                            kv16 += (size_t)e->cfg.num_pages * kKvTile * c.kv_heads * p.blocks * 64;
+                            br_q = std::max(br_q, (size_t)c.heads * p.key_blocks * 32);      // bf16 queries in the fp32 queries' buffer
+                            part_cols = std::max(part_cols, c.vdim);
+                        } else {
+                            ll.br_cache_off[k] = kv_floats;
+                            kv_floats += (size_t)e->cfg.num_pages * kKvTile * c.kv_heads * (c.dim + c.vdim);
+                        }
                     }
                     if (c.conv >= 1) {           // the last conv - 1 projected q | k | v rows of the sequence
                         const size_t ch = (size_t)c.heads * c.dim + (c.kv_lender > 0 ? 0 : (size_t)c.kv_heads * (c.dim + c.vdim));
@@ -1888,6 +1980,10 @@ static int engine_init_layered(Engine* e) {
                     L.slot_stride += (size_t)c.heads * c.dim * c.vdim;
                     br_o = std::max(br_o, hv);
                     L.n_stateful++;
+                    if (M.exact_f32 == 0 && retention_branch(c) && retention_tc_ok(c.dim, c.vdim)) {
+                        r16_cols = std::max(r16_cols, (size_t)c.heads * (2 * retention_padded(c.dim) + retention_padded(c.vdim)));
+                        ret_cols = std::max(ret_cols, (size_t)c.heads * c.dim * c.vdim);
+                    }
                 } else if (c.kind == FT_BRANCH_MATRIX_MEMORY) {
                     FT_REQUIRE(c.kv_heads == c.heads && c.gate_bias && c.gate_cap > 0.f && c.out_norm && c.o_v >= 0 && c.o_g >= 0 &&
                                    c.o_i >= 0 && c.o_f >= 0,
@@ -1997,6 +2093,11 @@ static int engine_init_layered(Engine* e) {
     if (cache16 && M.exact_f32 == 0) FT_TRY(alloc(&L.lat_cache16, cache16 * 2));
     FT_TRY(alloc(&L.state, L.slot_stride * (size_t)c.max_sessions * 4));
     if (kv_floats) FT_TRY(alloc(&L.kv_cache, kv_floats * 4));
+    if (kv16) FT_TRY(alloc(&L.kv_cache16, kv16 * 2));
+    if (r16_cols) {
+        FT_TRY(alloc(&L.r16, T * r16_cols * 2));
+        FT_TRY(alloc(&L.ret_ws, (size_t)retention_ws_runs((int)T, e->r_max) * ret_cols * 4));
+    }
     if (br_fin) {
         FT_TRY(alloc(&L.bq, T * br_q * 4));
         FT_TRY(alloc(&L.bv, T * br_v * 4));
@@ -2047,7 +2148,8 @@ static int engine_init_layered(Engine* e) {
     FT_TRY(alloc(&L.b3, T * buf * 4));
     FT_TRY(alloc(&L.b4, T * buf * 4));
     FT_TRY(alloc(&L.beta, T * heads_max * 4));
-    if (rank_max > 0) FT_TRY(alloc(&L.attn_part, (size_t)kLatentSplitPairs * kLatentMaxSplits * (rank_max + 2) * 4));
+    part_cols = std::max(part_cols, rank_max);
+    if (part_cols > 0) FT_TRY(alloc(&L.attn_part, (size_t)kAttnSplitPairs * kAttnMaxSplits * (part_cols + 2) * 4));
     FT_TRY(alloc(&L.mix, T * W * 4));
     FT_TRY(alloc(&L.act, T * top_max * act_cols * 4));
     FT_TRY(alloc(&L.eout, T * top_max * W * 4));
@@ -2097,7 +2199,7 @@ static void engine_free(Engine* e) {
         cudaFree(L.b3); cudaFree(L.b4); cudaFree(L.beta); cudaFree(L.attn_part); cudaFree(L.mix); cudaFree(L.act); cudaFree(L.eout);
         cudaFree(L.kv_cache); cudaFree(L.bq); cudaFree(L.bv); cudaFree(L.bo); cudaFree(L.bfin); cudaFree(L.ab); cudaFree(L.gates);
         cudaFree(L.hist); cudaFree(L.v_first); cudaFree(L.lstage); cudaFree(L.resid2); cudaFree(L.streams);
-        cudaFree(L.cat); cudaFree(L.cat_hi); cudaFree(L.cat_lo);
+        cudaFree(L.kv_cache16); cudaFree(L.r16); cudaFree(L.ret_ws); cudaFree(L.cat); cudaFree(L.cat_hi); cudaFree(L.cat_lo);
         cudaFree(L.floor); cudaFree(L.mix2); cudaFree(L.ffa); cudaFree(L.ffb); cudaFree(L.rlog);
         cudaFree(L.wts); cudaFree(L.xlast); cudaFree(L.ids); cudaFree(L.seg); cudaFree(L.slot_token);
         cudaFree(L.slot_pos); cudaFree(L.trail); cudaFree(L.pl_hi); cudaFree(L.pl_lo); cudaFree(L.hn_hi); cudaFree(L.hn_lo);

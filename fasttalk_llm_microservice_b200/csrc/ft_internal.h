@@ -137,7 +137,7 @@ struct LinearArgs {
 // rows_bound: M when batched; an upper bound of seg[P] when grouped
 int launch_linear(const LinearArgs& a, int rows_bound, cudaStream_t stream);
 // ---- heads_tc.cu: a batched LinearArgs (seg, a_rows null) on tcgen05, fp32 activations as bf16 hi + lo planes; K and N whole
-// 32-column pieces.  err as for launch_latent_prefill_tc
+// 32-column pieces.  err as for launch_paged16_tc
 bool linear_heads_ok(const LinearArgs& a);
 int launch_linear_heads(const LinearArgs& a, int* err, cudaStream_t stream);
 // hi / lo (may be null): the normed row once more as bf16 planes, the input form of the tensor-core projections
@@ -175,12 +175,16 @@ struct LatentArgs {
 };
 // Latent normed, shared key part rotated -> the caches; the rotated part of every query -> qlat or qlat16.
 int launch_latent_prep(const LatentArgs& a, int T, cudaStream_t stream);
-// With fewer than kLatentSplitPairs (token, head) pairs in a step the keys of each are cut into up to kLatentMaxSplits
+// With fewer than kAttnSplitPairs (token, head) pairs in a step the keys of each are cut into up to kAttnMaxSplits
 // shares that run side by side; `part` then holds pairs x shares x (rank + 2) floats (null: never split).
-constexpr int kLatentSplitPairs = 2048, kLatentMaxSplits = 8;
-int latent_attn_splits(int T, int H);
-// With cache16 and sizes the tensor-core kernel is built for (latent_attn_mma_ok) the attention runs on mma.sync from bf16
-// operands and `cache` may be null; otherwise on the CUDA cores in fp32.
+constexpr int kAttnSplitPairs = 2048, kAttnMaxSplits = 8;
+inline int attn_splits(int T, int H) {
+    const int pairs = T * H > 0 ? T * H : 1;
+    const int n = pairs >= kAttnSplitPairs ? 1 : kAttnSplitPairs / pairs;
+    return n < kAttnMaxSplits ? n : kAttnMaxSplits;
+}
+// With cache16 and sizes the tensor-core kernels are built for (latent_attn_mma_ok) the attention runs from bf16
+// operands (Paged16Args) and `cache` may be null; otherwise on the CUDA cores in fp32.
 bool latent_attn_mma_ok(int rank, int rot);
 int launch_latent_attn(const LatentArgs& a, int T, cudaStream_t stream);      // the step's first T rows
 // A page of the bf16 cache: [64-column block][64 tokens][64 columns], rows of latent_row16 columns (rank + rot padded with zeros to
@@ -309,10 +313,63 @@ struct WindowTiles {
 // n_single: how many of the step's first rows are single tokens of running sequences (they precede the portions)
 int launch_window_attention(const WindowArgs& a, int T, int n_single, const WindowTiles& tm, cudaStream_t stream);
 
-// ---- latent_tc.cu: latent attention of the step's prompt portions on tcgen05, from the bf16 cache.  err: set when a wait inside
-// the kernel ran out (never, unless something is broken); mapped host memory or null
-bool latent_prefill_tc_ok(int rank, int rot);
-int launch_latent_prefill_tc(const LatentArgs& a, const WindowTiles& tm, int* err, cudaStream_t stream);
+// ---- paged16.cu / paged16_tc.cu: softmax attention over a paged bf16 cache (the serving form of latent attention and of window
+// attention without a window).  A page holds, per key head, `blocks` blocks of [64 tokens][64 columns] whose 128-byte rows have
+// their eight 16-byte chunks XOR-swizzled by the token (latent_chunk16): key_blocks blocks of keys (dim columns, zeros behind),
+// the values from block v_block on (vdim columns, zeros behind) — v_block 0: the values are the keys' first columns.
+struct Paged16Args {
+    const __nv_bfloat16* q = nullptr;             // [T][H][key_blocks * 64]: bf16(query * scale), zeros behind
+    const void* cache = nullptr;                  // [pages][G][blocks][64][64] bf16
+    const int *positions = nullptr, *seq_rows = nullptr, *page_table = nullptr;
+    int max_pages = 0;
+    int H = 0, G = 1, key_blocks = 0, v_block = 0, blocks = 0, dim = 0, vdim = 0;      // head h reads key head h / (H / G)
+    const float* sink = nullptr;                  // [H] or null: exp(sink) joins the softmax denominator
+    const float* gate = nullptr;                  // result *= sigmoid(gate[t * ldg + h]), or with gate_wide of [t * ldg + h * vdim + column]
+    int ldg = 0, gate_wide = 0;
+    float* out = nullptr;                         // [T][H][vdim]
+    void *out_hi = nullptr, *out_lo = nullptr;    // when given: the result as bf16 planes instead (out is not written)
+    float* part = nullptr;                        // as LatentArgs::part, vdim + 2 floats per share
+};
+Paged16Args latent_paged(const LatentArgs& a, int rank, int rot);
+// The step's queries, keys and values of a window-attention branch (norms, gains, biases, rotation, temperature) -> q16 and the cache.
+bool paged16_write_ok(const WindowArgs& a);
+int launch_paged16_write(const WindowArgs& a, __nv_bfloat16* q16, void* cache, int T, cudaStream_t stream);
+// single tokens of running sequences: the step's first T rows
+bool paged16_mma_ok(const Paged16Args& a);
+int launch_paged16_merge(const Paged16Args& a, int n_pairs, int n_split, cudaStream_t stream);      // shares in `part` -> result
+int launch_paged16_mma(const Paged16Args& a, int T, cudaStream_t stream);
+// the step's prompt portions on tcgen05.  err: set when a wait inside the kernel ran out (never, unless something is broken); mapped
+// host memory or null
+bool paged16_tc_ok(const Paged16Args& a);
+int launch_paged16_tc(const Paged16Args& a, const WindowTiles& tm, int* err, cudaStream_t stream);
+
+// ---- retention.cu: decay attention whose heads are normed apart and gated, with rotated queries and keys, in one pass
+// per request of one token (fp32, any sizes) or for prompt portions on tcgen05 (retention_tc_ok)
+struct RetentionArgs {
+    const float* proj = nullptr;                  // q, k (heads x dim), v, gate (heads x vdim) columns at o_q, o_k, o_v, o_g
+    int ldp = 0, o_q = 0, o_k = 0, o_v = 0, o_g = 0;
+    int heads = 0, dim = 0, vdim = 0, rot_dims = 0, rot_half = 0, gate_act = 0;      // gate_act 0: sigmoid, 1: silu
+    const float *rot_freq = nullptr, *decay = nullptr;
+    float k_scale = 1.f, eps = 0.f;
+    const int* positions = nullptr;
+    float* state = nullptr;
+    long long slot_stride = 0, s_off = 0;
+    const int *req_start = nullptr, *req_pos0 = nullptr, *req_slot = nullptr;
+    float* out = nullptr;                         // [T][heads * vdim]
+    void *out_hi = nullptr, *out_lo = nullptr;    // when given: the result as bf16 planes instead
+    // portions: room for the packed rows ([rows][heads] x retention_padded(dim), _padded(dim), _padded(vdim) bf16) and the states at the
+    // starts of runs (retention_ws_runs x heads x dim x vdim floats)
+    void *q16 = nullptr, *k16 = nullptr, *v16 = nullptr;
+    float* ws = nullptr;
+};
+bool retention_tc_ok(int dim, int vdim);
+bool retention_one_pass(int vdim);                // otherwise launch_retention_tc leaves o before norm and gate in out (fp32)
+int retention_padded(int n);
+int retention_ws_runs(int rows, int portions);
+// requests 0 .. n_req - 1, each one token of this step
+int launch_retention_step(const RetentionArgs& a, int n_req, cudaStream_t stream);
+// the portions tm lists: rows row0 .. row0 + rows - 1 of the step, requests first_req .. first_req + portions - 1
+int launch_retention_tc(const RetentionArgs& a, const WindowTiles& tm, int first_req, int row0, int rows, int portions, int* err, cudaStream_t stream);
 
 // S <- a_t S + b_t k_t v_t^T, o_t = S^T q_t per (request, head) over the request's rows in order; S [dim][vd] of head h at
 // state + slot * slot_stride + s_off + h * dim * vd, zero at a sequence's start (req_pos0 == 0).

@@ -638,29 +638,6 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(LatentArgs a, int n_pa
     }
 }
 
-// The shares of one (token, head) put together: one CTA each.
-__global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, int n_split) {
-    __shared__ float share[kLatentMaxSplits];              // what a share's sums count in the result
-    const int pair = blockIdx.x, rank = a.rank;
-    const float* p = a.part + (size_t)pair * n_split * (rank + 2);
-    if (threadIdx.x < 32) {
-        const int s = threadIdx.x;
-        const float ms = s < n_split ? p[(size_t)s * (rank + 2)] : -INFINITY;
-        const float m = warp_max(ms);
-        const float w = ms > -INFINITY ? expf(ms - m) : 0.f;
-        const float l = warp_sum(w > 0.f ? p[(size_t)s * (rank + 2) + 1] * w : 0.f);
-        if (s < n_split) share[s] = w * latent_finish(m, l, a, pair / a.H, pair % a.H);
-    }
-    __syncthreads();
-    for (int c = threadIdx.x; c < rank; c += blockDim.x) {
-        float v = 0.f;
-#pragma unroll
-        for (int s = 0; s < kLatentMaxSplits; ++s)
-            if (s < n_split && share[s] > 0.f) v = fmaf(p[(size_t)s * (rank + 2) + 2 + c], share[s], v);
-        a.out[(size_t)pair * rank + c] = v;
-    }
-}
-
 int launch_latent_prep(const LatentArgs& a, int T, cudaStream_t stream) {
     FT_REQUIRE(a.proj && a.norm_w && (a.cache || a.cache16) && (a.rot == 0 || (a.rot_freq && (a.qlat || a.qlat16) && a.rot % 2 == 0)),
                "latent prep: missing operands");
@@ -669,215 +646,30 @@ int launch_latent_prep(const LatentArgs& a, int T, cudaStream_t stream) {
     return 0;
 }
 
-// The serving form of the same attention on the tensor cores (mma.sync m16n8k16, bf16 operands, fp32 accumulation and
-// softmax): one CTA per (token, key share, group of 16 heads and, for latents beyond 256, group of value columns).  The 16 heads are the M rows of every product, so all rows
-// of a tile see the same keys and one mask.  Each of the four warps takes every fourth 16-key tile of the share: the tile
-// (16 latents from the bf16 copy of the cache) is copied into the warp's own double buffer with cp.async one tile ahead,
-// S = Q C^T (ldmatrix fragments of Q and of the tile), online softmax in registers, O += P C with the SAME tile read
-// through ldmatrix.trans — keys and values are one array.  The warps' (max, sum, O) are merged through shared memory.
-// kc 32-column pieces per row, the first vc of them hold the latent (the last of those may hold rotated columns too, whose sums
-// nobody reads).  A CTA sums VC <= 8 pieces (O is 4 * VC accumulator tiles per thread).
-__device__ __forceinline__ void cp_async16(void* dst_smem, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst_smem)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async_wait_1() { asm volatile("cp.async.wait_group 1;" ::: "memory"); }
-
-template <int VC>
-__global__ void __launch_bounds__(128)
-latent_attn_mma_kernel(LatentArgs a, int kc, int vc, int head_groups, int n_split) {
-    const int row = 32 * kc, RS = row * 2 + 16;            // row stride in bytes: 16 bytes of padding keep ldmatrix conflict-free
-    const int TILE = 16 * RS;
-    extern __shared__ __align__(16) uint8_t lat_smem[];
-    uint8_t* Qs = lat_smem;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    uint8_t* kbuf = lat_smem + TILE + (size_t)warp * 2 * TILE;
-    const int t = blockIdx.x, split = blockIdx.y, h0 = (blockIdx.z % head_groups) * 16;
-    const int v_first = (blockIdx.z / head_groups) * VC;   // first 32-column piece of the values this CTA sums
-    const int H = a.H, rank = a.rank;
-    const __nv_bfloat16* cache16 = (const __nv_bfloat16*)a.cache16;
-    for (int idx = threadIdx.x; idx < 16 * 4 * kc; idx += 128) {
-        const int r = idx / (4 * kc), ch = idx % (4 * kc);
-        uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (h0 + r < H) v = *reinterpret_cast<const uint4*>(a.qlat16 + ((size_t)t * H + h0 + r) * row + ch * 8);
-        *reinterpret_cast<uint4*>(Qs + r * RS + ch * 16) = v;
-    }
-    __syncthreads();
-    const int n_keys = a.positions[t] + 1;
-    int j_lo = 0, j_hi = n_keys;
-    if (n_split > 1) {
-        const int share = ((n_keys + n_split - 1) / n_split + kKvTile - 1) / kKvTile * kKvTile;
-        j_lo = min(split * share, n_keys);
-        j_hi = min(j_lo + share, n_keys);
-    }
-    const int* pt = a.page_table + (size_t)a.seq_rows[t] * a.max_pages;
-    const int n_tiles = (j_hi - j_lo + 15) / 16;
-    auto stage = [&](int tile, int buf) {
-        const int key0 = j_lo + tile * 16;
-        uint8_t* dst = kbuf + buf * TILE;
-        for (int i = lane; i < 16 * 4 * kc; i += 32) {          // 16 rows of 4 * kc 16-byte pieces
-            const int r = i / (4 * kc), ch = i % (4 * kc);
-            const int j = min(key0 + r, j_hi - 1);
-            cp_async16(dst + r * RS + ch * 16, cache16 + (size_t)pt[j / kKvTile] * kKvTile * row + latent_chunk16(j % kKvTile, ch));
-        }
-        cp_async_commit();
-    };
-    float o[4 * VC][4];
-#pragma unroll
-    for (int nt = 0; nt < 4 * VC; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
-    float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;      // rows g and g + 8
-    const int g = lane >> 2, tq = lane & 3;
-    const uint32_t q_addr = smem_u32(Qs) + ((lane & 7) + ((lane >> 3) & 1) * 8) * RS + (lane >> 4) * 16;
-    if (warp < n_tiles) stage(warp, 0);
-    for (int tile = warp, it = 0; tile < n_tiles; tile += 4, ++it) {
-        const int cur = it & 1;
-        if (tile + 4 < n_tiles) { stage(tile + 4, cur ^ 1); cp_async_wait_1(); }
-        else cp_async_wait_all();
-        __syncwarp();
-        const uint32_t kb = smem_u32(kbuf + cur * TILE);
-        float sc[2][4];
-#pragma unroll
-        for (int j = 0; j < 2; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
-#pragma unroll 2
-        for (int kp = 0; kp < kc; ++kp) {                        // 32 columns per round
-            uint32_t a0[4], a1[4];
-            ldmatrix_x4(q_addr + (kp * 4) * 16, a0[0], a0[1], a0[2], a0[3]);
-            ldmatrix_x4(q_addr + (kp * 4 + 2) * 16, a1[0], a1[1], a1[2], a1[3]);
-#pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                uint32_t b0, b1, b2, b3;
-                ldmatrix_x4(kb + (8 * j + (lane & 7)) * RS + (kp * 4 + (lane >> 3)) * 16, b0, b1, b2, b3);
-                mma_bf16_16816(sc[j], a0[0], a0[1], a0[2], a0[3], b0, b1);
-                mma_bf16_16816(sc[j], a1[0], a1[1], a1[2], a1[3], b2, b3);
-            }
-        }
-        const int key0 = j_lo + tile * 16 + 2 * tq;
-        float ta = -INFINITY, tb = -INFINITY;
-#pragma unroll
-        for (int j = 0; j < 2; ++j)
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                if (key0 + 8 * j + e >= j_hi) sc[j][e] = sc[j][2 + e] = -INFINITY;
-                ta = fmaxf(ta, sc[j][e]);
-                tb = fmaxf(tb, sc[j][2 + e]);
-            }
-        ta = fmaxf(ta, __shfl_xor_sync(0xffffffffu, ta, 1));
-        ta = fmaxf(ta, __shfl_xor_sync(0xffffffffu, ta, 2));
-        tb = fmaxf(tb, __shfl_xor_sync(0xffffffffu, tb, 1));
-        tb = fmaxf(tb, __shfl_xor_sync(0xffffffffu, tb, 2));
-        const float na = fmaxf(m_a, ta), nb = fmaxf(m_b, tb);      // finite: the tile's first key is never masked
-        const float alpha_a = expf(m_a - na), alpha_b = expf(m_b - nb);
-        float sa = 0.f, sb = 0.f;
-#pragma unroll
-        for (int j = 0; j < 2; ++j)
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                sc[j][e] = expf(sc[j][e] - na);
-                sc[j][2 + e] = expf(sc[j][2 + e] - nb);
-                sa += sc[j][e];
-                sb += sc[j][2 + e];
-            }
-        l_a = l_a * alpha_a + sa;
-        l_b = l_b * alpha_b + sb;
-        m_a = na;
-        m_b = nb;
-        const uint32_t pa0 = pack_bf16(sc[0][0], sc[0][1]), pa1 = pack_bf16(sc[0][2], sc[0][3]);
-        const uint32_t pa2 = pack_bf16(sc[1][0], sc[1][1]), pa3 = pack_bf16(sc[1][2], sc[1][3]);
-        const int vrow = ((lane >> 3) & 1) * 8 + (lane & 7);
-#pragma unroll
-        for (int np = 0; np < 2 * VC; ++np) {                    // 16 latent columns per round
-            if (v_first + (np >> 1) >= vc) break;                // the last group of columns may be a partial one
-            uint32_t b0, b1, b2, b3;
-            ldmatrix_x4_trans(kb + vrow * RS + (4 * v_first + 2 * np + (lane >> 4)) * 16, b0, b1, b2, b3);
-            o[2 * np][0] *= alpha_a; o[2 * np][1] *= alpha_a; o[2 * np][2] *= alpha_b; o[2 * np][3] *= alpha_b;
-            o[2 * np + 1][0] *= alpha_a; o[2 * np + 1][1] *= alpha_a; o[2 * np + 1][2] *= alpha_b; o[2 * np + 1][3] *= alpha_b;
-            mma_bf16_16816(o[2 * np], pa0, pa1, pa2, pa3, b0, b1);
-            mma_bf16_16816(o[2 * np + 1], pa0, pa1, pa2, pa3, b2, b3);
-        }
-        __syncwarp();
-    }
-    // the warp's record in its own (now idle) buffer: 16 rows of rank results, then max and sum
-    l_a += __shfl_xor_sync(0xffffffffu, l_a, 1);
-    l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
-    l_b += __shfl_xor_sync(0xffffffffu, l_b, 1);
-    l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
-    constexpr int COLS = 32 * VC, REC = COLS + 2;
-    float* rec = reinterpret_cast<float*>(kbuf);
-#pragma unroll
-    for (int nt = 0; nt < 4 * VC; ++nt) {
-        rec[g * REC + nt * 8 + 2 * tq] = o[nt][0];
-        rec[g * REC + nt * 8 + 2 * tq + 1] = o[nt][1];
-        rec[(g + 8) * REC + nt * 8 + 2 * tq] = o[nt][2];
-        rec[(g + 8) * REC + nt * 8 + 2 * tq + 1] = o[nt][3];
-    }
-    if (tq == 0) {
-        rec[g * REC + COLS] = m_a; rec[g * REC + COLS + 1] = l_a;
-        rec[(g + 8) * REC + COLS] = m_b; rec[(g + 8) * REC + COLS + 1] = l_b;
-    }
-    __syncthreads();
-    for (int idx = threadIdx.x; idx < 16 * COLS; idx += 128) {
-        const int r = idx / COLS, c = idx % COLS, col = 32 * v_first + c;
-        if (h0 + r >= H || col >= rank) continue;
-        float m = -INFINITY;
-#pragma unroll
-        for (int w = 0; w < 4; ++w) m = fmaxf(m, reinterpret_cast<const float*>(lat_smem + TILE + (size_t)w * 2 * TILE)[r * REC + COLS]);
-        float l = 0.f, v = 0.f;
-#pragma unroll
-        for (int w = 0; w < 4; ++w) {
-            const float* rw = reinterpret_cast<const float*>(lat_smem + TILE + (size_t)w * 2 * TILE) + r * REC;
-            if (rw[COLS] > -INFINITY) {
-                const float f = expf(rw[COLS] - m);
-                l = fmaf(rw[COLS + 1], f, l);
-                v = fmaf(rw[c], f, v);
-            }
-        }
-        const size_t pair = (size_t)t * H + h0 + r;
-        if (n_split > 1) {
-            float* p = a.part + (pair * n_split + split) * (rank + 2);
-            p[2 + col] = v;
-            if (col == 0) { p[0] = m; p[1] = l; }
-        } else {
-            a.out[pair * rank + col] = v * latent_finish(m, l, a, t, h0 + r);
-        }
-    }
-}
-
-int latent_attn_splits(int T, int H) {
-    const int pairs = T * H;
-    if (pairs >= kLatentSplitPairs) return 1;
-    return std::max(1, std::min(kLatentMaxSplits, kLatentSplitPairs / std::max(pairs, 1)));
-}
-
 int latent_row16(int rank, int rot) { return (rank + rot + 63) / 64 * 64; }
-// the query tile and the four warps' double-buffered key tiles, 16 rows each
-static size_t latent_mma_smem(int rank, int rot) { return (size_t)9 * 16 * (latent_row16(rank, rot) * 2 + 16); }
 // the serving form keeps latents of whole 32-column pieces in bf16; other sizes stay in fp32 on the CUDA cores
-bool latent_attn_mma_ok(int rank, int rot) { return rank >= 32 && rank % 32 == 0 && latent_mma_smem(rank, rot) <= 224 * 1024; }
+bool latent_attn_mma_ok(int rank, int rot) { 
+    LatentArgs one;
+    one.H = 1;
+    return rank >= 32 && rank % 32 == 0 && paged16_mma_ok(latent_paged(one, rank, rot));
+}
+
+// The latent cache as a paged bf16 cache: one key row for all heads, whose first columns are also the value.
+Paged16Args latent_paged(const LatentArgs& a, int rank, int rot) {
+    Paged16Args p;
+    p.q = a.qlat16; p.cache = a.cache16; p.positions = a.positions; p.seq_rows = a.seq_rows; p.page_table = a.page_table;
+    p.max_pages = a.max_pages; p.H = a.H; p.G = 1; p.key_blocks = p.blocks = latent_row16(rank, rot) / 64; p.v_block = 0; p.dim = rank + rot;
+    p.vdim = rank; p.sink = a.sink; p.out = a.out; p.part = a.part;
+    if (a.o_gate >= 0) { p.gate = a.proj + a.o_gate; p.ldg = a.ldp; }
+    return p;
+}
 
 int launch_latent_attn(const LatentArgs& a, int T, cudaStream_t stream) {
     const int n_pairs = T * a.H;
-    const int n_split = a.part ? latent_attn_splits(T, a.H) : 1;
+    const int n_split = a.part ? attn_splits(T, a.H) : 1;
     if (a.cache16 && latent_attn_mma_ok(a.rank, a.rot)) {
         FT_REQUIRE(a.qlat16, "latent attention: no bf16 queries");
-        const int vc = (a.rank + 31) / 32, kc = latent_row16(a.rank, a.rot) / 32;
-        const int groups = (vc + 7) / 8, per = (vc + groups - 1) / groups, hg = (a.H + 15) / 16;
-        const dim3 grid(T, n_split, hg * groups);
-        const size_t smem = latent_mma_smem(a.rank, a.rot);
-#define FT_LATM(VC_)                                                                                                        \
-    case VC_: {                                                                                                             \
-        static PerDeviceFlag attr;                                                                                          \
-        if (!attr.done()) {                                                                                                 \
-            FT_CHECK_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<VC_>, cudaFuncAttributeMaxDynamicSharedMemorySize,    \
-                                               224 * 1024));                                                                \
-            attr.mark();                                                                                                    \
-        }                                                                                                                   \
-        latent_attn_mma_kernel<VC_><<<grid, 128, smem, stream>>>(a, kc, vc, hg, n_split);                                   \
-        break;                                                                                                              \
-    }
-        switch (per) {
-            FT_LATM(1) FT_LATM(2) FT_LATM(3) FT_LATM(4) FT_LATM(5) FT_LATM(6) FT_LATM(7) FT_LATM(8)
-            default: break;
-        }
-#undef FT_LATM
+        return launch_paged16_mma(latent_paged(a, a.rank, a.rot), T, stream);
     } else {
         FT_REQUIRE(a.cache && a.qlat, "latent attention: no fp32 cache or queries");
         const int kd = a.rank + a.rot;
@@ -893,8 +685,7 @@ int launch_latent_attn(const LatentArgs& a, int T, cudaStream_t stream) {
     }
     FT_CHECK_CUDA(cudaGetLastError());
     if (n_split > 1) {
-        latent_merge_kernel<<<n_pairs, 128, 0, stream>>>(a, n_split);
-        FT_CHECK_CUDA(cudaGetLastError());
+        return launch_paged16_merge(latent_paged(a, a.rank, a.rot), n_pairs, n_split, stream);
     }
     return 0;
 }

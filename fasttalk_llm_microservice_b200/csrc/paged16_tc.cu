@@ -1,22 +1,24 @@
-// Latent attention of prompt portions on tcgen05 / TMEM: one shared key row per token, [latent | rotated part], whose first
-// columns are also its value.
+// Softmax attention of prompt portions over the paged bf16 cache (Paged16Args) on tcgen05 / TMEM.
 //
-// The query rows of a portion are its (token, head) pairs, token-major: every head reads the same keys, so 128 consecutive
-// pairs are the M rows of one tile whatever the number of heads.  One CTA = one such tile of one 64-token query tile of a request
-// (and, for latents beyond 256, one group of value columns).  Keys come page by page: a page of the bf16 cache is
-// [64-column block][64 tokens][64 columns] with the 16-byte chunks of a row XOR-swizzled by the token, which as it lies is the
-// K-major 128-byte-swizzled operand of the scores and, block by block, the MN-major one of the values — ONE bulk copy per page,
-// one array in shared memory for both products.
+// The query rows of a portion that read one key head are its (token, head of the group) pairs, token-major: they all read the same
+// keys, so 128 consecutive pairs are the M rows of one tile whatever the number of heads.  One CTA = one such tile of a run of 64
+// tokens of a request (128 tokens where 64 would leave a tile half empty) and one key head (and, for values beyond 256 columns, one
+// group of value columns).  Keys come page by page: a (page, key head) of the cache is [64-column block][64 tokens][64 columns]
+// with the 16-byte chunks of a row XOR-swizzled by the token, which as it lies is the K-major 128-byte-swizzled operand of the
+// scores and, block by block, the MN-major one of the values — bulk copies, no rearrangement; where the values are columns of the
+// keys (latent attention) ONE array in shared memory serves both products.
 //
-//   S  = Q C^T   tcgen05.mma  M128 N64, over all columns.  Q sits in TENSOR MEMORY as far as there is room (4 or
+//   S  = Q K^T   tcgen05.mma  M128 N64, over all key columns.  Q sits in TENSOR MEMORY as far as there is room (4 or
 //                8 blocks of 64 columns): with both operands in shared memory an M128 N64 product asks for more than the port's
 //                128 B/clk.  Further blocks lie in shared memory.
 //   softmax      4 warps, one thread per row, running maximum and sum in fp32, exp2; the rescale of O is lazy (the reference
 //                maximum moves only when it is exceeded by more than 2^8), P -> bf16 -> TMEM over the scores it came from
-//   O += P C     tcgen05.mma  M128 N64..256, the value columns of the same page
+//   O += P V     tcgen05.mma  M128 N64..256, the value blocks of the same page
 //
 // Scores have two buffers: the product of tile j + 2 is queued right behind P V of tile j and runs while tile j + 1 is in the
-// softmax.  TMEM: O 256 columns, S 2 x 64, Q 128 (+ 128 of O's when the latent has at most 128 columns).
+// softmax.  TMEM: O 256 columns, S 2 x 64, Q 128 (+ 128 of O's when a value has at most 128 columns).
+// Heads of at most 128 columns leave room for TWO CTAs per SM, which hide each other's waits better than a second buffer does:
+// TMEM O 128, S 64, Q 64 each.
 //
 // Warp roles (192 threads): 0 = page producer, 1 = TMEM owner and MMA issuer (one thread), 2..5 = query staging, softmax, epilogue.
 // Every wait has a limit; a CTA whose wait runs out marks `err`, lets its copies and products finish and returns.
@@ -32,28 +34,38 @@ constexpr int LT_THREADS = 192, LT_ROWS = 128;
 constexpr int LT_SLAB = kKvTile * 128;                 // bytes of one [64 tokens][64 columns] block of a page
 constexpr int LT_QBLK = LT_ROWS * 128;                 // bytes of one [128 rows][64 columns] block of Q in shared memory
 constexpr int LT_MAX_STAGES = 6;
-constexpr int LT_COL_O = 0, LT_COL_S = 256, LT_COL_Q = 384, LT_COL_Q2 = 128;
+constexpr int LT_COL_O = 0;
+// TMEM columns and score buffers of the two forms: one CTA per SM (512 columns), two (256 columns)
+template <int PER_SM> struct LtTmem { static constexpr int COLS = 512, S = 256, Q = 384, Q2 = 128, NBUF = 2, QB = 5; };
+template <> struct LtTmem<2> { static constexpr int COLS = 256, S = 128, Q = 192, Q2 = 0, NBUF = 1, QB = 2; };
 constexpr float LT_RESCALE = 8.f;                      // log2 units
 constexpr int LT_SPIN = 1 << 20;
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr int LT_OUT_LD = 36;                          // floats per row of a warp's output staging (32 columns)
 constexpr size_t LT_SMEM_MAX = 227 * 1024;
 
-struct LatentTcCfg {
-    int nblk, tq, stages, nv, groups;                  // 64-column blocks, blocks of Q in TMEM, ring, value columns per CTA, groups of them
+struct PagedTcCfg {
+    int nblk, tq, stages, nv, groups;                  // key blocks, blocks of Q in TMEM, ring, value columns per CTA, groups of them
+    int sblk;                                          // blocks of one stage: the keys and, where they are apart, the CTA's values
+    int span, grp;                                     // tokens per run, query heads per key head
+    int per_sm;                                        // CTAs per SM
     size_t smem;
 };
 
-bool latent_tc_cfg(int rank, int rot, LatentTcCfg& c) {
-    const int vblk = (rank + 63) / 64;
-    c.nblk = latent_row16(rank, rot) / 64;
+bool paged_tc_cfg(const Paged16Args& a, PagedTcCfg& c) {
+    const int vblk = (a.vdim + 63) / 64;
+    c.nblk = a.key_blocks;
     c.groups = (vblk + 3) / 4;
     c.nv = (vblk + c.groups - 1) / c.groups * 64;
     c.tq = std::min(c.nblk, c.nv <= 128 ? 8 : 4);
-    const size_t fixed = 1024 + (size_t)(c.nblk - c.tq) * LT_QBLK + 256;
-    if (fixed >= LT_SMEM_MAX) return false;
-    c.stages = (int)std::min<size_t>(LT_MAX_STAGES, (LT_SMEM_MAX - fixed) / ((size_t)c.nblk * LT_SLAB));
-    c.smem = fixed + (size_t)std::max(c.stages, 0) * c.nblk * LT_SLAB;
+    c.sblk = c.nblk + (a.v_block > 0 ? c.nv / 64 : 0);
+    c.grp = a.G > 0 ? std::max(a.H / a.G, 1) : 1;
+    c.span = c.grp % 2 == 0 ? kKvTile : 2 * kKvTile;
+    c.per_sm = c.nblk <= 2 && c.groups == 1 && c.nv <= 128 ? 2 : 1;
+    const size_t fixed = 1024 + (size_t)(c.nblk - c.tq) * LT_QBLK + 256, room = c.per_sm == 2 ? 112 * 1024 : LT_SMEM_MAX;
+    if (fixed >= room) return false;
+    c.stages = (int)std::min<size_t>(LT_MAX_STAGES, (room - fixed) / ((size_t)c.sblk * LT_SLAB));
+    c.smem = fixed + (size_t)std::max(c.stages, 0) * c.sblk * LT_SLAB;
     return c.stages >= 2;
 }
 
@@ -67,13 +79,16 @@ __device__ __forceinline__ bool wait_limited(uint64_t* bar, uint32_t parity, vol
     return false;
 }
 
-__global__ void __launch_bounds__(LT_THREADS, 1)
-latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs, int* err) {
+template <int PER_SM>
+__global__ void __launch_bounds__(LT_THREADS, PER_SM)
+paged16_tc_kernel(Paged16Args a, WindowTiles tm, PagedTcCfg cfg, int subs, int* err) {
+    using TM = LtTmem<PER_SM>;
+    constexpr int NBUF = TM::NBUF;                                     // score buffers
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-    const int page_bytes = cfg.nblk * LT_SLAB;
-    uint8_t* kv_s = smem;                                              // [stages][nblk] slabs
-    uint8_t* q_s = kv_s + (size_t)cfg.stages * page_bytes;             // blocks of Q that TMEM has no room for
+    const int stage_bytes = cfg.sblk * LT_SLAB;
+    uint8_t* kv_s = smem;                                              // [stages][sblk] slabs
+    uint8_t* q_s = kv_s + (size_t)cfg.stages * stage_bytes;             // blocks of Q that TMEM has no room for
     uint64_t* kv_full = reinterpret_cast<uint64_t*>(q_s + (size_t)(cfg.nblk - cfg.tq) * LT_QBLK);      // [6]
     uint64_t* kv_empty = kv_full + LT_MAX_STAGES;                      // [6] the products of the page have retired: O holds its share
     uint64_t* q_full = kv_empty + LT_MAX_STAGES;
@@ -84,16 +99,19 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
     volatile int* dead = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
     // the last tiles of a request see the most keys: they go first
-    const int lin = (int)gridDim.x - 1 - (int)blockIdx.x, tile = lin / subs, sub = lin % subs;
+    const int lin = ((int)gridDim.x - 1 - (int)blockIdx.x) / a.G, tile = lin / subs, sub = lin % subs, kv_head = blockIdx.x % a.G;
     const int req = tm.tile_req[tile], q0 = tm.tile_q0[tile];
+    if (q0 % cfg.span != 0) return;                                    // a run of two query tiles belongs to the first of them
     const int row0 = tm.req_q_start[req] + q0, p0 = tm.req_pos0[req] + q0;
-    const int ntok = min(kKvTile, tm.req_q_start[req + 1] - row0);
+    const int grp = cfg.grp, head0 = kv_head * grp;
+    const int ntok = min(cfg.span, tm.req_q_start[req + 1] - row0);
     const int first = sub * LT_ROWS;                                   // first (token, head) pair of this tile
-    if (first >= ntok * a.H) return;
-    const int last_tok = min((first + LT_ROWS - 1) / a.H, ntok - 1);
+    if (first >= ntok * grp) return;
+    const int last_tok = min((first + LT_ROWS - 1) / grp, ntok - 1);
     const int n_tiles = (p0 + last_tok) / kKvTile + 1;
     const int v0 = blockIdx.y * cfg.nv;                                // first value column
-    const int nv = min(cfg.nv, cfg.nblk * 64 - v0);
+    const bool apart = a.v_block > 0;                                  // values in blocks of their own
+    const int nv = min(cfg.nv, (a.vdim + 63) / 64 * 64 - v0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
     if (threadIdx.x == 0) {
@@ -108,7 +126,7 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
         fence_mbar_init();
     }
     if (warp == 1) {
-        tmem_alloc(tmem_slot, 512);
+        tmem_alloc(tmem_slot, TM::COLS);
         tmem_relinquish();
     }
     tc_fence_before();
@@ -131,9 +149,12 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
                     const int s = issued % cfg.stages, round = issued / cfg.stages;
                     ok = wait_limited(&kv_empty[s], (round & 1) ^ 1, dead);
                     if (ok) {
-                        mbar_expect_tx(&kv_full[s], page_bytes);
-                        tma_bulk_g2s(kv_s + (size_t)s * page_bytes, (const uint8_t*)a.cache16 + (size_t)page * page_bytes, page_bytes,
-                                     &kv_full[s], pol);
+                        const uint8_t* src = (const uint8_t*)a.cache + ((size_t)page * a.G + kv_head) * a.blocks * LT_SLAB;
+                        uint8_t* dst = kv_s + (size_t)s * stage_bytes;
+                        const int kb = cfg.nblk * LT_SLAB, vb = apart ? nv * (LT_SLAB / 64) : 0;
+                        mbar_expect_tx(&kv_full[s], kb + vb);
+                        tma_bulk_g2s(dst, src, kb, &kv_full[s], pol);
+                        if (apart) tma_bulk_g2s(dst + kb, src + (size_t)(a.v_block + (v0 >> 6)) * LT_SLAB, vb, &kv_full[s], pol);
                         ++issued;
                     }
                 }
@@ -149,15 +170,15 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
             const uint32_t idesc_qk = umma_idesc_bf16(LT_ROWS, kKvTile);
             const uint32_t idesc_pv = umma_idesc_bf16(LT_ROWS, nv) | (1u << 16);      // B is MN-major
             const uint32_t kv_addr = smem_u32(kv_s), q_addr = smem_u32(q_s);
-            auto stage_at = [&](int j) { return kv_addr + (uint32_t)(j % cfg.stages) * page_bytes; };
+            auto stage_at = [&](int j) { return kv_addr + (uint32_t)(j % cfg.stages) * stage_bytes; };
             auto issue_qk = [&](int j) {
-                const uint32_t k_addr = stage_at(j), d = tmem + LT_COL_S + (j & 1) * 64;
+                const uint32_t k_addr = stage_at(j), d = tmem + TM::S + (j % NBUF) * 64;
                 uint64_t b = umma_desc_k128(k_addr);
                 uint32_t acc = 0;
                 // whole blocks: columns beyond the row's end are zeros on both sides.  Little besides the products in here: one
                 // thread issues them all
                 for (int blk = 0; blk < cfg.tq; ++blk, b += LT_SLAB >> 4) {
-                    const uint32_t qa = tmem + (blk < 4 ? LT_COL_Q : LT_COL_Q2 - 128) + 32 * blk;
+                    const uint32_t qa = tmem + (blk < 4 ? TM::Q : TM::Q2 - 128) + 32 * blk;
 #pragma unroll
                     for (int k = 0; k < 4; ++k) { umma_f16_ts(d, qa + 8 * k, b + 2 * k, idesc_qk, acc); acc = 1; }
                 }
@@ -166,31 +187,31 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
 #pragma unroll
                     for (int k = 0; k < 4; ++k) umma_bf16(d, qd + 2 * k, b + 2 * k, idesc_qk, 1);
                 }
-                umma_commit(&s_full[j & 1]);
+                umma_commit(&s_full[j % NBUF]);
             };
             bool ok = wait_limited(q_full, 0, dead);
             tc_fence_after();
-            for (int j = 0; j < 2 && j < n_tiles && ok; ++j) {
+            for (int j = 0; j < NBUF && j < n_tiles && ok; ++j) {
                 ok = wait_limited(&kv_full[j % cfg.stages], (j / cfg.stages) & 1, dead);
                 tc_fence_after();
                 if (ok) issue_qk(j);
             }
-            const bool ahead = cfg.stages >= 3;                        // page j + 2 does not wait for the products of page j
+            const bool ahead = cfg.stages > NBUF;                      // page j + NBUF does not wait for the products of page j
             for (int j = 0; j < n_tiles && ok; ++j) {
-                if (ahead && j + 2 < n_tiles) ok = wait_limited(&kv_full[(j + 2) % cfg.stages], ((j + 2) / cfg.stages) & 1, dead);
-                ok = ok && wait_limited(&p_full[j & 1], (j >> 1) & 1, dead);      // P(j) written, S(j) consumed, O rescaled if needed
+                if (ahead && j + NBUF < n_tiles) ok = wait_limited(&kv_full[(j + NBUF) % cfg.stages], ((j + NBUF) / cfg.stages) & 1, dead);
+                ok = ok && wait_limited(&p_full[j % NBUF], (j / NBUF) & 1, dead);      // P(j) written, S(j) consumed, O rescaled if needed
                 if (!ok) break;
                 tc_fence_after();
-                const uint32_t p = tmem + LT_COL_S + (j & 1) * 64, v_addr = stage_at(j) + (v0 >> 6) * LT_SLAB;
+                const uint32_t p = tmem + TM::S + (j % NBUF) * 64, v_addr = stage_at(j) + (apart ? cfg.nblk : v0 >> 6) * LT_SLAB;
                 const uint64_t vd = umma_desc_mn128(v_addr);
 #pragma unroll
                 for (int k = 0; k < kKvTile / 16; ++k)
                     umma_f16_ts(tmem + LT_COL_O, p + 8 * k, vd + k * (2048 >> 4), idesc_pv, (j | k) != 0);
                 umma_commit(&kv_empty[j % cfg.stages]);
-                if (j + 2 < n_tiles) {
-                    if (!ahead) ok = wait_limited(&kv_full[(j + 2) % cfg.stages], ((j + 2) / cfg.stages) & 1, dead);
+                if (j + NBUF < n_tiles) {
+                    if (!ahead) ok = wait_limited(&kv_full[(j + NBUF) % cfg.stages], ((j + NBUF) / cfg.stages) & 1, dead);
                     tc_fence_after();
-                    if (ok) issue_qk(j + 2);                           // behind the product that reads P out of this buffer
+                    if (ok) issue_qk(j + NBUF);                           // behind the product that reads P out of this buffer
                 }
             }
             if (!ok) {
@@ -201,12 +222,12 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
     } else {
         // ---------------------------------------------------------------- queries in, softmax, results out (one thread per row)
         const int quarter = warp & 3, row = quarter * 32 + lane;       // TMEM lane == row
-        const int pair = first + row, tok = pair / a.H, head = pair % a.H;
+        const int pair = first + row, tok = pair / grp, head = head0 + pair % grp;
         const bool valid = tok < ntok;
         const int pos = valid ? p0 + tok : p0 + last_tok;
         const uint32_t lanes = tmem + ((uint32_t)(quarter * 32) << 16);
-        const uint4* q = reinterpret_cast<const uint4*>(a.qlat16 + ((size_t)row0 * a.H + pair) * (cfg.nblk * 64));
-        constexpr int QB = 5;                                          // blocks of a row on their way at a time
+        const uint4* q = reinterpret_cast<const uint4*>(a.q + ((size_t)(row0 + (valid ? tok : 0)) * a.H + head) * (cfg.nblk * 64));
+        constexpr int QB = TM::QB;                                        // blocks of a row on their way at a time
         for (int b0 = 0; b0 < cfg.nblk; b0 += QB) {
             uint4 v[QB][8];
 #pragma unroll
@@ -218,7 +239,7 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
             for (int i = 0; i < QB; ++i) {
                 const int blk = b0 + i;
                 if (blk < cfg.tq) {
-                    const uint32_t dst = lanes + (blk < 4 ? LT_COL_Q : LT_COL_Q2 - 128) + 32 * blk;
+                    const uint32_t dst = lanes + (blk < 4 ? TM::Q : TM::Q2 - 128) + 32 * blk;
                     tmem_st16(dst, &v[i][0].x);
                     tmem_st16(dst + 16, &v[i][4].x);
                 } else if (blk < cfg.nblk) {
@@ -237,10 +258,10 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
         float m_ref = -INFINITY, l_run = 0.f;                          // log2 units
         bool ok = true;
         for (int j = 0; j < n_tiles; ++j) {
-            ok = __all_sync(0xffffffffu, wait_limited(&s_full[j & 1], (j >> 1) & 1, dead));
+            ok = __all_sync(0xffffffffu, wait_limited(&s_full[j % NBUF], (j / NBUF) & 1, dead));
             if (!ok) break;
             tc_fence_after();
-            const uint32_t s_addr = lanes + LT_COL_S + (j & 1) * 64;
+            const uint32_t s_addr = lanes + TM::S + (j % NBUF) * 64;
             uint32_t sr[64];
 #pragma unroll
             for (int c = 0; c < 4; ++c) tmem_ld16_nowait(s_addr + 16 * c, sr + 16 * c);
@@ -295,7 +316,7 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
             l_run += (ps[0] + ps[1]) + (ps[2] + ps[3]);
             tc_fence_before();
             __syncwarp();
-            if (lane == 0) mbar_arrive(&p_full[j & 1]);
+            if (lane == 0) mbar_arrive(&p_full[j % NBUF]);
         }
         if (ok) ok = __all_sync(0xffffffffu, wait_limited(&kv_empty[(n_tiles - 1) % cfg.stages], ((n_tiles - 1) / cfg.stages) & 1, dead));
         if (ok) {
@@ -306,26 +327,75 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
                 f = exp2f(m_ref - top);
                 l_run = l_run * f + exp2f(s - top);
             }
-            if (a.o_gate >= 0 && valid) f *= 1.f / (1.f + expf(-a.proj[(size_t)(row0 + tok) * a.ldp + a.o_gate + head]));
+            if (a.gate && !a.gate_wide && valid) f *= 1.f / (1.f + expf(-a.gate[(size_t)(row0 + tok) * a.ldg + head]));
             f /= l_run;
             // 32 columns at a time through shared memory (the ring is idle now), so that a store covers whole 128-byte runs
             float* stage = reinterpret_cast<float*>(kv_s) + quarter * 32 * LT_OUT_LD;
-            float* out = a.out + ((size_t)row0 * a.H + first + quarter * 32) * a.rank + v0;
-            const int rows = min(32, ntok * a.H - first - quarter * 32);      // valid rows of this warp (may be <= 0)
-            for (int c = 0; c < nv && v0 + c < a.rank; c += 32) {
+            const int rows = min(32, ntok * grp - first - quarter * 32);      // valid rows of this warp (may be <= 0)
+            const bool v4 = (a.vdim & 3) == 0 && (a.ldg & 3) == 0;
+            __nv_bfloat16 *hi = (__nv_bfloat16*)a.out_hi, *lo = (__nv_bfloat16*)a.out_lo;
+            for (int c = 0; c < nv && v0 + c < a.vdim; c += 32) {
+                const int k = (lane & 7) * 4, col = v0 + c + k;               // the four columns this lane stores, of every fourth row
+                size_t at[8];
+                float4 g[8];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {                                 // all gate values on the way before the first is used
+                    const int r = i * 4 + (lane >> 3), pr = first + quarter * 32 + r;
+                    const size_t t = row0 + pr / grp, h = head0 + pr % grp;
+                    at[i] = (t * a.H + h) * a.vdim + col;
+                    g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                    if (a.gate && a.gate_wide && r < rows && col < a.vdim) {
+                        const float* gp = a.gate + t * a.ldg + h * a.vdim + col;
+                        if (v4) g[i] = *reinterpret_cast<const float4*>(gp);
+                        else {
+                            g[i].x = gp[0];
+                            if (col + 1 < a.vdim) g[i].y = gp[1];
+                            if (col + 2 < a.vdim) g[i].z = gp[2];
+                            if (col + 3 < a.vdim) g[i].w = gp[3];
+                        }
+                    }
+                }
                 uint32_t o[32];
+                __syncwarp();
                 tmem_ld16_nowait(lanes + LT_COL_O + c, o);
                 tmem_ld16_nowait(lanes + LT_COL_O + c + 16, o + 16);
                 tmem_ld_wait();
 #pragma unroll
-                for (int k = 0; k < 32; k += 4)
-                    *reinterpret_cast<float4*>(stage + lane * LT_OUT_LD + k) =
-                        make_float4(__uint_as_float(o[k]) * f, __uint_as_float(o[k + 1]) * f, __uint_as_float(o[k + 2]) * f, __uint_as_float(o[k + 3]) * f);
+                for (int q4 = 0; q4 < 32; q4 += 4)
+                    *reinterpret_cast<float4*>(stage + lane * LT_OUT_LD + q4) =
+                        make_float4(__uint_as_float(o[q4]) * f, __uint_as_float(o[q4 + 1]) * f, __uint_as_float(o[q4 + 2]) * f, __uint_as_float(o[q4 + 3]) * f);
                 __syncwarp();
 #pragma unroll
-                for (int r0 = 0; r0 < 32; r0 += 4) {
-                    const int r = r0 + (lane >> 3), k = (lane & 7) * 4;
-                    if (r < rows) *reinterpret_cast<float4*>(out + (size_t)r * a.rank + c + k) = *reinterpret_cast<const float4*>(stage + r * LT_OUT_LD + k);
+                for (int i = 0; i < 8; ++i) {
+                    const int r = i * 4 + (lane >> 3);
+                    if (r >= rows || col >= a.vdim) continue;
+                    float4 v = *reinterpret_cast<const float4*>(stage + r * LT_OUT_LD + k);
+                    if (a.gate && a.gate_wide) {
+                        v.x *= 1.f / (1.f + expf(-g[i].x)); v.y *= 1.f / (1.f + expf(-g[i].y));
+                        v.z *= 1.f / (1.f + expf(-g[i].z)); v.w *= 1.f / (1.f + expf(-g[i].w));
+                    }
+                    const float e[4] = {v.x, v.y, v.z, v.w};
+                    if (v4) {
+                        if (hi) {
+                            const uint32_t h0 = pack_bf16(v.x, v.y), h1 = pack_bf16(v.z, v.w);
+                            *reinterpret_cast<uint2*>(hi + at[i]) = make_uint2(h0, h1);
+                            *reinterpret_cast<uint2*>(lo + at[i]) = make_uint2(pack_bf16(v.x - bf16_lo(h0), v.y - bf16_hi(h0)),
+                                                                               pack_bf16(v.z - bf16_lo(h1), v.w - bf16_hi(h1)));
+                        } else {
+                            *reinterpret_cast<float4*>(a.out + at[i]) = v;
+                        }
+                    } else {
+#pragma unroll
+                        for (int q1 = 0; q1 < 4; ++q1)
+                            if (col + q1 < a.vdim) {
+                                if (hi) {
+                                    hi[at[i] + q1] = __float2bfloat16_rn(e[q1]);
+                                    lo[at[i] + q1] = __float2bfloat16_rn(e[q1] - __bfloat162float(hi[at[i] + q1]));
+                                } else {
+                                    a.out[at[i] + q1] = e[q1];
+                                }
+                            }
+                    }
                 }
                 __syncwarp();
             }
@@ -335,29 +405,31 @@ latent_prefill_tc_kernel(LatentArgs a, WindowTiles tm, LatentTcCfg cfg, int subs
     __syncthreads();
     if (warp == 1) {
         tc_fence_after();
-        tmem_dealloc(tmem, 512);
+        tmem_dealloc(tmem, TM::COLS);
     }
     if (threadIdx.x == 0 && *dead && err) *err = 1;
 }
 
 }  // namespace
 
-bool latent_prefill_tc_ok(int rank, int rot) {
-    LatentTcCfg c;
-    return latent_attn_mma_ok(rank, rot) && latent_tc_cfg(rank, rot, c);
+bool paged16_tc_ok(const Paged16Args& a) {
+    PagedTcCfg c;
+    return a.H >= 1 && a.G >= 1 && a.H % a.G == 0 && a.key_blocks >= 1 && a.vdim >= 1 && paged_tc_cfg(a, c);
 }
 
-int launch_latent_prefill_tc(const LatentArgs& a, const WindowTiles& tm, int* err, cudaStream_t stream) {
-    LatentTcCfg c;
-    FT_REQUIRE(a.cache16 && a.qlat16 && a.rank % 32 == 0 && latent_tc_cfg(a.rank, a.rot, c), "latent attention (tcgen05): sizes %d + %d do not fit", a.rank, a.rot);
+int launch_paged16_tc(const Paged16Args& a, const WindowTiles& tm, int* err, cudaStream_t stream) {
+    PagedTcCfg c;
+    FT_REQUIRE(a.cache && a.q && paged16_tc_ok(a) && paged_tc_cfg(a, c), "paged attention (tcgen05): sizes %d + %d do not fit", a.dim, a.vdim);
     static PerDeviceFlag attr;
     if (!attr.done()) {
-        FT_CHECK_CUDA(cudaFuncSetAttribute(latent_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LT_SMEM_MAX));
+        FT_CHECK_CUDA(cudaFuncSetAttribute(paged16_tc_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LT_SMEM_MAX));
+        FT_CHECK_CUDA(cudaFuncSetAttribute(paged16_tc_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024));
         attr.mark();
     }
-    const int subs = (kKvTile * a.H + LT_ROWS - 1) / LT_ROWS;
-    const dim3 grid(tm.n_tiles * subs, c.groups);
-    latent_prefill_tc_kernel<<<grid, LT_THREADS, c.smem, stream>>>(a, tm, c, subs, err);
+    const int subs = (c.span * c.grp + LT_ROWS - 1) / LT_ROWS;
+    const dim3 grid(tm.n_tiles * subs * a.G, c.groups);
+    if (c.per_sm == 2) paged16_tc_kernel<2><<<grid, LT_THREADS, c.smem, stream>>>(a, tm, c, subs, err);
+    else paged16_tc_kernel<1><<<grid, LT_THREADS, c.smem, stream>>>(a, tm, c, subs, err);
     FT_CHECK_CUDA(cudaGetLastError());
     return 0;
 }

@@ -915,7 +915,7 @@ class BranchDesc(C.Structure):
         ("q_gain", C.c_void_p), ("k_gain", C.c_void_p), ("out_gain", C.c_void_p),
         ("dt_rank", C.c_int), ("w_x", C.c_void_p), ("w_dt", C.c_void_p), ("x_rows", C.c_int),
         ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int), ("plain_qkv", C.c_int), ("head_norm", C.c_int), ("gate_act", C.c_int),
-        ("k_scale", C.c_float),
+        ("k_scale", C.c_float), ("tensor_cache", C.c_int),
     ]
 
 
@@ -1028,7 +1028,7 @@ def _pack_sandwich_layer(l: LayerSpec, w: Dict[str, torch.Tensor], p: str, d, W:
                 c.q_bias, c.k_bias = dev(w[m + "q.b"], f32).data_ptr(), dev(w[m + "k.b"], f32).data_ptr()
             if b.out_gate:
                 c.o_v, c.o_g = offs[f"{k}v"], offs[f"{k}g"]
-                c.qk_norm = 1
+                c.qk_norm = c.tensor_cache = 1
                 c.q_gain, c.k_gain = dev(w[m + "q.norm"], f32).data_ptr(), dev(w[m + "k.norm"], f32).data_ptr()
             if b.q_temp:
                 c.q_temp_coef, c.q_temp_every = b.q_temp[0], int(b.q_temp[1])

@@ -332,6 +332,8 @@ typedef struct {
     /* decay-attention options (see above) */
     int plain_qkv, head_norm, gate_act;
     float k_scale;
+    int tensor_cache;          /* window attention without window, cap, distance bias, kept or lent keys: 1 = the serving form keeps
+                                  queries, keys, values and softmax weights in bf16 and runs on the tensor cores */
 } ft_branch_desc;
 
 typedef struct {

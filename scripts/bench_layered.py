@@ -5,6 +5,7 @@
     python bench.py --design vonedra  [--sizes s,m] [--arms vonedra,gedelorn,gitozen,llama] [--steps K] [--warmup W]
     python bench.py --design lotinex  [--sizes s,m] [--arms lotinex,vonedra,gedelorn,llama] [--steps K] [--warmup W]
     python bench.py --design gedalix  [--sizes s,m,l] [--arms gedalix,gitozen,vonedra,llama] [--steps K] [--warmup W]
+    python bench.py --design fedutar  [--sizes s,m,l] [--arms fedutar,gedelorn,gedalix,llama] [--steps K] [--warmup W]
 
 For every size all arms get the same width, depth, heads x head size, active feed-forward width (top x expert ff =
 Llama's ffn) and vocabulary.  Gedelorn's closest relative in the framework is Gitozen (the same engine path: stacked
@@ -130,6 +131,23 @@ def gedalix_spec(name, c):
     return spec_from_config(cfg, name=f"gedalix-{name}")
 
 
+def fedutar_spec(name, c):
+    """Four sandwich layer runs, three layers: attention without positions (a quarter as many key heads, query temperature, output
+    gate) beside a retention of the same heads x head size; dense feed-forward with biases in the first layer, clipped experts in
+    the other two, of which the first is run twice."""
+    from fasttalk_llm_microservice_b200.layered import spec_from_config
+    W, H, D = c["width"], c["heads"], c["dim"]
+    mixer = {"left": {"dim": D, "heads": H, "kv_heads": max(1, H // 4), "q_temp": {"coef": 0.1, "every": 512}, "scale": D ** -0.5, "vdim": D},
+             "left_scale": 1.0, "right": {"decay": [1.0 - 2.0 ** -(3 + 7 * h / max(1, H - 1)) for h in range(H)], "dim": D, "heads": H,
+                                          "rot": {"base": 1e4, "dims": D}, "vdim": D}, "right_scale": 1.0}
+    dense = {"ff": c["top"] * c["ff"], "kind": "dense"}
+    moe = {"expert": {"ff": c["ff"], "limit": 7.0}, "kind": "moe", "router": {"experts": c["experts"], "top": c["top"]}}
+    layers = [{"type": "parallel", "mixer": mixer, "mlp": f} for f in (dense, moe, moe)]
+    cfg = {"architecture": "Fedutar", "embedding": {"scale": W ** 0.5}, "layers": layers, "logit_scale": W ** -0.5, "logit_softcap": 30.0,
+           "loop": {"start": 1, "stop": 2, "times": 2}, "norm": {"eps": 1e-6}, "vocab": c["vocab"], "width": W}
+    return spec_from_config(cfg, name=f"fedutar-{name}")
+
+
 def llama_spec(name, c):
     from fasttalk_llm_microservice_b200.model_spec import ModelSpec
     return ModelSpec(name=f"llama-{name}", hidden=c["width"], ffn=c["top"] * c["ff"], layers=len(c["order"]),
@@ -192,10 +210,11 @@ def run(args) -> None:
         c = SIZES[name]
         row = {"config": c}
         design = getattr(args, "design", "") or "gitozen"
-        default_arms = {"gedalix": "gedalix,gitozen,vonedra,llama", "lotinex": "lotinex,vonedra,gedelorn,llama", "vonedra": "vonedra,gedelorn,gitozen,llama",
+        default_arms = {"fedutar": "fedutar,gedelorn,gedalix,llama", "gedalix": "gedalix,gitozen,vonedra,llama", "lotinex": "lotinex,vonedra,gedelorn,llama", "vonedra": "vonedra,gedelorn,gitozen,llama",
                         "gedelorn": "gedelorn,gitozen,llama"}.get(design, "gitozen,llama")
         for arm in (getattr(args, "arms", "") or default_arms).split(","):
-            specs = {"gitozen": gitozen_spec, "gedelorn": gedelorn_spec, "vonedra": vonedra_spec, "lotinex": lotinex_spec, "gedalix": gedalix_spec}
+            specs = {"gitozen": gitozen_spec, "gedelorn": gedelorn_spec, "vonedra": vonedra_spec, "lotinex": lotinex_spec, "gedalix": gedalix_spec,
+                     "fedutar": fedutar_spec}
             if arm in specs:
                 spec = specs[arm](name, c)
                 w = init_layered(spec, seed=0, device="cuda")
