@@ -321,6 +321,9 @@ __device__ __forceinline__ float ex2_fast(float x) {
     return y;
 }
 
+// 1 / (1 + exp(-z)) in a handful of instructions (a few ulp), for epilogues that gate every element
+__device__ __forceinline__ float sigmoid_quick(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+
 // ------------------------------------------------------------------ mma.sync path (attention)
 __device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t& r0, uint32_t& r1,
                                             uint32_t& r2, uint32_t& r3) {

@@ -174,12 +174,14 @@ __global__ void __launch_bounds__(LTHREADS) linear_tile_kernel(LinearArgs a) {
 
 // ------------------------------------------------------------------ linear: few rows (decode)
 // A CTA of 8 warps owns 32 output columns (16 column pairs with the SwiGLU epilogue) of one problem and walks its rows
-// LROWS at a time: a 512-wide slice of those rows is staged in shared memory once and reused by every column, each warp
+// LROWS at a time: a slice of LKC columns of those rows is staged in shared memory once and reused by every column, each warp
 // streams the weights of its columns 16 bytes per lane per load, so the weights are read once per LROWS rows.
-constexpr int LROWS = 16, LKC = 512, LWARPS = 8;
+// LROWS x LKC: 16 x 512, or 4 x 2048 where a problem has a handful of rows at most (more warps per SM, fewer barriers).
+constexpr int LWARPS = 8, LROWS_MANY = 16, LROWS_FEW = 4, LSTAGE = 8192;
 
-template <bool PAIR, bool VEC>
+template <bool PAIR, bool VEC, int LROWS>
 __global__ void __launch_bounds__(LWARPS * 32) linear_rows_kernel(LinearArgs a) {
+    constexpr int LKC = LSTAGE / LROWS;
     constexpr int CPW = PAIR ? 2 : 4;                 // output columns per warp
     constexpr int WR = PAIR ? 2 * CPW : CPW;          // weight rows per warp
     __shared__ __align__(16) float sA[LROWS][LKC];
@@ -290,7 +292,7 @@ int launch_linear(const LinearArgs& a, int rows_bound, cudaStream_t stream) {
     FT_REQUIRE(a.K >= 1 && a.P >= 1, "linear: bad sizes");
     FT_REQUIRE(a.epi != LIN_SWIGLU_PAIR || (a.N & 1) == 0, "linear: the paired epilogue needs an even number of rows");
     // few rows per problem: one warp per output column, the weights stream once
-    const bool few = a.seg ? rows_bound <= 4 * LROWS : rows_bound <= 2 * LROWS;
+    const bool few = a.seg ? rows_bound <= 4 * LROWS_MANY : rows_bound <= 2 * LROWS_MANY;
     if (few) {
         const bool pair = a.epi == LIN_SWIGLU_PAIR;
         const int cols = pair ? a.N / 2 : a.N;
@@ -298,13 +300,21 @@ int launch_linear(const LinearArgs& a, int rows_bound, cudaStream_t stream) {
         const bool v8 = (a.K & 7) == 0 && (a.ldw & 7) == 0 && (a.lda & 3) == 0 && (a.a_col_stride & 3) == 0 &&
                         (a.w_stride & 7) == 0 && ((uintptr_t)a.A & 15) == 0 && ((uintptr_t)a.W & 15) == 0;
         dim3 grid((cols + per_cta - 1) / per_cta, a.P);
+        // rows per problem: M, or about rows_bound / P of a grouped launch
+        const bool handful = a.seg ? rows_bound <= 3 * a.P : a.M <= LROWS_FEW;
+#define FT_ROWS(PAIR_, VEC_)                                                                                             \
+    do {                                                                                                                 \
+        if (handful) linear_rows_kernel<PAIR_, VEC_, LROWS_FEW><<<grid, LWARPS * 32, 0, stream>>>(a);                    \
+        else linear_rows_kernel<PAIR_, VEC_, LROWS_MANY><<<grid, LWARPS * 32, 0, stream>>>(a);                           \
+    } while (0)
         if (pair) {
-            if (v8) linear_rows_kernel<true, true><<<grid, LWARPS * 32, 0, stream>>>(a);
-            else linear_rows_kernel<true, false><<<grid, LWARPS * 32, 0, stream>>>(a);
+            if (v8) FT_ROWS(true, true);
+            else FT_ROWS(true, false);
         } else {
-            if (v8) linear_rows_kernel<false, true><<<grid, LWARPS * 32, 0, stream>>>(a);
-            else linear_rows_kernel<false, false><<<grid, LWARPS * 32, 0, stream>>>(a);
+            if (v8) FT_ROWS(false, true);
+            else FT_ROWS(false, false);
         }
+#undef FT_ROWS
         FT_CHECK_CUDA(cudaGetLastError());
         return 0;
     }

@@ -254,6 +254,9 @@ paged16_tc_kernel(Paged16Args a, WindowTiles tm, PagedTcCfg cfg, int subs, int* 
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(q_full);
+        if (a.gate && a.gate_wide && valid)                            // the row's gate values on their way to L2 meanwhile
+            for (int c = 0; c < nv && v0 + c < a.vdim; c += 32)
+                asm volatile("prefetch.global.L2 [%0];" ::"l"(a.gate + (size_t)(row0 + tok) * a.ldg + (size_t)head * a.vdim + v0 + c));
 
         float m_ref = -INFINITY, l_run = 0.f;                          // log2 units
         bool ok = true;
@@ -334,24 +337,32 @@ paged16_tc_kernel(Paged16Args a, WindowTiles tm, PagedTcCfg cfg, int subs, int* 
             const int rows = min(32, ntok * grp - first - quarter * 32);      // valid rows of this warp (may be <= 0)
             const bool v4 = (a.vdim & 3) == 0 && (a.ldg & 3) == 0;
             __nv_bfloat16 *hi = (__nv_bfloat16*)a.out_hi, *lo = (__nv_bfloat16*)a.out_lo;
+            const bool wide = a.gate && a.gate_wide;
+            // where this lane's eight rows (every fourth) lie in the result and in the gate, from the run's first row
+            const size_t out0 = (size_t)row0 * a.H * a.vdim, gate0 = (size_t)row0 * a.ldg;
+            int at[8], gat[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const int pr = first + quarter * 32 + i * 4 + (lane >> 3), t = pr / grp, h = head0 + pr - t * grp;
+                at[i] = (t * a.H + h) * a.vdim;
+                gat[i] = t * a.ldg + h * a.vdim;
+            }
             for (int c = 0; c < nv && v0 + c < a.vdim; c += 32) {
                 const int k = (lane & 7) * 4, col = v0 + c + k;               // the four columns this lane stores, of every fourth row
-                size_t at[8];
                 float4 g[8];
+                if (wide) {
 #pragma unroll
-                for (int i = 0; i < 8; ++i) {                                 // all gate values on the way before the first is used
-                    const int r = i * 4 + (lane >> 3), pr = first + quarter * 32 + r;
-                    const size_t t = row0 + pr / grp, h = head0 + pr % grp;
-                    at[i] = (t * a.H + h) * a.vdim + col;
-                    g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-                    if (a.gate && a.gate_wide && r < rows && col < a.vdim) {
-                        const float* gp = a.gate + t * a.ldg + h * a.vdim + col;
-                        if (v4) g[i] = *reinterpret_cast<const float4*>(gp);
-                        else {
-                            g[i].x = gp[0];
-                            if (col + 1 < a.vdim) g[i].y = gp[1];
-                            if (col + 2 < a.vdim) g[i].z = gp[2];
-                            if (col + 3 < a.vdim) g[i].w = gp[3];
+                    for (int i = 0; i < 8; ++i) {                             // all gate values on the way before the first is used
+                        g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                        if (i * 4 + (lane >> 3) < rows && col < a.vdim) {
+                            const float* gp = a.gate + gate0 + gat[i] + col;
+                            if (v4) g[i] = *reinterpret_cast<const float4*>(gp);
+                            else {
+                                g[i].x = gp[0];
+                                if (col + 1 < a.vdim) g[i].y = gp[1];
+                                if (col + 2 < a.vdim) g[i].z = gp[2];
+                                if (col + 3 < a.vdim) g[i].w = gp[3];
+                            }
                         }
                     }
                 }
@@ -365,36 +376,51 @@ paged16_tc_kernel(Paged16Args a, WindowTiles tm, PagedTcCfg cfg, int subs, int* 
                     *reinterpret_cast<float4*>(stage + lane * LT_OUT_LD + q4) =
                         make_float4(__uint_as_float(o[q4]) * f, __uint_as_float(o[q4 + 1]) * f, __uint_as_float(o[q4 + 2]) * f, __uint_as_float(o[q4 + 3]) * f);
                 __syncwarp();
+                if (v4) {
+                    float4 v[8];
 #pragma unroll
-                for (int i = 0; i < 8; ++i) {
-                    const int r = i * 4 + (lane >> 3);
-                    if (r >= rows || col >= a.vdim) continue;
-                    float4 v = *reinterpret_cast<const float4*>(stage + r * LT_OUT_LD + k);
-                    if (a.gate && a.gate_wide) {
-                        v.x *= 1.f / (1.f + expf(-g[i].x)); v.y *= 1.f / (1.f + expf(-g[i].y));
-                        v.z *= 1.f / (1.f + expf(-g[i].z)); v.w *= 1.f / (1.f + expf(-g[i].w));
+                    for (int i = 0; i < 8; ++i) v[i] = *reinterpret_cast<const float4*>(stage + (i * 4 + (lane >> 3)) * LT_OUT_LD + k);
+                    if (wide) {
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) {
+                            v[i].x *= sigmoid_quick(g[i].x); v[i].y *= sigmoid_quick(g[i].y);
+                            v[i].z *= sigmoid_quick(g[i].z); v[i].w *= sigmoid_quick(g[i].w);
+                        }
                     }
-                    const float e[4] = {v.x, v.y, v.z, v.w};
-                    if (v4) {
-                        if (hi) {
-                            const uint32_t h0 = pack_bf16(v.x, v.y), h1 = pack_bf16(v.z, v.w);
-                            *reinterpret_cast<uint2*>(hi + at[i]) = make_uint2(h0, h1);
-                            *reinterpret_cast<uint2*>(lo + at[i]) = make_uint2(pack_bf16(v.x - bf16_lo(h0), v.y - bf16_hi(h0)),
-                                                                               pack_bf16(v.z - bf16_lo(h1), v.w - bf16_hi(h1)));
-                        } else {
-                            *reinterpret_cast<float4*>(a.out + at[i]) = v;
+                    if (hi) {
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) {
+                            const uint32_t h0 = pack_bf16(v[i].x, v[i].y), h1 = pack_bf16(v[i].z, v[i].w);
+                            const uint32_t l0 = pack_bf16(v[i].x - bf16_lo(h0), v[i].y - bf16_hi(h0)), l1 = pack_bf16(v[i].z - bf16_lo(h1), v[i].w - bf16_hi(h1));
+                            if (i * 4 + (lane >> 3) < rows && col < a.vdim) {
+                                *reinterpret_cast<uint2*>(hi + out0 + at[i] + col) = make_uint2(h0, h1);
+                                *reinterpret_cast<uint2*>(lo + out0 + at[i] + col) = make_uint2(l0, l1);
+                            }
                         }
                     } else {
 #pragma unroll
-                        for (int q1 = 0; q1 < 4; ++q1)
-                            if (col + q1 < a.vdim) {
-                                if (hi) {
-                                    hi[at[i] + q1] = __float2bfloat16_rn(e[q1]);
-                                    lo[at[i] + q1] = __float2bfloat16_rn(e[q1] - __bfloat162float(hi[at[i] + q1]));
-                                } else {
-                                    a.out[at[i] + q1] = e[q1];
-                                }
+                        for (int i = 0; i < 8; ++i)
+                            if (i * 4 + (lane >> 3) < rows && col < a.vdim) *reinterpret_cast<float4*>(a.out + out0 + at[i] + col) = v[i];
+                    }
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) {
+                        const int r = i * 4 + (lane >> 3);
+                        const float gv[4] = {g[i].x, g[i].y, g[i].z, g[i].w};
+#pragma unroll
+                        for (int q1 = 0; q1 < 4; ++q1) {
+                            if (r >= rows || col + q1 >= a.vdim) continue;
+                            float v = stage[r * LT_OUT_LD + k + q1];
+                            if (wide) v *= sigmoid_quick(gv[q1]);
+                            const size_t to = out0 + at[i] + col + q1;
+                            if (hi) {
+                                const __nv_bfloat16 b = __float2bfloat16_rn(v);
+                                hi[to] = b;
+                                lo[to] = __float2bfloat16_rn(v - __bfloat162float(b));
+                            } else {
+                                a.out[to] = v;
                             }
+                        }
                     }
                 }
                 __syncwarp();

@@ -27,7 +27,7 @@ constexpr int RT_RUN = 128, RT_THREADS = 256, RT_SPIN = 1 << 20;
 constexpr int RT_BLK = RT_RUN * 128;                    // bytes of one [128 tokens][64 columns] block
 
 __device__ __forceinline__ float gate_value(float g, int act) {
-    const float s = 1.f / (1.f + expf(-g));
+    const float s = sigmoid_quick(g);
     return act ? g * s : s;
 }
 __device__ __forceinline__ bool rt_wait(uint64_t* bar, uint32_t parity) {
@@ -237,6 +237,18 @@ __device__ __forceinline__ void split8(const float (&x)[8], uint4& hi, uint4& lo
     lo = make_uint4(l[0], l[1], l[2], l[3]);
 }
 
+// 128 rows x nv columns of TMEM -> tile (row stride ld floats): warps w and w + 4 share the lanes of a quarter
+__device__ __forceinline__ void tile_out(float* tile, int ld, uint32_t tmem, int nv, int warp, int lane) {
+    const int row = (warp & 3) * 32 + lane;
+    for (int c = (warp >> 2) * 16; c < nv; c += 32) {
+        float v[16];
+        tmem_ld16(tmem + ((uint32_t)((warp & 3) * 32) << 16) + c, v);
+#pragma unroll
+        for (int i = 0; i < 16; i += 4) *reinterpret_cast<float4*>(tile + row * ld + c + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+        __syncwarp();
+    }
+}
+
 // ------------------------------------------------------------------ what a run adds to the state
 // D[d][v] (TMEM, M = 128 key channels, N = up to 128 value columns) = Kd^T V over the run's tokens; both operands MN-major.
 __global__ void __launch_bounds__(RT_THREADS) retention_gain_kernel(RetentionArgs a, WindowTiles tm, int Dp, int Vp, int* err) {
@@ -304,29 +316,27 @@ __global__ void __launch_bounds__(RT_THREADS) retention_gain_kernel(RetentionArg
         umma_commit(&done);
     }
     __syncwarp();
-    const bool ok = rt_wait(&done, 0);
+    bool ok = rt_wait(&done, 0);
     tc_fence_after();
+    __syncwarp();
+    ok = __syncthreads_and(ok);
     if (ok) {
-        const int d = (warp & 3) * 32 + lane;
-        float* dst = a.ws + (((size_t)run.slot * a.heads + h) * a.dim + d) * a.vdim + v0;
-        const bool v4 = (a.vdim & 3) == 0;
-        __syncwarp();
-        for (int c = (warp >> 2) * 16; c < nv; c += 32) {
-            float v[16];
-            tmem_ld16(tmem + ((uint32_t)((warp & 3) * 32) << 16) + c, v);
-            if (d < a.dim) {
-                if (v4) {
-#pragma unroll
-                    for (int i = 0; i < 16; i += 4)
-                        if (v0 + c + i < a.vdim) *reinterpret_cast<float4*>(dst + c + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
-                } else {
-#pragma unroll
-                    for (int i = 0; i < 16; ++i) if (v0 + c + i < a.vdim) dst[c + i] = v[i];
-                }
+        // through shared memory (the operands have been read), so that a warp writes whole rows
+        const int ld = nv + 4;
+        float* tile = reinterpret_cast<float*>(smem);
+        tile_out(tile, ld, tmem, nv, warp, lane);
+        __syncthreads();
+        float* dst = a.ws + ((size_t)run.slot * a.heads + h) * a.dim * a.vdim + v0;
+        const int cols = min(nv, a.vdim - v0);
+        if ((a.vdim & 3) == 0) {
+            for (int i = tid; i < a.dim * (cols / 4); i += RT_THREADS) {
+                const int d = i / (cols / 4), c = i % (cols / 4) * 4;
+                *reinterpret_cast<float4*>(dst + (size_t)d * a.vdim + c) = *reinterpret_cast<const float4*>(tile + d * ld + c);
             }
-            __syncwarp();
+        } else {
+            for (int i = tid; i < a.dim * cols; i += RT_THREADS) dst[(size_t)(i / cols) * a.vdim + i % cols] = tile[i / cols * ld + i % cols];
         }
-    } else if (err) {
+    } else if (tid == 0 && err) {
         *err = 1;
     }
     tc_fence_before();
@@ -374,73 +384,35 @@ __global__ void __launch_bounds__(256) retention_carry_kernel(RetentionArgs a, W
 }
 
 // ------------------------------------------------------------------ the results of a run
-// TMEM: scores 0..127, their decayed values as planes (hi 128..191, lo 192..255), state part 256..383, run part 384..511.
-constexpr int RT_COL_S = 0, RT_COL_PH = 128, RT_COL_PL = 192, RT_COL_O1 = 256, RT_COL_O2 = 384;
-__global__ void __launch_bounds__(RT_THREADS, 1) retention_runs_kernel(RetentionArgs a, WindowTiles tm, int Dp, int Vp, int raw, int first_req, int* err) {
+// Two CTAs per SM.  TMEM: scores 0..127, over them their decayed values as planes (hi 0..63, lo 64..127), over those at last the
+// state's part; run's part 128..255.  Shared memory: q | k | v; the state's hi plane takes the place of k once the scores are there,
+// its lo plane that of v once the run's part is.
+constexpr int RT_COL_S = 0, RT_COL_PH = 0, RT_COL_PL = 64, RT_COL_O1 = 0, RT_COL_O2 = 128;
+__global__ void __launch_bounds__(RT_THREADS, 2) retention_runs_kernel(RetentionArgs a, WindowTiles tm, int Dp, int Vp, int raw, int first_req, int* err) {
     extern __shared__ uint8_t rr_raw[];
     __shared__ float pw[RT_RUN + 1];
-    __shared__ float sums[2][RT_RUN];
-    __shared__ uint64_t done[2];
+    __shared__ uint64_t done[3];
     __shared__ uint32_t tmem_slot;
     Run run;
-    // the longest-waiting rows of a long request need nothing from one another: any order
     if (!find_run(tm, blockIdx.x, run)) return;
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(rr_raw) + 1023) & ~uintptr_t(1023));
     const int db = Dp / 64, h = blockIdx.y, v0 = blockIdx.z * 128, nv = min(128, Vp - v0), vb = nv / 64, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int sblk = Dp * 128;                           // bytes of one [Dp channels][64 columns] block of the state
-    uint8_t *q_s = smem, *k_s = q_s + db * RT_BLK, *v_s = k_s + db * RT_BLK, *s_hi = v_s + vb * RT_BLK, *s_lo = s_hi + vb * sblk;
+    uint8_t *q_s = smem, *k_s = q_s + db * RT_BLK, *v_s = k_s + db * RT_BLK, *s_hi = k_s, *s_lo = v_s;
     const bool carried = a.req_pos0[first_req + run.portion] > 0 || run.q0 > 0;      // otherwise the state it starts from is zero
     if (tid == 0) {
-        mbar_init(&done[0], 1);
-        mbar_init(&done[1], 1);
+        for (int i = 0; i < 3; ++i) mbar_init(&done[i], 1);
         fence_mbar_init();
     }
     if (warp == 0) {
-        tmem_alloc(&tmem_slot, 512);
+        tmem_alloc(&tmem_slot, 256);
         tmem_relinquish();
     }
-    if (tid <= RT_RUN) pw[tid] = powf(a.decay[h], (float)tid);
     const size_t hd = (size_t)a.heads * Dp;
     stage_rows(q_s, (const __nv_bfloat16*)a.q16 + ((size_t)run.row * a.heads + h) * Dp, hd, db, run.n);
     stage_rows(k_s, (const __nv_bfloat16*)a.k16 + ((size_t)run.row * a.heads + h) * Dp, hd, db, run.n);
     stage_rows(v_s, (const __nv_bfloat16*)a.v16 + ((size_t)run.row * a.heads + h) * Vp + v0, (size_t)a.heads * Vp, vb, run.n);
-    if (carried) {
-        const float* ws = a.ws + ((size_t)run.slot * a.heads + h) * a.dim * a.vdim;
-        const bool v4 = (a.vdim & 3) == 0;
-        const int ch = tid & 7, d0 = tid >> 3;
-        constexpr int ND = 4;                            // channels of a block on their way at a time
-        for (int b = 0; b < vb; ++b)
-            for (int dd = d0; dd < Dp; dd += ND * (RT_THREADS / 8)) {      // Dp: a multiple of 64, RT_THREADS / 8 = 32
-                const int c = v0 + b * 64 + ch * 8;
-                float x[ND][8];
-#pragma unroll
-                for (int i = 0; i < ND; ++i) {
-                    const int d = dd + i * (RT_THREADS / 8);
-#pragma unroll
-                    for (int e = 0; e < 8; ++e) x[i][e] = 0.f;
-                    if (d < a.dim) {
-                        const float* src = ws + (size_t)d * a.vdim + c;
-                        if (v4) {
-                            if (c < a.vdim) { const float4 t = *reinterpret_cast<const float4*>(src); x[i][0] = t.x; x[i][1] = t.y; x[i][2] = t.z; x[i][3] = t.w; }
-                            if (c + 4 < a.vdim) { const float4 t = *reinterpret_cast<const float4*>(src + 4); x[i][4] = t.x; x[i][5] = t.y; x[i][6] = t.z; x[i][7] = t.w; }
-                        } else {
-#pragma unroll
-                            for (int e = 0; e < 8; ++e) if (c + e < a.vdim) x[i][e] = src[e];
-                        }
-                    }
-                }
-#pragma unroll
-                for (int i = 0; i < ND; ++i) {
-                    const int d = dd + i * (RT_THREADS / 8);
-                    if (d >= Dp) break;
-                    uint4 hi, lo;
-                    split8(x[i], hi, lo);
-                    const int at = b * sblk + d * 128 + ((ch ^ (d & 7)) << 4);
-                    *reinterpret_cast<uint4*>(s_hi + at) = hi;
-                    *reinterpret_cast<uint4*>(s_lo + at) = lo;
-                }
-            }
-    }
+    if (tid <= RT_RUN) pw[tid] = powf(a.decay[h], (float)tid);
     rt_landed();
     fence_proxy_async();
     tc_fence_before();
@@ -454,8 +426,117 @@ __global__ void __launch_bounds__(RT_THREADS, 1) retention_runs_kernel(Retention
 #pragma unroll
             for (int k = 0; k < 4; ++k) umma_bf16(tmem + RT_COL_S, qd + 2 * k, kd + 2 * k, idesc_qk, (b | k) != 0);
         }
-        if (carried) {
-            const uint32_t idesc_qs = umma_idesc_bf16(RT_RUN, nv) | (1u << 16);      // B MN-major
+        umma_commit(&done[0]);
+    }
+    __syncwarp();
+    bool ok = rt_wait(&done[0], 0);
+    tc_fence_after();
+    __syncwarp();
+    const int i_row = (warp & 3) * 32 + lane, col_half = warp >> 2;      // TMEM lane == row of the run
+    const uint32_t lanes = tmem + ((uint32_t)((warp & 3) * 32) << 16);
+    // scores times decay^(i - j), zero above the diagonal
+    uint32_t ph[2][16], pl[2][16];
+    if (ok) {
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+            const int col = col_half * 64 + x * 32;
+            uint32_t s[32];
+            tmem_ld16_nowait(lanes + RT_COL_S + col, s);
+            tmem_ld16_nowait(lanes + RT_COL_S + col + 16, s + 16);
+            tmem_ld_wait();
+#pragma unroll
+            for (int e = 0; e < 16; ++e) {
+                const int j = col + 2 * e;
+                const float u = j <= i_row ? __uint_as_float(s[2 * e]) * pw[i_row - j] : 0.f;
+                const float v = j + 1 <= i_row ? __uint_as_float(s[2 * e + 1]) * pw[i_row - j - 1] : 0.f;
+                ph[x][e] = pack_bf16(u, v);
+                pl[x][e] = pack_bf16(u - bf16_lo(ph[x][e]), v - bf16_hi(ph[x][e]));
+            }
+        }
+    }
+    tc_fence_before();
+    ok = __syncthreads_and(ok);                          // every score has been read
+    tc_fence_after();
+    if (ok) {
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+            tmem_st16(lanes + RT_COL_PH + col_half * 32 + x * 16, ph[x]);
+            tmem_st16(lanes + RT_COL_PL + col_half * 32 + x * 16, pl[x]);
+        }
+        tmem_st_wait();
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    if (ok && tid == 0) {
+        const uint32_t idesc_pv = umma_idesc_bf16(RT_RUN, nv) | (1u << 16);      // B MN-major
+        const uint64_t vd = umma_desc_mn128(smem_u32(v_s), RT_BLK);
+        const int steps = (run.n + 15) / 16;
+        for (int k = 0; k < steps; ++k) {
+            umma_f16_ts(tmem + RT_COL_O2, tmem + RT_COL_PH + 8 * k, vd + k * (2048 >> 4), idesc_pv, k > 0);
+            umma_f16_ts(tmem + RT_COL_O2, tmem + RT_COL_PL + 8 * k, vd + k * (2048 >> 4), idesc_pv, 1);
+        }
+        umma_commit(&done[1]);
+    }
+    __syncwarp();
+    // the state meanwhile: hi plane to its place, lo plane in registers until the values have been read
+    constexpr int ND = 4, ST = RT_THREADS / 8;           // channels per thread and block, their stride
+    const int ch = tid & 7, d0 = tid >> 3;
+    uint4 lo[2][ND];
+    if (carried) {
+        const float* ws = a.ws + ((size_t)run.slot * a.heads + h) * a.dim * a.vdim;
+        const bool v4 = (a.vdim & 3) == 0;
+#pragma unroll
+        for (int b = 0; b < 2; ++b) {
+            if (b >= vb) break;
+            const int c = v0 + b * 64 + ch * 8;
+            float x[ND][8];
+#pragma unroll
+            for (int i = 0; i < ND; ++i) {
+                const int d = d0 + i * ST;
+#pragma unroll
+                for (int e = 0; e < 8; ++e) x[i][e] = 0.f;
+                if (d < a.dim) {
+                    const float* src = ws + (size_t)d * a.vdim + c;
+                    if (v4) {
+                        if (c < a.vdim) { const float4 t = *reinterpret_cast<const float4*>(src); x[i][0] = t.x; x[i][1] = t.y; x[i][2] = t.z; x[i][3] = t.w; }
+                        if (c + 4 < a.vdim) { const float4 t = *reinterpret_cast<const float4*>(src + 4); x[i][4] = t.x; x[i][5] = t.y; x[i][6] = t.z; x[i][7] = t.w; }
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) if (c + e < a.vdim) x[i][e] = src[e];
+                    }
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < ND; ++i) {
+                const int d = d0 + i * ST;
+                uint4 hi;
+                split8(x[i], hi, lo[b][i]);
+                if (d < Dp) *reinterpret_cast<uint4*>(s_hi + b * sblk + d * 128 + ((ch ^ (d & 7)) << 4)) = hi;
+            }
+        }
+    }
+    if (ok) ok = rt_wait(&done[1], 0);
+    tc_fence_after();
+    __syncwarp();
+    if (carried) {                                       // the same for the whole CTA
+        if (ok) {
+#pragma unroll
+            for (int b = 0; b < 2; ++b) {
+                if (b >= vb) break;
+#pragma unroll
+                for (int i = 0; i < ND; ++i) {
+                    const int d = d0 + i * ST;
+                    if (d < Dp) *reinterpret_cast<uint4*>(s_lo + b * sblk + d * 128 + ((ch ^ (d & 7)) << 4)) = lo[b][i];
+                }
+            }
+        }
+        fence_proxy_async();
+        tc_fence_before();
+        ok = __syncthreads_and(ok);
+        tc_fence_after();
+        if (ok && tid == 0) {
+            const uint32_t idesc_qs = umma_idesc_bf16(RT_RUN, nv) | (1u << 16);
             const uint64_t sh = umma_desc_mn128(smem_u32(s_hi), sblk), sl = umma_desc_mn128(smem_u32(s_lo), sblk);
             for (int b = 0; b < db; ++b) {
                 const uint64_t qd = umma_desc_k128(smem_u32(q_s + b * RT_BLK));
@@ -466,129 +547,87 @@ __global__ void __launch_bounds__(RT_THREADS, 1) retention_runs_kernel(Retention
                     umma_bf16(tmem + RT_COL_O1, qd + 2 * k, sl + off, idesc_qs, 1);
                 }
             }
+            umma_commit(&done[2]);
         }
-        umma_commit(&done[0]);
+        __syncwarp();
+        if (ok) ok = rt_wait(&done[2], 0);
+        tc_fence_after();
+        __syncwarp();
     }
-    __syncwarp();
-    bool ok = rt_wait(&done[0], 0);
-    tc_fence_after();
-    __syncwarp();
-    const int i_row = (warp & 3) * 32 + lane, col_half = warp >> 2;      // TMEM lane == row of the run
-    const uint32_t lanes = tmem + ((uint32_t)((warp & 3) * 32) << 16);
-    // scores times decay^(i - j), zero above the diagonal: 32 columns at a time
-    if (ok) {
-#pragma unroll
-        for (int c0 = 0; c0 < 64; c0 += 32) {
-            const int col = col_half * 64 + c0;
-            uint32_t s[32], ph[16], pl[16];
-            tmem_ld16_nowait(lanes + RT_COL_S + col, s);
-            tmem_ld16_nowait(lanes + RT_COL_S + col + 16, s + 16);
-            tmem_ld_wait();
-#pragma unroll
-            for (int e = 0; e < 16; ++e) {
-                const int j = col + 2 * e;
-                const float x = j <= i_row ? __uint_as_float(s[2 * e]) * pw[i_row - j] : 0.f;
-                const float y = j + 1 <= i_row ? __uint_as_float(s[2 * e + 1]) * pw[i_row - j - 1] : 0.f;
-                ph[e] = pack_bf16(x, y);
-                pl[e] = pack_bf16(x - bf16_lo(ph[e]), y - bf16_hi(ph[e]));
-            }
-            tmem_st16(lanes + RT_COL_PH + col / 2, ph);
-            tmem_st16(lanes + RT_COL_PL + col / 2, pl);
-        }
-        tmem_st_wait();
-    }
-    tc_fence_before();
-    ok = __syncthreads_and(ok);
-    tc_fence_after();
-    if (ok && tid == 0) {
-        const uint32_t idesc_pv = umma_idesc_bf16(RT_RUN, nv) | (1u << 16);
-        const uint64_t vd = umma_desc_mn128(smem_u32(v_s), RT_BLK);
-        const int steps = (run.n + 15) / 16;
-        for (int k = 0; k < steps; ++k) {
-            umma_f16_ts(tmem + RT_COL_O2, tmem + RT_COL_PH + 8 * k, vd + k * (2048 >> 4), idesc_pv, k > 0);
-            umma_f16_ts(tmem + RT_COL_O2, tmem + RT_COL_PL + 8 * k, vd + k * (2048 >> 4), idesc_pv, 1);
-        }
-        umma_commit(&done[1]);
-    }
-    __syncwarp();
-    if (ok) ok = rt_wait(&done[1], 0);
-    tc_fence_after();
-    __syncwarp();
     ok = __syncthreads_and(ok);
     if (ok) {
-        const bool in = i_row < run.n;
-        const int row = tm.req_q_start[0] + run.row + (in ? i_row : 0);
+        // through shared memory (all operands have been read): then a warp per row
+        const int ld = nv + 4;
+        float* tile = reinterpret_cast<float*>(smem);
         const float after = pw[min(i_row + 1, RT_RUN)];
-        constexpr int PIECES = 4;                        // a thread's 16-column pieces: half of at most 128 columns
-        float o[PIECES][16];
-        float ss = 0.f;
-        const int half = nv / 2;                         // columns of this warp: col_half * half .. + half (32 or 64)
-#pragma unroll
-        for (int p = 0; p < PIECES; ++p) {
-            if (p * 16 >= half) break;                   // uniform
-            const int c = col_half * half + p * 16;
-            float x[16];
-            tmem_ld16(lanes + RT_COL_O2 + c, o[p]);
+        for (int c = col_half * 16; c < nv; c += 32) {
+            float o[16], x[16];
+            tmem_ld16(lanes + RT_COL_O2 + c, o);
             if (carried) {
                 tmem_ld16(lanes + RT_COL_O1 + c, x);
 #pragma unroll
-                for (int i = 0; i < 16; ++i) o[p][i] = fmaf(after, x[i], o[p][i]);
+                for (int i = 0; i < 16; ++i) o[i] = fmaf(after, x[i], o[i]);
             }
 #pragma unroll
-            for (int i = 0; i < 16; ++i) ss = fmaf(o[p][i], o[p][i], ss);      // columns beyond vdim are zero
+            for (int i = 0; i < 16; i += 4) *reinterpret_cast<float4*>(tile + i_row * ld + c + i) = make_float4(o[i], o[i + 1], o[i + 2], o[i + 3]);
+            __syncwarp();
         }
-        float rr = 1.f;
-        if (!raw) {
-            sums[col_half][i_row] = ss;
-            __syncthreads();
-            rr = 1.f / sqrtf((sums[0][i_row] + sums[1][i_row]) / (float)a.vdim + a.eps);
-        }
-        __nv_bfloat16 *hi = (__nv_bfloat16*)a.out_hi, *lo = (__nv_bfloat16*)a.out_lo;
-        const bool w16 = (a.vdim & 15) == 0 && (a.ldp & 3) == 0 && (a.o_g & 3) == 0;
-        const float* gate = a.proj + (size_t)row * a.ldp + a.o_g + h * a.vdim;
-        const size_t base = ((size_t)row * a.heads + h) * a.vdim;
+        __syncthreads();
+        __nv_bfloat16 *oh = (__nv_bfloat16*)a.out_hi, *ol = (__nv_bfloat16*)a.out_lo;
+        const bool v4 = (a.vdim & 3) == 0 && (a.ldp & 3) == 0 && (a.o_g & 3) == 0;
+        const int row0 = tm.req_q_start[0] + run.row, cols = min(nv, a.vdim - v0);
+        constexpr int NR = 4;                            // rows of a warp on their way at a time
+        for (int r0 = warp; r0 < run.n; r0 += NR * (RT_THREADS / 32)) {
+            if (v4) {
+                float4 g[NR];
+                const int c = lane * 4;
 #pragma unroll
-        for (int p = 0; p < PIECES; ++p) {
-            if (p * 16 >= half) break;
-            const int c = v0 + col_half * half + p * 16;
-            if (!in || c >= a.vdim) continue;
-            if (w16) {
-                if (!raw) {
-                    float g[16];
-#pragma unroll
-                    for (int i = 0; i < 16; i += 4) {
-                        const float4 t = *reinterpret_cast<const float4*>(gate + c + i);
-                        g[i] = t.x; g[i + 1] = t.y; g[i + 2] = t.z; g[i + 3] = t.w;
-                    }
-#pragma unroll
-                    for (int i = 0; i < 16; ++i) o[p][i] *= rr * gate_value(g[i], a.gate_act);
+                for (int i = 0; i < NR; ++i) {
+                    const int r = r0 + i * (RT_THREADS / 32);
+                    g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                    if (!raw && r < run.n && c < cols) g[i] = *reinterpret_cast<const float4*>(a.proj + (size_t)(row0 + r) * a.ldp + a.o_g + h * a.vdim + c);
                 }
-                if (hi && !raw) {
 #pragma unroll
-                    for (int i = 0; i < 16; i += 8) {
-                        const float x[8] = {o[p][i], o[p][i + 1], o[p][i + 2], o[p][i + 3], o[p][i + 4], o[p][i + 5], o[p][i + 6], o[p][i + 7]};
-                        uint4 vh, vl;
-                        split8(x, vh, vl);
-                        *reinterpret_cast<uint4*>(hi + base + c + i) = vh;
-                        *reinterpret_cast<uint4*>(lo + base + c + i) = vl;
+                for (int i = 0; i < NR; ++i) {
+                    const int r = r0 + i * (RT_THREADS / 32);
+                    if (r >= run.n) break;
+                    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+                    if (c < cols) v = *reinterpret_cast<const float4*>(tile + r * ld + c);
+                    const size_t at = ((size_t)(row0 + r) * a.heads + h) * a.vdim + v0 + c;
+                    if (!raw) {
+                        const float rr = 1.f / sqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / (float)a.vdim + a.eps);
+                        v.x *= rr * gate_value(g[i].x, a.gate_act); v.y *= rr * gate_value(g[i].y, a.gate_act);
+                        v.z *= rr * gate_value(g[i].z, a.gate_act); v.w *= rr * gate_value(g[i].w, a.gate_act);
                     }
-                } else {
-#pragma unroll
-                    for (int i = 0; i < 16; i += 4)
-                        *reinterpret_cast<float4*>(a.out + base + c + i) = make_float4(o[p][i], o[p][i + 1], o[p][i + 2], o[p][i + 3]);
+                    if (c >= cols) continue;
+                    if (oh && !raw) {
+                        const uint32_t h0 = pack_bf16(v.x, v.y), h1 = pack_bf16(v.z, v.w);
+                        *reinterpret_cast<uint2*>(oh + at) = make_uint2(h0, h1);
+                        *reinterpret_cast<uint2*>(ol + at) = make_uint2(pack_bf16(v.x - bf16_lo(h0), v.y - bf16_hi(h0)),
+                                                                        pack_bf16(v.z - bf16_lo(h1), v.w - bf16_hi(h1)));
+                    } else {
+                        *reinterpret_cast<float4*>(a.out + at) = v;
+                    }
                 }
             } else {
-#pragma unroll
-                for (int i = 0; i < 16; ++i) {
-                    if (c + i >= a.vdim) continue;
-                    float v = o[p][i];
-                    if (!raw) v *= rr * gate_value(gate[c + i], a.gate_act);
-                    if (hi && !raw) {
-                        const __nv_bfloat16 b = __float2bfloat16_rn(v);
-                        hi[base + c + i] = b;
-                        lo[base + c + i] = __float2bfloat16_rn(v - __bfloat162float(b));
-                    } else {
-                        a.out[base + c + i] = v;
+                for (int i = 0; i < NR; ++i) {
+                    const int r = r0 + i * (RT_THREADS / 32);
+                    if (r >= run.n) break;
+                    float ss = 0.f;
+                    for (int c = lane; c < cols; c += 32) ss = fmaf(tile[r * ld + c], tile[r * ld + c], ss);
+                    const float rr = raw ? 1.f : 1.f / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
+                    const float* gate = a.proj + (size_t)(row0 + r) * a.ldp + a.o_g + h * a.vdim;
+                    for (int c = lane; c < cols; c += 32) {
+                        float v = tile[r * ld + c];
+                        if (!raw) v *= rr * gate_value(gate[c], a.gate_act);
+                        const size_t at = ((size_t)(row0 + r) * a.heads + h) * a.vdim + v0 + c;
+                        if (oh && !raw) {
+                            const __nv_bfloat16 b = __float2bfloat16_rn(v);
+                            oh[at] = b;
+                            ol[at] = __float2bfloat16_rn(v - __bfloat162float(b));
+                        } else {
+                            a.out[at] = v;
+                        }
                     }
                 }
             }
@@ -600,14 +639,14 @@ __global__ void __launch_bounds__(RT_THREADS, 1) retention_runs_kernel(Retention
     __syncthreads();
     if (warp == 0) {
         tc_fence_after();
-        tmem_dealloc(tmem, 512);
+        tmem_dealloc(tmem, 256);
     }
 }
 
 int pad64(int n) { return (n + 63) / 64 * 64; }
 size_t runs_smem(int dim, int vdim) {
     const int Dp = pad64(dim), nv = std::min(pad64(vdim), 128);
-    return 1024 + (size_t)2 * (Dp / 64) * RT_BLK + (size_t)(nv / 64) * (RT_BLK + 2 * Dp * 128);
+    return 1024 + std::max((size_t)(2 * (Dp / 64) + nv / 64) * RT_BLK, (size_t)RT_RUN * (nv + 4) * 4);
 }
 constexpr size_t RT_GAIN_SMEM = 1024 + 6 * RT_BLK;
 
@@ -615,7 +654,7 @@ constexpr size_t RT_GAIN_SMEM = 1024 + 6 * RT_BLK;
 
 // state slots of the work buffer for a step of `rows` portion rows in `portions` portions
 int retention_ws_runs(int rows, int portions) { return rows / RT_RUN + portions + 1; }
-bool retention_tc_ok(int dim, int vdim) { return dim >= 1 && dim <= 128 && vdim >= 1 && runs_smem(dim, vdim) <= 220 * 1024; }
+bool retention_tc_ok(int dim, int vdim) { return dim >= 1 && dim <= 128 && vdim >= 1; }
 bool retention_one_pass(int vdim) { return vdim <= 128; }
 int retention_padded(int n) { return pad64(n); }
 
@@ -639,7 +678,7 @@ int launch_retention_tc(const RetentionArgs& a, const WindowTiles& tm, int first
     static PerDeviceFlag attr;
     if (!attr.done()) {
         FT_CHECK_CUDA(cudaFuncSetAttribute(retention_gain_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)RT_GAIN_SMEM));
-        FT_CHECK_CUDA(cudaFuncSetAttribute(retention_runs_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+        FT_CHECK_CUDA(cudaFuncSetAttribute(retention_runs_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024));
         attr.mark();
     }
     retention_pack_kernel<<<rows, 256, (size_t)a.rot_dims * 4, stream>>>(a, row0, Dp, Vp);
