@@ -100,6 +100,17 @@ __device__ __forceinline__ void mbar_wait(uint64_t* bar, uint32_t parity) {
     }
 }
 
+// Waits inside kernels that must end: false when the limit ran out here or another warp of the CTA has given up (*dead)
+constexpr int kWaitLimit = 1 << 20;
+__device__ __forceinline__ bool mbar_wait_limited(uint64_t* bar, uint32_t parity, volatile int* dead) {
+    for (int i = 0; i < kWaitLimit; ++i) {
+        if (mbar_try_wait(bar, parity)) return true;
+        if ((i & 31) == 31 && *dead) return false;
+    }
+    *dead = 1;
+    return false;
+}
+
 // ------------------------------------------------------------------ L2 cache policies
 __device__ __forceinline__ uint64_t policy_evict_first() {
     uint64_t p;

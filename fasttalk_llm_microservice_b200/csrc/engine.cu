@@ -202,15 +202,8 @@ struct Layered {
     int *ids = nullptr, *seg = nullptr, *slot_token = nullptr, *slot_pos = nullptr;
     void *pl_hi = nullptr, *pl_lo = nullptr;      // bf16 planes of a projection's input [t_max][k_max]
     void *hn_hi = nullptr, *hn_lo = nullptr;      // bf16 planes of the normed layer input [t_max][width]
-    // experts on the tensor cores: planes of the gathered rows, fp32 gate/up results, planes of the activations, and the
-    // segment table on the host (the per-expert launches need the row counts)
+    // experts on the tensor cores: planes of the gathered rows and of the activations
     void *mx_hi = nullptr, *mx_lo = nullptr, *ax_hi = nullptr, *ax_lo = nullptr;
-    float* gu = nullptr;
-    int* h_seg = nullptr;
-    // the per-expert GEMMs are small (a few dozen CTAs): they are dealt over the engine's stream and three side streams
-    static constexpr int kSide = 3;
-    cudaStream_t side[kSide] = {};
-    cudaEvent_t side_done[kSide] = {}, main_ready = nullptr;
     bool tensor = false;               // projections that tile run on the tensor cores (ft_layered_model.exact_f32 == 0)
     // post-norm layers: the stream as every layer left it [n_layers + 1][t_max][width] (the sum over depth reads them all), the
     // values of the first value-mixing attention layer of the step, the staging rows of latent window attention
@@ -588,7 +581,7 @@ static bool dense_tiles(const Engine* e, int T, int N, int K) { return e->lay->t
 constexpr int kAttnTcMinTokens = 32;         // portion tokens of a step from which attention over a bf16 cache takes 128-row tiles
 constexpr int kRetentionTcMinTokens = 32;    // portion tokens of a step from which a retention runs on the tensor cores
 constexpr int kFuseCanonRows = 256;          // steps up to this many rows form the feed-forward's input inside the post-norm kernel
-constexpr int kMoeTensorMinPairs = 256;      // (token, choice) pairs from which the experts run as per-expert tensor-core GEMMs
+constexpr int kMoeTensorMinPairs = 256;      // (token, choice) pairs from which the experts run on the tensor cores
 static int dense(Engine* e, const float* A, const void* hi, const void* lo, const void* W, float* C, int T, int N, int K,
                  float softcap = 0.f) {
     Layered& L = *e->lay;
@@ -654,52 +647,18 @@ static int run_experts(Engine* e, const ft_layer_desc& c, const float* logits, i
                         L.seg, L.slot_token, L.slot_pos, T, st, sandwich ? c.route_kind : FT_ROUTE_SOFTMAX,
                         sandwich ? c.route_norm : 0, sandwich ? c.route_scale : 1.f, sandwich ? c.router_bias : nullptr));
     const int pairs = T * top;
-    const bool on_tensor = L.tensor && pairs >= kMoeTensorMinPairs && n_up % 128 == 0 && c.ff % 64 == 0 && W % 128 == 0 &&
-                           W % 64 == 0;
+    const bool on_tensor = L.tensor && pairs >= kMoeTensorMinPairs && experts_tc_ok(n_up, W) && experts_tc_ok(W, c.ff);
     if (on_tensor) {
-        // One tcgen05 GEMM per expert over its run of sorted rows.  The launches need the run lengths on the host:
-        // a copy of E + 1 integers and a wait, a few microseconds against the milliseconds of such a step.
-        FT_CHECK_CUDA(cudaMemcpyAsync(L.h_seg, L.seg, (size_t)(c.experts + 1) * 4, cudaMemcpyDeviceToHost, st));
+        // every expert's run of sorted rows in one launch per matrix; the activation in the first one's epilogue
         if (scaled_in) FT_TRY(launch_scaled_rows(L.hn, L.wts, L.slot_pos, top, nullptr, L.mx_hi, L.mx_lo, pairs, W, st));
         else FT_TRY(launch_gather_planes_rows(L.hn, L.slot_token, L.mx_hi, L.mx_lo, pairs, W, st));
-        FT_CHECK_CUDA(cudaStreamSynchronize(st));
-        auto off = [](const void* p, size_t elems) { return (const void*)((const uint8_t*)p + elems * 2); };
-        ft_gemm_epilogue ep = {};
-        ep.mode = FT_EPI_PARTIAL;
-        auto lane_of = [&](int k) { return k % (Layered::kSide + 1) == 0 ? st : L.side[k % (Layered::kSide + 1) - 1]; };
-        auto join = [&]() -> int {          // the engine's stream waits for what the side streams were given
-            for (int k = 0; k < Layered::kSide; ++k) {
-                FT_CHECK_CUDA(cudaEventRecord(L.side_done[k], L.side[k]));
-                FT_CHECK_CUDA(cudaStreamWaitEvent(st, L.side_done[k], 0));
-            }
-            return 0;
-        };
-        FT_CHECK_CUDA(cudaEventRecord(L.main_ready, st));
-        for (int i = 0; i < Layered::kSide; ++i) FT_CHECK_CUDA(cudaStreamWaitEvent(L.side[i], L.main_ready, 0));
-        int k = 0;
-        for (int x = 0; x < c.experts; ++x) {
-            const int r0 = L.h_seg[x], nr = L.h_seg[x + 1] - r0;
-            if (nr <= 0) continue;
-            ep.out = L.gu + (size_t)r0 * n_up;
-            FT_TRY(ft_gemm_fused(off(c.w_gu, (size_t)x * n_up * W), off(L.mx_hi, (size_t)r0 * W),
-                                 off(L.mx_lo, (size_t)r0 * W), n_up, nr, W, 1, &ep, lane_of(k++)));
-            launched();
-        }
-        FT_TRY(join());
-        FT_TRY(launch_act_planes(L.gu, L.ax_hi, L.ax_lo, pairs, c.ff, act, glu, st));
-        FT_CHECK_CUDA(cudaEventRecord(L.main_ready, st));
-        for (int i = 0; i < Layered::kSide; ++i) FT_CHECK_CUDA(cudaStreamWaitEvent(L.side[i], L.main_ready, 0));
-        k = 0;
-        for (int x = 0; x < c.experts; ++x) {
-            const int r0 = L.h_seg[x], nr = L.h_seg[x + 1] - r0;
-            if (nr <= 0) continue;
-            ep.out = L.eout + (size_t)r0 * W;
-            FT_TRY(ft_gemm_fused(off(c.w_down, (size_t)x * W * c.ff), off(L.ax_hi, (size_t)r0 * c.ff),
-                                 off(L.ax_lo, (size_t)r0 * c.ff), W, nr, c.ff, 1, &ep, lane_of(k++)));
-            launched();
-        }
-        FT_TRY(join());
-        launched(4);
+        ExpertsTcArgs x;
+        x.w = c.w_gu; x.x_hi = L.mx_hi; x.x_lo = L.mx_lo; x.seg = L.seg; x.E = c.experts; x.n_rows = n_up; x.K = W; x.pairs = pairs;
+        x.act = act; x.glu = glu; x.out_hi = L.ax_hi; x.out_lo = L.ax_lo; x.err = e->h_kernel_err;
+        FT_TRY(launch_experts_tc(x, st));
+        x.w = c.w_down; x.x_hi = L.ax_hi; x.x_lo = L.ax_lo; x.n_rows = W; x.K = c.ff; x.out = L.eout;
+        FT_TRY(launch_experts_tc(x, st));
+        launched();
     } else {
         LinearArgs gu;                  // first matrix of every (token, choice) pair, grouped by expert, with its activation
         gu.A = L.hn; gu.a_rows = L.slot_token; gu.lda = W; gu.W = (const __nv_bfloat16*)c.w_gu;
@@ -2137,7 +2096,6 @@ static int engine_init_layered(Engine* e) {
         FT_TRY(alloc(&L.mx_lo, T * top_max * W * 2));
         FT_TRY(alloc(&L.ax_hi, T * top_max * act_cols * 2));
         FT_TRY(alloc(&L.ax_lo, T * top_max * act_cols * 2));
-        FT_TRY(alloc(&L.gu, T * top_max * act_cols * 2 * 4));
     }
     FT_TRY(alloc(&L.b1, T * buf * 4));
     FT_TRY(alloc(&L.b2, T * buf * 4));
@@ -2161,14 +2119,6 @@ static int engine_init_layered(Engine* e) {
         int e_max = 1;
         for (const LayeredLayer& ll : L.layers) e_max = std::max(e_max, ll.d.experts);
         FT_TRY(alloc(&L.seg, (size_t)(e_max + 1) * 4));
-        FT_CHECK_CUDA(cudaMallocHost(&L.h_seg, (size_t)(e_max + 1) * 4));
-        if (L.tensor) {
-            for (int k = 0; k < Layered::kSide; ++k) {
-                FT_CHECK_CUDA(cudaStreamCreateWithFlags(&L.side[k], cudaStreamNonBlocking));
-                FT_CHECK_CUDA(cudaEventCreateWithFlags(&L.side_done[k], cudaEventDisableTiming));
-            }
-            FT_CHECK_CUDA(cudaEventCreateWithFlags(&L.main_ready, cudaEventDisableTiming));
-        }
     }
     const size_t rows_last = std::max<size_t>(e->logit_rows, 256);
     e->rows_last = (int)rows_last;
@@ -2203,13 +2153,7 @@ static void engine_free(Engine* e) {
         cudaFree(L.floor); cudaFree(L.mix2); cudaFree(L.ffa); cudaFree(L.ffb); cudaFree(L.rlog);
         cudaFree(L.wts); cudaFree(L.xlast); cudaFree(L.ids); cudaFree(L.seg); cudaFree(L.slot_token);
         cudaFree(L.slot_pos); cudaFree(L.trail); cudaFree(L.pl_hi); cudaFree(L.pl_lo); cudaFree(L.hn_hi); cudaFree(L.hn_lo);
-        cudaFree(L.mx_hi); cudaFree(L.mx_lo); cudaFree(L.ax_hi); cudaFree(L.ax_lo); cudaFree(L.gu);
-        if (L.h_seg) cudaFreeHost(L.h_seg);
-        for (int k = 0; k < Layered::kSide; ++k) {
-            if (L.side[k]) cudaStreamDestroy(L.side[k]);
-            if (L.side_done[k]) cudaEventDestroy(L.side_done[k]);
-        }
-        if (L.main_ready) cudaEventDestroy(L.main_ready);
+        cudaFree(L.mx_hi); cudaFree(L.mx_lo); cudaFree(L.ax_hi); cudaFree(L.ax_lo);
         delete e->lay;
     }
     if (e->meta.h) cudaFreeHost(e->meta.h);

@@ -140,6 +140,20 @@ int launch_linear(const LinearArgs& a, int rows_bound, cudaStream_t stream);
 // 32-column pieces.  err as for launch_paged16_tc
 bool linear_heads_ok(const LinearArgs& a);
 int launch_linear_heads(const LinearArgs& a, int* err, cudaStream_t stream);
+// ---- experts_tc.cu: one matrix of every expert over the sorted (token, choice) pairs, seg as launch_route leaves it.  x: planes
+// [pairs][K]; w [E][n_rows][K].  out: fp32 [pairs][n_rows]; without it the activation's planes, [pairs][n_rows / 2] for the (gate, up)
+// forms or [pairs][n_rows] for FT_ACT_RELU2.  err as for launch_paged16_tc
+struct ExpertsTcArgs {
+    const void *w = nullptr, *x_hi = nullptr, *x_lo = nullptr;
+    const int* seg = nullptr;
+    int E = 0, n_rows = 0, K = 0, pairs = 0, act = 0;
+    GluSpec glu;
+    float* out = nullptr;
+    void *out_hi = nullptr, *out_lo = nullptr;
+    int* err = nullptr;
+};
+bool experts_tc_ok(int n_rows, int K);
+int launch_experts_tc(const ExpertsTcArgs& a, cudaStream_t stream);
 // hi / lo (may be null): the normed row once more as bf16 planes, the input form of the tensor-core projections
 // gain_w (may be null): a gain per coordinate instead of the single `gain`
 int launch_embed_norm(const int* tokens, const void* embed, float* x, float* hn, void* hi, void* lo, int T, int W, float eps,

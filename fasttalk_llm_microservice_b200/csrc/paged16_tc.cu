@@ -39,7 +39,6 @@ constexpr int LT_COL_O = 0;
 template <int PER_SM> struct LtTmem { static constexpr int COLS = 512, S = 256, Q = 384, Q2 = 128, NBUF = 2, QB = 5; };
 template <> struct LtTmem<2> { static constexpr int COLS = 256, S = 128, Q = 192, Q2 = 0, NBUF = 1, QB = 2; };
 constexpr float LT_RESCALE = 8.f;                      // log2 units
-constexpr int LT_SPIN = 1 << 20;
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr int LT_OUT_LD = 36;                          // floats per row of a warp's output staging (32 columns)
 constexpr size_t LT_SMEM_MAX = 227 * 1024;
@@ -67,16 +66,6 @@ bool paged_tc_cfg(const Paged16Args& a, PagedTcCfg& c) {
     c.stages = (int)std::min<size_t>(LT_MAX_STAGES, (room - fixed) / ((size_t)c.sblk * LT_SLAB));
     c.smem = fixed + (size_t)std::max(c.stages, 0) * c.sblk * LT_SLAB;
     return c.stages >= 2;
-}
-
-// false: the limit ran out here or another warp of the CTA has given up
-__device__ __forceinline__ bool wait_limited(uint64_t* bar, uint32_t parity, volatile int* dead) {
-    for (int i = 0; i < LT_SPIN; ++i) {
-        if (mbar_try_wait(bar, parity)) return true;
-        if ((i & 31) == 31 && *dead) return false;
-    }
-    *dead = 1;
-    return false;
 }
 
 template <int PER_SM>
@@ -147,7 +136,7 @@ paged16_tc_kernel(Paged16Args a, WindowTiles tm, PagedTcCfg cfg, int subs, int* 
                 const int page = __shfl_sync(0xffffffffu, my_page, i);
                 if (lane == 0) {
                     const int s = issued % cfg.stages, round = issued / cfg.stages;
-                    ok = wait_limited(&kv_empty[s], (round & 1) ^ 1, dead);
+                    ok = mbar_wait_limited(&kv_empty[s], (round & 1) ^ 1, dead);
                     if (ok) {
                         const uint8_t* src = (const uint8_t*)a.cache + ((size_t)page * a.G + kv_head) * a.blocks * LT_SLAB;
                         uint8_t* dst = kv_s + (size_t)s * stage_bytes;
@@ -163,7 +152,7 @@ paged16_tc_kernel(Paged16Args a, WindowTiles tm, PagedTcCfg cfg, int subs, int* 
         }
         if (!ok && lane == 0)                                          // copies in flight land before the CTA's memory goes away
             for (int k = max(0, issued - cfg.stages); k < issued; ++k)
-                for (int i = 0; i < LT_SPIN && !mbar_try_wait(&kv_full[k % cfg.stages], (k / cfg.stages) & 1); ++i) {}
+                for (int i = 0; i < kWaitLimit && !mbar_try_wait(&kv_full[k % cfg.stages], (k / cfg.stages) & 1); ++i) {}
     } else if (warp == 1) {
         // ---------------------------------------------------------------- products
         if (elect_one()) {
@@ -189,17 +178,17 @@ paged16_tc_kernel(Paged16Args a, WindowTiles tm, PagedTcCfg cfg, int subs, int* 
                 }
                 umma_commit(&s_full[j % NBUF]);
             };
-            bool ok = wait_limited(q_full, 0, dead);
+            bool ok = mbar_wait_limited(q_full, 0, dead);
             tc_fence_after();
             for (int j = 0; j < NBUF && j < n_tiles && ok; ++j) {
-                ok = wait_limited(&kv_full[j % cfg.stages], (j / cfg.stages) & 1, dead);
+                ok = mbar_wait_limited(&kv_full[j % cfg.stages], (j / cfg.stages) & 1, dead);
                 tc_fence_after();
                 if (ok) issue_qk(j);
             }
             const bool ahead = cfg.stages > NBUF;                      // page j + NBUF does not wait for the products of page j
             for (int j = 0; j < n_tiles && ok; ++j) {
-                if (ahead && j + NBUF < n_tiles) ok = wait_limited(&kv_full[(j + NBUF) % cfg.stages], ((j + NBUF) / cfg.stages) & 1, dead);
-                ok = ok && wait_limited(&p_full[j % NBUF], (j / NBUF) & 1, dead);      // P(j) written, S(j) consumed, O rescaled if needed
+                if (ahead && j + NBUF < n_tiles) ok = mbar_wait_limited(&kv_full[(j + NBUF) % cfg.stages], ((j + NBUF) / cfg.stages) & 1, dead);
+                ok = ok && mbar_wait_limited(&p_full[j % NBUF], (j / NBUF) & 1, dead);      // P(j) written, S(j) consumed, O rescaled if needed
                 if (!ok) break;
                 tc_fence_after();
                 const uint32_t p = tmem + TM::S + (j % NBUF) * 64, v_addr = stage_at(j) + (apart ? cfg.nblk : v0 >> 6) * LT_SLAB;
@@ -209,14 +198,14 @@ paged16_tc_kernel(Paged16Args a, WindowTiles tm, PagedTcCfg cfg, int subs, int* 
                     umma_f16_ts(tmem + LT_COL_O, p + 8 * k, vd + k * (2048 >> 4), idesc_pv, (j | k) != 0);
                 umma_commit(&kv_empty[j % cfg.stages]);
                 if (j + NBUF < n_tiles) {
-                    if (!ahead) ok = wait_limited(&kv_full[(j + NBUF) % cfg.stages], ((j + NBUF) / cfg.stages) & 1, dead);
+                    if (!ahead) ok = mbar_wait_limited(&kv_full[(j + NBUF) % cfg.stages], ((j + NBUF) / cfg.stages) & 1, dead);
                     tc_fence_after();
                     if (ok) issue_qk(j + NBUF);                           // behind the product that reads P out of this buffer
                 }
             }
             if (!ok) {
                 umma_commit(drain);
-                for (int i = 0; i < LT_SPIN && !mbar_try_wait(drain, 0); ++i) {}
+                for (int i = 0; i < kWaitLimit && !mbar_try_wait(drain, 0); ++i) {}
             }
         }
     } else {
@@ -261,7 +250,7 @@ paged16_tc_kernel(Paged16Args a, WindowTiles tm, PagedTcCfg cfg, int subs, int* 
         float m_ref = -INFINITY, l_run = 0.f;                          // log2 units
         bool ok = true;
         for (int j = 0; j < n_tiles; ++j) {
-            ok = __all_sync(0xffffffffu, wait_limited(&s_full[j % NBUF], (j / NBUF) & 1, dead));
+            ok = __all_sync(0xffffffffu, mbar_wait_limited(&s_full[j % NBUF], (j / NBUF) & 1, dead));
             if (!ok) break;
             tc_fence_after();
             const uint32_t s_addr = lanes + TM::S + (j % NBUF) * 64;
@@ -285,7 +274,7 @@ paged16_tc_kernel(Paged16Args a, WindowTiles tm, PagedTcCfg cfg, int subs, int* 
             if (j == 0) {
                 m_ref = m_new;                                         // finite: position 0 is visible to every row
             } else if (__any_sync(0xffffffffu, m_new > m_ref + LT_RESCALE)) {      // tcgen05.ld / st move whole warps
-                ok = __all_sync(0xffffffffu, wait_limited(&kv_empty[(j - 1) % cfg.stages], ((j - 1) / cfg.stages) & 1, dead));
+                ok = __all_sync(0xffffffffu, mbar_wait_limited(&kv_empty[(j - 1) % cfg.stages], ((j - 1) / cfg.stages) & 1, dead));
                 if (!ok) break;
                 tc_fence_after();
                 const float alpha = exp2f(m_ref - m_new);
@@ -321,7 +310,7 @@ paged16_tc_kernel(Paged16Args a, WindowTiles tm, PagedTcCfg cfg, int subs, int* 
             __syncwarp();
             if (lane == 0) mbar_arrive(&p_full[j % NBUF]);
         }
-        if (ok) ok = __all_sync(0xffffffffu, wait_limited(&kv_empty[(n_tiles - 1) % cfg.stages], ((n_tiles - 1) / cfg.stages) & 1, dead));
+        if (ok) ok = __all_sync(0xffffffffu, mbar_wait_limited(&kv_empty[(n_tiles - 1) % cfg.stages], ((n_tiles - 1) / cfg.stages) & 1, dead));
         if (ok) {
             tc_fence_after();
             float f = 1.f;
