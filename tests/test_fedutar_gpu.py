@@ -485,6 +485,25 @@ def test_projections_and_experts_on_tensor_cores(exact):
         eng.close()
 
 
+@pytest.mark.parametrize("experts,top,ff,skew", [(4, 1, 64, False), (40, 3, 64, False), (70, 2, 128, False), (40, 2, 64, True)],
+                         ids=["few", "forty", "seventy", "skewed"])
+def test_many_experts_in_one_launch(experts, top, ff, skew):
+    """Experts with no pair, a few pairs and several tiles of 128 pairs in one launch, tiles found from the segment table across more
+    than one warp's worth of experts.  The mixer adds nothing here, so the router sees what the restatement sees and no choice is close."""
+    def tweak(w):
+        only("left", w)
+        only("right", w)
+    spec, w = make([layer(parallel(), moe(ff=ff, experts=experts, top=top, limit=0.9))], width=128, vocab=256, seed=61, tweak=tweak)
+    toks = [11] * 430 + tokens_of(spec, 70, 62) if skew else tokens_of(spec, 500, 62)
+    ref = oracle_logits(spec, w, toks)
+    eng = engine(spec, w, exact_f32=False)
+    try:
+        assert rel(eng.feed([("a", toks, list(range(500)))]), ref) < 4e-4
+        assert rel(feed_cut(eng, "b", toks, [300, 1, 9, 130, 2, 58]), ref) < 4e-4
+    finally:
+        eng.close()
+
+
 # ------------------------------------------------------------------------------------------------ the serving path
 def greedy_oracle(spec, w, prompt, n):
     toks = list(prompt)
