@@ -402,7 +402,7 @@ def test_pages_and_slots_are_used_again(exact):
 
 
 # ------------------------------------------------------------------------------------------------ tensor cores
-@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 4, 32, 32), (6, 2, 96, 192), (8, 2, 128, 128), (5, 1, 20, 33), (16, 1, 64, 64), (40, 2, 16, 8),
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 4, 32, 32), (10, 2, 96, 160), (8, 2, 128, 128), (5, 1, 20, 33), (16, 1, 64, 64), (40, 2, 16, 8),
                                                      (2, 2, 200, 100), (4, 2, 256, 256), (3, 3, 64, 300), (2, 1, 130, 512), (1, 1, 5, 3), (2, 1, 300, 20)])
 @pytest.mark.parametrize("sharp", [1.0, 6.0], ids=["plain", "sharp"])
 def test_attention_on_tensor_cores(heads, kv_heads, dim, vdim, sharp):
